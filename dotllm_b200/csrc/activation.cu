@@ -72,7 +72,7 @@ extern "C" int dl_gated_activation(const void* gate, const void* up, int in_stri
     return DL_OK;
 }
 
-// An activation of one product (gating.cuh: the kinds that read no gate, e.g. relu(x)^2): out = act(x), float32 arithmetic.
+// An activation of one product (gating.cuh: the kinds that read no gate, relu(x)^2, gelu(x)): out = act(x), float32 arithmetic.
 // x: [rows, width] with rows in_stride apart; out: contiguous [rows, width].
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -80,7 +80,7 @@ unary_activation_kernel(const T* __restrict__ x, int in_stride, T* __restrict__ 
     const size_t n = (size_t)rows * width;
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
         const size_t r = i / width, c = i - r * width;
-        out[i] = dl_from_f32<T>(dl_gate_value(kind, 0.f, dl_to_f32<T>(x[r * in_stride + c]), 0.f, 0.f));
+        out[i] = dl_from_f32<T>(dl_unary_value(kind, dl_to_f32<T>(x[r * in_stride + c])));
     }
 }
 

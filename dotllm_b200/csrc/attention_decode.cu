@@ -280,6 +280,10 @@ struct AdFresh {
     // two options of the mask and of the softmax that travel with the others
     int keep_first;                  // with a window: the sequence's first keys that stay visible behind it
     const float* sinks;              // [nh] float32 or NULL: one more term exp(sinks[head]) in the head's denominator, no key, no value
+    DlScoreCap cap;                  // post > 0: scaled scores s become c tanh(s / c) before the softmax
+    int pool_heads;                  // KV heads of the pages; nkv is a multiple of it: neighbouring KV heads of the launch then read
+                                     // (and, for the step's own token, write) the same head of the pages, so that more query heads
+                                     // than a tile has rows can share one
 };
 
 // The same roundings as the rope kernels (no contraction), so that the fused and the separate way
@@ -418,6 +422,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int g = lane >> 2, t = lane & 3;
     const AdWin window = {window_size, window_size > 0 ? fresh.keep_first : 0};
+    const int pkv = fresh.pool_heads, per_pool = nkv / pkv;      // heads of the pages, heads of the launch that share one
     // The kernel checks its own shared-memory layout: if the launch gave it less dynamic shared
     // memory than the stages and merge buffers need, it records status 11 and touches nothing.
     uint32_t smem_bytes;
@@ -476,8 +481,8 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_
                             }
                             __nv_bfloat16* dst = stage_mem + (size_t)s * 2 * PAGE_ELEMS;
                             ad_mbar_expect(&full_bar[s], 2 * PAGE_BYTES);
-                            ad_bulk_copy(dst, k_pool + dl_k_offset(page, nkv, w.kvh, 0, HD), PAGE_BYTES, &full_bar[s], policy);
-                            ad_bulk_copy(dst + PAGE_ELEMS, v_pool + dl_v_offset(page, nkv, w.kvh, 0, HD), PAGE_BYTES, &full_bar[s], policy);
+                            ad_bulk_copy(dst, k_pool + dl_k_offset(page, pkv, w.kvh / per_pool, 0, HD), PAGE_BYTES, &full_bar[s], policy);
+                            ad_bulk_copy(dst + PAGE_ELEMS, v_pool + dl_v_offset(page, pkv, w.kvh / per_pool, 0, HD), PAGE_BYTES, &full_bar[s], policy);
                         }
                     }
                     bad = __shfl_sync(0xffffffffu, bad, 0);
@@ -501,7 +506,8 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_
         // The cut needs the lengths only, which are older than the kernel before this one: it is made
         // while that kernel finishes, and q is waited for after it.
         float* my_o = merge_o + (size_t)warp * group * (HD + 4);
-        const float scale2 = scale * 1.4426950408889634f;    // scores in units of log2
+        const bool capped = fresh.cap.post > 0.f;
+        const float scale2 = capped ? 1.f : scale * 1.4426950408889634f;    // scores in units of log2 (capped ones come in them)
         int n0 = 0;                                          // pages of the runs before this one
         const AdCut cut = ad_cut(seq_len, n_seqs, nkv, window, gridDim.x, lane);
         AdWalk walk = ad_walk_begin(cut, seq_len, n_seqs, nkv, window, blockIdx.x, lane);
@@ -562,8 +568,8 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_
             float4 kn_blo = make_float4(0.f, 0.f, 0.f, 0.f), kn_bhi = make_float4(0.f, 0.f, 0.f, 0.f);   // the new key's biases
             __nv_bfloat16 vn_r[HD / 32];
             if (mine_new) {
-                const __nv_bfloat16* kn = fresh.k + (size_t)w.b * fresh.k_stride + (size_t)w.kvh * HD;
-                const __nv_bfloat16* vn = fresh.v + (size_t)w.b * fresh.v_stride + (size_t)w.kvh * HD;
+                const __nv_bfloat16* kn = fresh.k + (size_t)w.b * fresh.k_stride + (size_t)(w.kvh / per_pool) * HD;
+                const __nv_bfloat16* vn = fresh.v + (size_t)w.b * fresh.v_stride + (size_t)(w.kvh / per_pool) * HD;
                 const int pos = min(w.len - 1, fresh.table_rows - 1);
                 if (lane * 4 < HD / 2) {                         // four rotation pairs per lane (HD <= 256)
                     kn_lo = *reinterpret_cast<const uint2*>(kn + lane * 4);
@@ -573,7 +579,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_
                         kn_s = *reinterpret_cast<const float4*>(fresh.sin_t + (size_t)pos * (HD / 2) + lane * 4);
                     }
                     if (fresh.k_bias != nullptr) {
-                        const float* kb = fresh.k_bias + (size_t)w.kvh * HD;
+                        const float* kb = fresh.k_bias + (size_t)(w.kvh / per_pool) * HD;
                         kn_blo = make_float4(kb[lane * 4], kb[lane * 4 + 1], kb[lane * 4 + 2], kb[lane * 4 + 3]);
                         kn_bhi = make_float4(kb[HD / 2 + lane * 4], kb[HD / 2 + lane * 4 + 1], kb[HD / 2 + lane * 4 + 2], kb[HD / 2 + lane * 4 + 3]);
                     }
@@ -582,7 +588,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_
                 for (int j = 0; j < HD / 32; ++j) {
                     vn_r[j] = vn[lane + 32 * j];
                     if (fresh.v_bias != nullptr)
-                        vn_r[j] = __float2bfloat16_rn(__bfloat162float(vn_r[j]) + fresh.v_bias[(size_t)w.kvh * HD + lane + 32 * j]);
+                        vn_r[j] = __float2bfloat16_rn(__bfloat162float(vn_r[j]) + fresh.v_bias[(size_t)(w.kvh / per_pool) * HD + lane + 32 * j]);
                 }
             }
             for (int i = i_first; i < w.n_pages; i += n_stages) {
@@ -630,7 +636,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_
                         *reinterpret_cast<uint2*>(kp + in_page * HD + i4) = *reinterpret_cast<uint2*>(lo);
                         *reinterpret_cast<uint2*>(kp + in_page * HD + HD / 2 + i4) = *reinterpret_cast<uint2*>(hi);
                         if (page >= 0 && page < n_pages) {
-                            __nv_bfloat16* kg = k_pool + dl_k_offset(page, nkv, w.kvh, in_page, HD);
+                            __nv_bfloat16* kg = k_pool + dl_k_offset(page, pkv, w.kvh / per_pool, in_page, HD);
                             *reinterpret_cast<uint2*>(kg + i4) = *reinterpret_cast<uint2*>(lo);
                             *reinterpret_cast<uint2*>(kg + HD / 2 + i4) = *reinterpret_cast<uint2*>(hi);
                         }
@@ -639,7 +645,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_
                     for (int j = 0; j < HD / 32; ++j) {
                         const int d = lane + 32 * j;
                         vp[d * DL_PAGE + in_page] = vn_r[j];
-                        if (page >= 0 && page < n_pages) v_pool[dl_v_offset(page, nkv, w.kvh, d, HD) + in_page] = vn_r[j];
+                        if (page >= 0 && page < n_pages) v_pool[dl_v_offset(page, pkv, w.kvh / per_pool, d, HD) + in_page] = vn_r[j];
                     }
                     __syncwarp();
                 }
@@ -703,6 +709,14 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_
 #pragma unroll
                         for (int j = 0; j < 4; ++j)
                             ad_mma(sc[h][j], qf_lo[c].z, qf_hi[c].z, qf_lo[c].w, qf_hi[c].w, kf[h][j].z, kf[h][j].w);
+                }
+                if (capped) {                                 // before the mask: a hidden key's score is replaced, not capped
+#pragma unroll
+                    for (int h = 0; h < 2; ++h)
+#pragma unroll
+                        for (int j = 0; j < 4; ++j)
+#pragma unroll
+                            for (int e = 0; e < (WIDE ? 4 : 2); ++e) sc[h][j][e] = dl_capped_score(sc[h][j][e], fresh.cap);
                 }
                 // ---- mask (ragged pages only; lane holds keys base + 32h + 8t + 2j + {0,1}) and row maximum
                 if (ragged) {
@@ -942,6 +956,8 @@ static int ad_launch(cudaStream_t s, const void* q, int q_stride, void* out, int
 // q: bf16 [B, nh*hd] rows q_stride apart (one token per sequence); out likewise.
 // seq_len[b]: keys of sequence b including the new token; block_table: int32 [B, bt_stride] page ids.
 // blocks: persistent blocks to use (<= 0: one per multiprocessor).
+// sinks: float32 [nh] or NULL; softcap: 0 for none, else scaled scores s become softcap * tanh(s / softcap).
+// pool_heads: KV heads of the pages (usually nkv); a divisor of nkv lets neighbouring KV heads of the launch share one.
 // part_o: float32 [part_slots, group, hd]; part_ml: float32 [part_slots, group, 2]: scratch for the
 // segments of (sequence, head) pairs that the cut spreads over several blocks, two per block.
 // pair_counters: int32 [n_counters >= n_seqs * nkv], zero before the first launch; every launch leaves
@@ -957,6 +973,7 @@ static int ad_dispatch(const void* q, int q_stride, void* out, int out_stride, v
     DL_REQUIRE(n_seqs >= 0 && nh > 0 && nkv > 0 && nh % nkv == 0, "attention_decode: bad head counts");
     DL_REQUIRE(nh / nkv <= 16, "attention_decode: groups of more than 16 query heads are not supported (%d)", nh / nkv);
     DL_REQUIRE(scale > 0.f, "attention_decode: the score scale must be positive");
+    DL_REQUIRE(fresh.pool_heads >= 1 && nkv % fresh.pool_heads == 0, "attention_decode: %d KV heads do not share %d heads of the pages evenly", nkv, fresh.pool_heads);
     DL_REQUIRE(part_o && part_ml && part_slots >= 2, "attention_decode: needs scratch for the cut segments");
     DL_REQUIRE(status != nullptr, "attention_decode: needs a status word");
     DL_REQUIRE(bt_stride >= 1 && window >= 0, "attention_decode: bad block table stride or window");
@@ -966,7 +983,7 @@ static int ad_dispatch(const void* q, int q_stride, void* out, int out_stride, v
     DL_REQUIRE((long long)n_seqs * nkv * bt_stride < (1ll << 30) && n_seqs <= 65535, "attention_decode: too many pages");
     if (fresh.k != nullptr) {
         DL_REQUIRE(fresh.v != nullptr && fresh.k_stride % 4 == 0 && fresh.v_stride % 4 == 0 && ((uintptr_t)fresh.k % 8) == 0 &&
-                       ((uintptr_t)fresh.v % 8) == 0 && fresh.k_stride >= nkv * hd && fresh.v_stride >= nkv * hd,
+                       ((uintptr_t)fresh.v % 8) == 0 && fresh.k_stride >= fresh.pool_heads * hd && fresh.v_stride >= fresh.pool_heads * hd,
                    "attention_decode: the new keys and values must be 8-byte aligned rows of nkv*hd");
     }
     DL_REQUIRE(!fresh.rotate || ((hd == 64 || hd == 128) && fresh.cos_t && fresh.sin_t && fresh.table_rows > 0 &&
@@ -995,13 +1012,16 @@ static int ad_dispatch(const void* q, int q_stride, void* out, int out_stride, v
 extern "C" int dl_attention_decode_bf16(const void* q, int q_stride, void* out, int out_stride, const void* k_pool,
                                         const void* v_pool, int n_pages, const int32_t* seq_len,
                                         const int32_t* block_table, int bt_stride, int n_seqs, int nh, int nkv,
-                                        int hd, float scale, int window, int keep_first, const float* sinks, int blocks,
+                                        int hd, float scale, int window, int keep_first, const float* sinks, float softcap, int pool_heads,
+                                        int blocks,
                                         float* part_o, float* part_ml, int part_slots, int* pair_counters, int n_counters,
                                         int* status, void* stream) {
     DL_REQUIRE(keep_first >= 0 && (keep_first == 0 || window > 0), "attention_decode: kept first keys need a window");
     AdFresh none = {};
     none.keep_first = keep_first;
     none.sinks = sinks;
+    none.cap = dl_score_cap(softcap, scale);
+    none.pool_heads = pool_heads;
     return ad_dispatch(q, q_stride, out, out_stride, const_cast<void*>(k_pool), const_cast<void*>(v_pool), n_pages, seq_len,
                        block_table, bt_stride, n_seqs, nh, nkv, hd, scale, window, blocks, part_o, part_ml, part_slots,
                        pair_counters, n_counters, none, status, stream);
@@ -1030,6 +1050,7 @@ extern "C" int dl_attention_decode_fresh_bf16(const void* q, int q_stride, const
     fresh.sin_t = sin_t;
     fresh.table_rows = table_rows;
     fresh.rotate = rotate;
+    fresh.pool_heads = nkv;
     return ad_dispatch(q, q_stride, out, out_stride, k_pool, v_pool, n_pages, seq_len, block_table, bt_stride, n_seqs, nh, nkv,
                        hd, scale, window, blocks, part_o, part_ml, part_slots, pair_counters, n_counters, fresh, status, stream);
 }
@@ -1038,11 +1059,12 @@ extern "C" int dl_attention_decode_fresh_bf16(const void* q, int q_stride, const
 // [nkv*hd] (float32, each NULL for none) are added before the rotation, with one rounding behind it as in
 // dl_rope_cache_write; gate (bfloat16, one logit per (sequence, query head), rows gate_stride apart, or NULL) multiplies
 // a head's output by sigmoid(logit) where it is written.  k_new and v_new may be NULL: a layer that reads another
-// layer's cache only biases and rotates its queries, and writes nothing to the pages.
+// layer's cache only biases and rotates its queries, and writes nothing to the pages.  sinks, softcap and pool_heads as in
+// dl_attention_decode_bf16.
 extern "C" int dl_attention_decode_gated_bf16(const void* q, int q_stride, const void* k_new, int k_stride, const void* v_new,
                                               int v_stride, const float* cos_t, const float* sin_t, int table_rows, int rotate,
                                               const float* q_bias, const float* k_bias, const float* v_bias, const void* gate,
-                                              int gate_stride, void* out, int out_stride, void* k_pool, void* v_pool, int n_pages,
+                                              int gate_stride, const float* sinks, float softcap, int pool_heads, void* out, int out_stride, void* k_pool, void* v_pool, int n_pages,
                                               const int32_t* seq_len, const int32_t* block_table, int bt_stride, int n_seqs,
                                               int nh, int nkv, int hd, float scale, int window, int blocks, float* part_o,
                                               float* part_ml, int part_slots, int* pair_counters, int n_counters, int* status,
@@ -1062,6 +1084,9 @@ extern "C" int dl_attention_decode_gated_bf16(const void* q, int q_stride, const
     fresh.v_bias = v_bias;
     fresh.gate = (const __nv_bfloat16*)gate;
     fresh.gate_stride = gate_stride;
+    fresh.sinks = sinks;
+    fresh.cap = dl_score_cap(softcap, scale);
+    fresh.pool_heads = pool_heads;
     return ad_dispatch(q, q_stride, out, out_stride, k_pool, v_pool, n_pages, seq_len, block_table, bt_stride, n_seqs, nh, nkv,
                        hd, scale, window, blocks, part_o, part_ml, part_slots, pair_counters, n_counters, fresh, status, stream);
 }

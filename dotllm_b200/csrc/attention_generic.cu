@@ -25,7 +25,8 @@
 #include "common.cuh"
 
 #define AG_WARPS 4
-#define AG_MAX_HD 512
+#define AG_MAX_HD 512                     // value channels a head: what a lane keeps in registers
+#define AG_MAX_KEY 2048                   // key channels a head: what shared memory holds of the queries
 
 template <typename T>
 __global__ void __launch_bounds__(32 * AG_WARPS)
@@ -245,7 +246,7 @@ extern "C" int dl_attention_generic(const void* q, int q_stride, void* out, int 
     DL_REQUIRE(vd <= AG_MAX_HD, "attention: value width %d exceeds the supported maximum %d", vd, AG_MAX_HD);
     DL_REQUIRE(gate == nullptr || gate_stride >= nh, "attention: a row of gate logits holds one per query head");
     DL_REQUIRE(nh % nkv == 0, "attention: %d query heads are not a multiple of %d KV heads", nh, nkv);
-    DL_REQUIRE(hd <= AG_MAX_HD, "attention: head_dim %d exceeds the supported maximum %d", hd, AG_MAX_HD);
+    DL_REQUIRE(hd <= AG_MAX_KEY, "attention: head_dim %d exceeds the supported maximum %d", hd, AG_MAX_KEY);
     DL_REQUIRE(q_stride >= nh * hd && out_stride >= nh * vd, "attention: row strides shorter than the rows");
     DL_REQUIRE(window >= 0, "attention: window must be 0 (none) or positive");
     DL_REQUIRE(keep_first >= 0, "attention: the number of kept first tokens cannot be negative");

@@ -88,7 +88,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
                          const int32_t* __restrict__ seq_start, const int32_t* __restrict__ seq_new,
                          const int32_t* __restrict__ cu_new, const int32_t* __restrict__ block_table,
                          int bt_stride, int nh, int nkv, float scale, int window, int keep_first,
-                         const float* __restrict__ sinks, int* __restrict__ status) {
+                         const float* __restrict__ sinks, const DlScoreCap cap, int* __restrict__ status) {
     constexpr int DC = HD / 32;
     constexpr int DT = HD / 8;
     constexpr int PAGE_ELEMS = DL_PAGE * HD;
@@ -166,7 +166,8 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
         const int first_lo = (window > 0) ? pos_lo - window + 1 : 0;
         const int first_hi = (window > 0) ? pos_hi - window + 1 : 0;
         const int warp_first = (window > 0 && warp_pos_min - window + 1 > 0) ? warp_pos_min - window + 1 : 0;
-        const float scale2 = scale * 1.4426950408889634f;    // scores in units of log2
+        const bool capped = cap.post > 0.f;
+        const float scale2 = capped ? 1.f : scale * 1.4426950408889634f;    // scores in units of log2 (capped ones come in them)
 
         uint4 qf_lo[DC], qf_hi[DC];
 #pragma unroll
@@ -224,6 +225,14 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
 #pragma unroll
                         for (int j = 0; j < 4; ++j)
                             ap_mma(sc[hh][j], qf_lo[c].z, qf_hi[c].z, qf_lo[c].w, qf_hi[c].w, kf[hh][j].z, kf[hh][j].w);
+                }
+                if (capped) {                                 // before the mask: a hidden key's score is replaced, not capped
+#pragma unroll
+                    for (int hh = 0; hh < 2; ++hh)
+#pragma unroll
+                        for (int j = 0; j < 4; ++j)
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) sc[hh][j][e] = dl_capped_score(sc[hh][j][e], cap);
                 }
                 if (ragged) {
                     // lane holds keys base + 32hh + 8t + 2j + {0,1} of rows g (lo) and g+8 (hi).  Masked
@@ -349,7 +358,7 @@ static int ap_launch(dim3 grid, cudaStream_t s, const void* q, int q_stride, voi
                      const void* k_pool, const void* v_pool, int n_pages, const int32_t* tile_seq,
                      const int32_t* tile_row0, const int32_t* seq_start, const int32_t* seq_new,
                      const int32_t* cu_new, const int32_t* block_table, int bt_stride, int nh, int nkv, float scale,
-                     int window, int keep_first, const float* sinks, int* status) {
+                     int window, int keep_first, const float* sinks, float softcap, int* status) {
     const size_t smem = (size_t)AP_STAGES * 2 * DL_PAGE * HD * 2;
     static bool configured = false;
     if (!configured) {
@@ -360,7 +369,7 @@ static int ap_launch(dim3 grid, cudaStream_t s, const void* q, int q_stride, voi
     attention_prefill_kernel<HD><<<grid, AP_THREADS, smem, s>>>(
         (const __nv_bfloat16*)q, q_stride, (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)k_pool,
         (const __nv_bfloat16*)v_pool, n_pages, tile_seq, tile_row0, seq_start, seq_new, cu_new, block_table, bt_stride,
-        nh, nkv, scale, window, keep_first, sinks, status);
+        nh, nkv, scale, window, keep_first, sinks, dl_score_cap(softcap, scale), status);
     DL_CHECK_LAUNCH("attention_prefill");
     return DL_OK;
 }
@@ -369,13 +378,13 @@ static int ap_launch(dim3 grid, cudaStream_t s, const void* q, int q_stride, voi
 // 128-row tile its sequence and its first row among that sequence's new tokens.  seq_start,
 // seq_new: cached length before the step and new tokens, per sequence; cu_new: packed offsets.
 // keep_first: with a window, that many first keys of a sequence stay visible.  sinks: float32 [nh] or NULL, exp(sinks[h])
-// joins head h's softmax denominator.  status: int32, set non-zero if a wait expired.
+// joins head h's softmax denominator.  softcap: 0 for none, else scaled scores s become softcap * tanh(s / softcap).  status: int32, set non-zero if a wait expired.
 extern "C" int dl_attention_prefill_bf16(const void* q, int q_stride, void* out, int out_stride,
                                          const void* k_pool, const void* v_pool, int n_pages,
                                          const int32_t* tile_seq, const int32_t* tile_row0, int n_tiles,
                                          const int32_t* seq_start, const int32_t* seq_new, const int32_t* cu_new,
                                          const int32_t* block_table, int bt_stride, int nh, int nkv, int hd,
-                                         float scale, int window, int keep_first, const float* sinks, int* status,
+                                         float scale, int window, int keep_first, const float* sinks, float softcap, int* status,
                                          void* stream) {
     DL_REQUIRE(n_tiles >= 0 && nh > 0 && nkv > 0 && nh % nkv == 0, "attention_prefill: bad sizes");
     DL_REQUIRE(scale > 0.f, "attention_prefill: the score scale must be positive");
@@ -392,7 +401,7 @@ extern "C" int dl_attention_prefill_bf16(const void* q, int q_stride, void* out,
 #define AP_CASE(HDV)                                                                                                  \
     if (hd == HDV)                                                                                                    \
         return ap_launch<HDV>(grid, s, q, q_stride, out, out_stride, k_pool, v_pool, n_pages, tile_seq, tile_row0,     \
-                              seq_start, seq_new, cu_new, block_table, bt_stride, nh, nkv, scale, window, keep_first, sinks, status);
+                              seq_start, seq_new, cu_new, block_table, bt_stride, nh, nkv, scale, window, keep_first, sinks, softcap, status);
     AP_CASE(32) AP_CASE(64) AP_CASE(96) AP_CASE(128)
 #undef AP_CASE
     return dl_fail(DL_ERR_UNSUPPORTED, "attention_prefill: head_dim %d (takes 32, 64, 96, 128)", hd);

@@ -86,14 +86,15 @@ struct PtTile {
     int j_lo, j_hi;          // the pages of the block's walk it takes part in (j_lo > j_hi: none)
 };
 
-template <int HD>
+// CAP: scaled scores s become c tanh(s / c) before the softmax.
+template <int HD, bool CAP>
 __global__ void __launch_bounds__(PT_THREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                             const __grid_constant__ CUtensorMap tmap_v, __nv_bfloat16* __restrict__ out, int out_stride,
                             int n_pages, const int32_t* __restrict__ tile_seq, const int32_t* __restrict__ tile_row0,
                             const int32_t* __restrict__ seq_start, const int32_t* __restrict__ seq_new,
                             const int32_t* __restrict__ cu_new, const int32_t* __restrict__ block_table, int bt_stride,
-                            int nkv, int group, float scale, int window, int keep_first, const float* __restrict__ sinks,
+                            int nkv, int group, float scale, int window, int keep_first, const float* __restrict__ sinks, const DlScoreCap cap,
                             int* __restrict__ status) {
     constexpr int ATOMS = HD / 64;                           // 64-dim (128-byte) slices of a head
     constexpr int STAGES = PT_STAGES(HD);
@@ -306,7 +307,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
         const bool stamps = (warp == 4 && lane == 0);
         const uint32_t lane_base = (uint32_t)(quarter * 32) << 16;
         const uint32_t my_s = tmem_s + lane_base + (uint32_t)(2 * t * DL_PAGE), my_o = tmem_o + lane_base + (uint32_t)(t * HD);
-        const float scale2 = scale * 1.4426950408889634f;    // scores in units of log2
+        const float scale2 = CAP ? 1.f : scale * 1.4426950408889634f;    // scores in units of log2 (capped ones come in them)
         float m_ref = -INFINITY, l = 0.f;                    // reference maximum (log2 units), sum of weights
         bool ok = true;
         const int n_mine = T.j_hi - T.j_lo + 1;
@@ -335,6 +336,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
             if (lane == 0) tc_mbar_arrive(&s_empty[t][sb]);     // the score buffer may take the tile's page after next
             if (stamps) PT_STAMP(7, j);                         // scores read into registers
 
+            if (CAP) {                                          // before the mask: a hidden key's score is replaced, not capped
+#pragma unroll
+                for (int i = 0; i < 64; ++i) sc[i] = dl_capped_score(sc[i], cap);
+            }
             const int key0 = page_of(j) * DL_PAGE;
             // pages wholly visible to every row of the tile need no mask
             const bool ragged = T.rows < PT_ROWS || key0 + DL_PAGE - 1 > T.pos0 || key0 < T.first_key ||
@@ -486,16 +491,17 @@ static int pt_tensor_map(CUtensorMap* out, const void* base, long long rows, lon
     return DL_OK;
 }
 
-template <int HD>
+template <int HD, bool CAP>
 static int pt_launch(dim3 grid, cudaStream_t s, const void* q, int q_stride, int n_tokens, void* out, int out_stride,
                      const void* k_pool, const void* v_pool, int n_pages, const int32_t* tile_seq, const int32_t* tile_row0,
                      const int32_t* seq_start, const int32_t* seq_new, const int32_t* cu_new, const int32_t* block_table,
-                     int bt_stride, int nh, int nkv, float scale, int window, int keep_first, const float* sinks, int* status) {
+                     int bt_stride, int nh, int nkv, float scale, int window, int keep_first, const float* sinks, float softcap,
+                     int* status) {
     const size_t smem = (size_t)PT_TILES * PT_ROWS * HD * 2 + (size_t)PT_STAGES(HD) * 2 * DL_PAGE * HD * 2 +
                         (size_t)PT_TILES * 2 * PT_ROWS * DL_PAGE * 2 + 1024;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<HD, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return dl_fail(DL_ERR_LAUNCH, "attention_prefill_tc: shared memory %zu: %s", smem, cudaGetErrorString(e));
         configured = true;
     }
@@ -506,9 +512,10 @@ static int pt_launch(dim3 grid, cudaStream_t s, const void* q, int q_stride, int
     if (rc != DL_OK) return rc;
     rc = pt_tensor_map(&tmap_v, v_pool, (long long)n_pages * nkv * HD, DL_PAGE, (long long)DL_PAGE * 2, HD);
     if (rc != DL_OK) return rc;
-    attention_prefill_tc_kernel<HD><<<grid, PT_THREADS, smem, s>>>(tmap_q, tmap_k, tmap_v, (__nv_bfloat16*)out, out_stride, n_pages,
+    attention_prefill_tc_kernel<HD, CAP><<<grid, PT_THREADS, smem, s>>>(tmap_q, tmap_k, tmap_v, (__nv_bfloat16*)out, out_stride, n_pages,
                                                                   tile_seq, tile_row0, seq_start, seq_new, cu_new, block_table,
-                                                                  bt_stride, nkv, nh / nkv, scale, window, keep_first, sinks, status);
+                                                                  bt_stride, nkv, nh / nkv, scale, window, keep_first, sinks,
+                                                                  dl_score_cap(softcap, scale), status);
     DL_CHECK_LAUNCH("attention_prefill_tc");
     return DL_OK;
 }
@@ -518,13 +525,14 @@ static int pt_launch(dim3 grid, cudaStream_t s, const void* q, int q_stride, int
 // that see the most keys first.  seq_start,
 // seq_new: cached length before the step and new tokens, per sequence; cu_new: packed offsets.
 // head_dim 64 or 128.  keep_first: with a window, that many first tokens of a sequence stay visible; sinks: float32 [nh]
-// or null, exp(sinks[h]) joins head h's sum of weights.  status: int32, set non-zero if a wait expired.
+// or null, exp(sinks[h]) joins head h's sum of weights; softcap: 0 for none, else scaled scores s become
+// softcap * tanh(s / softcap).  status: int32, set non-zero if a wait expired.
 extern "C" int dl_attention_prefill_tc_bf16(const void* q, int q_stride, int n_tokens, void* out, int out_stride,
                                             const void* k_pool, const void* v_pool, int n_pages, const int32_t* tile_seq,
                                             const int32_t* tile_row0, int n_tiles, const int32_t* seq_start,
                                             const int32_t* seq_new, const int32_t* cu_new, const int32_t* block_table,
                                             int bt_stride, int nh, int nkv, int hd, float scale, int window, int keep_first,
-                                            const float* sinks, int* status, void* stream) {
+                                            const float* sinks, float softcap, int* status, void* stream) {
     DL_REQUIRE(n_tiles >= 0 && n_tokens >= 0 && nh > 0 && nkv > 0 && nh % nkv == 0, "attention_prefill_tc: bad sizes");
     DL_REQUIRE(scale > 0.f && window >= 0, "attention_prefill_tc: the score scale must be positive, the window not negative");
     DL_REQUIRE(keep_first >= 0 && (keep_first == 0 || window > 0), "attention_prefill_tc: kept first tokens go with a window");
@@ -539,11 +547,12 @@ extern "C" int dl_attention_prefill_tc_bf16(const void* q, int q_stride, int n_t
     DL_REQUIRE(n_tiles <= 65535, "attention_prefill_tc: too many tiles (%d)", n_tiles);
     dim3 grid(nh, n_tiles);
     cudaStream_t s = (cudaStream_t)stream;
-    if (hd == 64)
-        return pt_launch<64>(grid, s, q, q_stride, n_tokens, out, out_stride, k_pool, v_pool, n_pages, tile_seq, tile_row0,
-                             seq_start, seq_new, cu_new, block_table, bt_stride, nh, nkv, scale, window, keep_first, sinks, status);
-    if (hd == 128)
-        return pt_launch<128>(grid, s, q, q_stride, n_tokens, out, out_stride, k_pool, v_pool, n_pages, tile_seq, tile_row0,
-                              seq_start, seq_new, cu_new, block_table, bt_stride, nh, nkv, scale, window, keep_first, sinks, status);
+#define PT_CASE(HDV, CAPV)                                                                                              \
+    if (hd == HDV && (softcap > 0.f) == CAPV)                                                                          \
+        return pt_launch<HDV, CAPV>(grid, s, q, q_stride, n_tokens, out, out_stride, k_pool, v_pool, n_pages, tile_seq, \
+                                    tile_row0, seq_start, seq_new, cu_new, block_table, bt_stride, nh, nkv, scale, window, \
+                                    keep_first, sinks, softcap, status);
+    PT_CASE(64, false) PT_CASE(128, false) PT_CASE(64, true) PT_CASE(128, true)
+#undef PT_CASE
     return dl_fail(DL_ERR_UNSUPPORTED, "attention_prefill_tc: head_dim %d (takes 64 and 128)", hd);
 }

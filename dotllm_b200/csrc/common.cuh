@@ -101,6 +101,23 @@ __device__ __forceinline__ float dl_warp_max(float v) {
     return v;
 }
 
+// c tanh(s / c) of a raw score s in units of log2: pre = 2 log2(e) scale / c turns the raw score into twice the argument (base
+// 2), post = c log2(e).  tanh(z) = 1 - 2 / (exp(2 z) + 1): exact at both ends, absolute error of some 1e-7 between.
+struct DlScoreCap {
+    float pre, post;             // post 0: no cap
+};
+static inline DlScoreCap dl_score_cap(float softcap, float scale) {
+    DlScoreCap c = {0.f, 0.f};
+    if (softcap > 0.f) c.pre = 2.f * 1.4426950408889634f * scale / softcap, c.post = softcap * 1.4426950408889634f;
+    return c;
+}
+__device__ __forceinline__ float dl_capped_score(float raw, DlScoreCap cap) {
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(raw * cap.pre));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(e + 1.f));
+    return fmaf(-2.f * cap.post, r, cap.post);
+}
+
 // Sum over a block of up to 1024 threads; every thread gets the result.  The order of
 // additions is fixed by the block size alone, so a row's result does not depend on
 // which other rows are in the launch.

@@ -161,9 +161,9 @@ __device__ __forceinline__ void gs_epilogue(const float (&acc_in)[NT][4], TOut* 
                 if (g == 0 && tok0 + e < M) fuse.sumsq_out[(size_t)tile * 16 + tok0 + e] = ss[e];
             }
         } else {
-            if (fuse.gate_kind == GATE_RELU2) {              // an activation of the one product: relu(y)^2
+            if (!dl_gate_is_gated(fuse.gate_kind)) {         // an activation of the one product
 #pragma unroll
-                for (int e = 0; e < 4; ++e) acc[e] = fmaxf(acc[e], 0.f) * fmaxf(acc[e], 0.f);
+                for (int e = 0; e < 4; ++e) acc[e] = dl_unary_value(fuse.gate_kind, acc[e]);
             }
             const int row_lo = tile * 16 + g, row_hi = row_lo + 8;
             if (row_lo < N) {

@@ -357,9 +357,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_constant
                             for (int i = 0; i < 32; ++i) v[i] = v[i] * (1.0f / (1.0f + expf(-v[i]))) * u[i];
                         }
                     }
-                    if (!GATED && grp.gate_kind == GATE_RELU2) {     // an activation of the one product: relu(v)^2
+                    if (!GATED && grp.gate_kind == GATE_RELU2) {     // an activation of the one product
 #pragma unroll
-                        for (int i = 0; i < 32; ++i) v[i] = fmaxf(v[i], 0.f) * fmaxf(v[i], 0.f);
+                        for (int i = 0; i < 32; ++i) v[i] = dl_unary_value(GATE_RELU2, v[i]);
+                    } else if (!GATED && grp.gate_kind == GATE_GELU) {
+#pragma unroll
+                        for (int i = 0; i < 32; ++i) v[i] = dl_unary_value(GATE_GELU, v[i]);
                     }
                     if (row < M && col_base + c0 < N) gt_store32<TOut>(row_ptr, col_base + c0, N, v, vec_ok != 0);
                 }

@@ -24,7 +24,14 @@ _library.register_signatures({
     "dl_gla_scan": [_P, _P, _P, _I, _P, _I, _P, _I, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _F, _F, _P],
     "dl_head_norm_gate": [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P],
     "dl_route_topk": [_P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _I, _F, _P],
-    "dl_head_rmsnorm": [_P, _I, _P, _I, _I, _P, _P, _I, _I, _I, _I, _F, _P],
+    "dl_head_rmsnorm": [_P, _I, _P, _I, _I, _P, _P, _I, _I, _I, _I, _I, _F, _P],
+    "dl_post_norm": [_P, _P, _I, _I, _F, _P, _I, _F, _P, _I, _F, _P, _I, _I, _I, _P, ctypes.c_long, _I, _P, _P, _I, _P],
+    "dl_causal_conv": [_P, _I, _I, _P, _I, _P, _I, _I, _P, ctypes.c_long, _I, _P, _P, _P, _I, _I, _I, _I, _I, _P],
+    "dl_ssd_scan": [_P, _I, _P, _I, _I, _P, _P, _P, _P, _P, _P, ctypes.c_long, _I, _P, _I, _I, _I, _I, _I, _I, _I, _P],
+    "dl_gated_group_norm": [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _F, _P],
+    "dl_latent_rows": [_P, _I, _I, _I, _I, _I, _I, _P, _P, _F, _P, _P, _I, _P, _P, _P, _I, _I, _P],
+    "dl_latent_query_tail": [_P, _I, _I, _I, _I, _I, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P],
+    "dl_channel_gate": [_P, _I, _I, _P, _I, _P, _I, _I, _I, _I, _I, _F, _P],
     "dl_delta_rule": [_P, _I, _P, _I, _I, _P, _I, _P, _I, _P, _P, _P, _P, _P, _P, _P, ctypes.c_long, _I,
                       _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _I, _P],
     "dl_expert_gate_up": [_P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _F, _P, _P],
@@ -203,7 +210,7 @@ def narrow_rows(value, ids):
     if isinstance(value, PendingProduct):
         x = resolve(value.x)
         return PendingProduct(gather_rows(x, ids, out_dtype=x.dtype), value.w, value.resident)
-    if isinstance(value, StreamWrite):
+    if isinstance(value, (StreamWrite, PostNormed)):
         return value.narrowed(ids)
     if isinstance(value, NormedBranch):
         return NormedBranch(narrow_rows(value.data, ids), value.gain, value.eps,
@@ -387,6 +394,86 @@ def scale_values(values, factor):
     return values
 
 
+class PostNormed:
+    """A sublayer's output that has not joined a post-norm stream yet: the stream x becomes u / sqrt(mean(u^2) + eps) * gain
+    with u = alpha x + data.  ``data`` [T, H] is a tensor or a product not yet launched, ``gain`` float32 [1] or [H]."""
+
+    def __init__(self, data, alpha, gain, eps):
+        self.data, self.alpha, self.gain, self.eps = data, float(alpha), gain, float(eps)
+        self.shape = tuple(data.shape)
+
+    def narrowed(self, ids):
+        return PostNormed(narrow_rows(self.data, ids), self.alpha, self.gain, self.eps)
+
+
+def post_norm(x, write, out_dtype=None, last=None, conv=None):
+    """The stream x (float32 [T, H] contiguous, updated in place) after ``write`` (a ``PostNormed``, or None: x stays as it is)
+    has joined it; returns a copy in ``out_dtype`` (None: no copy; float32: x itself, not copied, where nothing else is asked).
+    ``last`` (gain, eps): the copy is RMS-normalised once more (the model's last norm).  ``conv`` (taps float32 [K, H], memory
+    float32 [slots, >= (K - 1) H], slots int32 [T]): the copy is x plus a causal convolution of x over the row's own history,
+    which moves on - for steps of one token per sequence (``causal_conv`` takes any step)."""
+    y = gain = None
+    alpha, eps = 0.0, 0.0
+    if write is not None:
+        y, gain, alpha, eps = resolve(write.data), write.gain, write.alpha, write.eps
+    gain2, eps2 = last if last is not None else (None, 0.0)
+    taps, memory, slots = conv if conv is not None else (None, None, None)
+    _need_cuda(x, y, gain, gain2, taps, memory, slots)
+    if x.dtype != torch.float32 or x.dim() != 2 or not x.is_contiguous():
+        raise KernelError("post_norm: the stream must be contiguous float32 [T, H]")
+    T, H = x.shape
+    for g in (gain, gain2):
+        if g is not None and (g.dtype != torch.float32 or g.numel() not in (1, H) or not g.is_contiguous()):
+            raise KernelError(f"post_norm: a gain holds one float32 value or {H}")
+    if y is not None and tuple(y.shape) != (T, H):
+        raise KernelError(f"post_norm: a sublayer's output of shape {tuple(y.shape)} does not fit a stream of {(T, H)}")
+    K = 0
+    if conv is not None:
+        K = taps.shape[0]
+        if taps.dtype != torch.float32 or taps.shape != (K, H) or not taps.is_contiguous() or memory.dtype != torch.float32 \
+                or memory.dim() != 2 or memory.stride(1) != 1 or memory.shape[1] < (K - 1) * H or slots.numel() != T:
+            raise KernelError("post_norm: float32 taps [K, H], memory [slots, (K - 1) H] and one slot per row")
+        _int32(slots, "post_norm slots")
+    out = None
+    if out_dtype is not None:
+        if out_dtype == torch.float32 and last is None and conv is None:
+            if write is None:
+                return x
+        else:
+            out = torch.empty((T, H), dtype=out_dtype, device=x.device)
+    _library.call("dl_post_norm", _ptr(x), _ptr(y), _code(y.dtype) if y is not None else 0,
+                  _rows_view(y, "post_norm y") if y is not None else 0, alpha, _ptr(gain), gain.numel() if gain is not None else 1, eps,
+                  _ptr(gain2), gain2.numel() if gain2 is not None else 1, float(eps2), _ptr(out), _code(out_dtype) if out is not None else 0,
+                  T, H, _ptr(memory), memory.stride(0) if memory is not None else 0, memory.shape[0] if memory is not None else 0, _ptr(slots),
+                  _ptr(taps), K, _stream())
+    return x if out is None and out_dtype is not None else out
+
+
+def causal_conv(x, taps, memory, cu_new, slots, max_new, bias=None, activation=None, add_input=False, out_dtype=None):
+    """A causal convolution over time per channel of each sequence's new rows: y_t = act(bias + sum_j taps[j] x_(t-K+1+j)), plus
+    x_t with ``add_input``.  x [T, C] (a column view is fine); taps float32 [K, C], the last row meets the current token; memory
+    float32 [slots, >= (K - 1) C]: a sequence's last K - 1 inputs, read and moved on; ``activation`` None or "silu"; sums and
+    activation in float32.  ``max_new``: the most tokens a sequence brings.  Returns [T, C] in ``out_dtype`` (default float32)."""
+    _need_cuda(x, taps, memory, cu_new, slots, bias)
+    T, C = x.shape
+    K = taps.shape[0]
+    if activation not in (None, "silu"):
+        raise KernelError(f"causal_conv: unknown activation {activation!r}")
+    if taps.dtype != torch.float32 or taps.shape != (K, C) or not taps.is_contiguous():
+        raise KernelError(f"causal_conv: the taps must be contiguous float32 [K, {C}]")
+    if bias is not None and (bias.dtype != torch.float32 or bias.shape != (C,) or not bias.is_contiguous()):
+        raise KernelError(f"causal_conv: the bias must be float32 [{C}]")
+    if memory.dtype != torch.float32 or memory.dim() != 2 or memory.stride(1) != 1 or memory.shape[1] < (K - 1) * C:
+        raise KernelError("causal_conv: a slot's memory must hold the last K - 1 inputs in float32")
+    _int32(cu_new, "causal_conv cu_new")
+    _int32(slots, "causal_conv slots")
+    out = torch.empty((T, C), dtype=out_dtype or torch.float32, device=x.device)
+    _library.call("dl_causal_conv", _ptr(x), _code(x.dtype), _rows_view(x, "causal_conv x"), _ptr(taps), K, _ptr(bias),
+                  1 if activation == "silu" else 0, 1 if add_input else 0, _ptr(memory), memory.stride(0), memory.shape[0], _ptr(cu_new),
+                  _ptr(slots), _ptr(out), _code(out.dtype), out.stride(0), slots.numel(), int(max_new), C, _stream())
+    return out
+
+
 def _add_product_scaled(residual, product, gain, eps, out_dtype):
     x = product.x
     rows = x.row_sums() if isinstance(x, ScaledRows) else None
@@ -479,8 +566,7 @@ def head_gate(o, gate, n_heads, width):
 class ScoreHook:
     """A change of the attention scores before the softmax: ``softcap`` > 0 turns a score s into
     softcap * tanh(s / softcap); ``slopes`` (float32 [n_heads] on the device) then adds
-    slope * (key position - query position).  Only the generic kernel honours a hook: the
-    tensor-core kernels take none, so a mixer that sets one runs on the generic kernel."""
+    slope * (key position - query position).  The tensor-core kernels take the cap; slopes send a mixer to the generic kernel."""
 
     def __init__(self, softcap=0.0, slopes=None):
         self.softcap = float(softcap)
@@ -499,8 +585,8 @@ def attention(q, k_pool, v_pool, token_seq, token_pos, block_table, n_heads, n_k
     q [T, nh*hd] (row-contiguous view); returns [T, nh*vd] of q's dtype (vd = ``value_dim``, default hd).
     ``window`` 0 means every earlier key; w > 0 means the last w keys.  ``plan`` carries the per-step layout
     (sequence lengths, chunking) that the tensor-core kernels need; without one, for sizes
-    they do not take (values of another width than the keys among them), or with a ``score_hook``, the generic
-    kernel runs.  ``gate`` [T, nh] of q's dtype (a column view is fine): head h's output is multiplied by
+    they do not take (values of another width than the keys among them), or with a ``score_hook`` that has slopes, the
+    generic kernel runs.  ``gate`` [T, nh] of q's dtype (a column view is fine): head h's output is multiplied by
     sigmoid(gate[t, h]) - in the generic kernel's last step, or by ``head_gate`` behind a tensor-core kernel.
     ``keep_first`` n > 0 (with a window): a sequence's first n keys stay visible when the window has passed them.
     ``sinks`` float32 [nh]: head h's softmax has one more term exp(sinks[h]) in its denominator, with no key and no value."""
@@ -532,10 +618,10 @@ def attention(q, k_pool, v_pool, token_seq, token_pos, block_table, n_heads, n_k
         if slopes is not None and (slopes.dtype != torch.float32 or slopes.shape != (n_heads,) or not slopes.is_contiguous()
                                    or not slopes.is_cuda):
             raise KernelError(f"attention: a score hook's slopes must be contiguous float32 [{n_heads}] on the device")
-    if plan is not None and q.dtype == torch.bfloat16 and not score_hook and vd == head_dim:
+    if plan is not None and q.dtype == torch.bfloat16 and slopes is None and vd == head_dim:
         if attention_fast.run(q, qs, out, k_pool, v_pool, n_pages, token_seq, token_pos, block_table,
                               n_heads, n_kv_heads, head_dim, float(scale), int(window), plan,
-                              keep_first=int(keep_first), sinks=sinks):
+                              keep_first=int(keep_first), sinks=sinks, softcap=softcap):
             return out if gate is None else head_gate(out, gate, n_heads, vd)
     _library.call("dl_attention_generic", _ptr(q), qs, _ptr(out), out.stride(0), _code(q.dtype),
                   _ptr(k_pool), _ptr(v_pool), n_pages, _ptr(token_seq), _ptr(token_pos),
@@ -551,10 +637,11 @@ def rope_cache_attention(q, k, v, cos, sin, rotary_dim, token_seq, token_pos, bl
     decode step (one new token per sequence) with a full-width rotation of head size 64 or 128, or
     with no rotation, runs as one kernel that adds the biases, rotates q, puts the new keys and values into the
     cache, attends and gates the heads; everything else runs the kernels one after the other."""
-    if plan is not None and q.is_cuda and q.dtype == torch.bfloat16 and not score_hook and (value_dim or head_dim) == head_dim \
-            and (k is not None or biases is not None or gate is not None) and not keep_first and sinks is None:
+    if plan is not None and q.is_cuda and q.dtype == torch.bfloat16 and (not score_hook or score_hook.slopes is None) \
+            and (value_dim or head_dim) == head_dim and (k is not None or biases is not None or gate is not None) and not keep_first:
         out = attention_fast.decode_fresh(q, k, v, cos, sin, rotary_dim, block_table, k_pool, v_pool, n_heads,
-                                          n_kv_heads, head_dim, float(scale), int(window), plan, biases=biases, gate=gate)
+                                          n_kv_heads, head_dim, float(scale), int(window), plan, biases=biases, gate=gate, sinks=sinks,
+                                          softcap=score_hook.softcap if score_hook else 0.0)
         if out is not None:
             return out
     rope_cache_write(q, k, v, cos, sin, rotary_dim, token_seq, token_pos, block_table, k_pool, v_pool,
@@ -601,8 +688,8 @@ def swiglu(gate_up):
     return out
 
 
-GATINGS = {"silu": 0, "gelu_tanh": 1, "clamped_sigmoid": 2, "relu2": 3}
-UNGATED = frozenset({"relu2"})      # activations of ONE product, act(u): no gate rows in the matrix (GATE_RELU2 in csrc/gating.cuh)
+GATINGS = {"silu": 0, "gelu_tanh": 1, "clamped_sigmoid": 2, "relu2": 3, "gelu": 4}
+UNGATED = frozenset({"relu2", "gelu"})      # activations of ONE product, act(u): no gate rows in the matrix ("gelu": the exact, erf form)
 
 
 def gated_activation(gate_up, kind, limit=0.0, alpha=1.0):
@@ -674,20 +761,132 @@ def head_norm_gate(o, g, gain, n_heads, vdim, eps, out_dtype, gate="silu"):
     return out
 
 
-def head_rmsnorm(x, gain_a, heads_a, dim, eps, gain_b=None, heads_b=0):
+def head_rmsnorm(x, gain_a, heads_a, dim, eps, gain_b=None, heads_b=0, lay=None):
     """Every head of a row normalised on its own: y[t, h, :] = x[t, h, :] / sqrt(mean(x[t, h, :]^2) + eps) * gain[:].  The
     row holds ``heads_a`` heads under ``gain_a`` and behind them ``heads_b`` heads under ``gain_b`` (queries and keys of
-    one stacked projection), each ``dim`` wide; x may be a column view.  Returns a new tensor of x's dtype."""
+    one stacked projection), each ``dim`` wide; x may be a column view.  Returns a new tensor of x's dtype whose heads are
+    ``lay`` (default ``dim``) wide, zeros behind their values."""
     _need_cuda(x, gain_a, gain_b)
+    lay = int(lay or dim)
     T, width = x.shape[0], (heads_a + heads_b) * dim
     if x.dim() != 2 or x.shape[1] != width:
         raise KernelError(f"head_rmsnorm: x must be [T, {width}]")
     for g, n in ((gain_a, heads_a), (gain_b, heads_b)):
         if n and (g is None or g.dtype != torch.float32 or g.shape != (dim,) or not g.is_contiguous()):
             raise KernelError(f"head_rmsnorm: a gain must be contiguous float32 [{dim}]")
-    out = torch.empty((T, width), dtype=x.dtype, device=x.device)
+    out = torch.empty((T, (heads_a + heads_b) * lay), dtype=x.dtype, device=x.device)
     _library.call("dl_head_rmsnorm", _ptr(x), _rows_view(x, "head_rmsnorm x"), _ptr(out), out.stride(0), _code(x.dtype),
-                  _ptr(gain_a), _ptr(gain_b), T, int(heads_a), int(heads_b), int(dim), float(eps), _stream())
+                  _ptr(gain_a), _ptr(gain_b), T, int(heads_a), int(heads_b), int(dim), lay, float(eps), _stream())
+    return out
+
+
+# --------------------------------------------------- state-space recurrence
+def ssd_scan(xbc, z, dt_bias, a_log, skip, cu_new, slots, memory, n_heads, groups, state, vdim):
+    """The recurrence S <- exp(-exp(a_log_h) dt) S + dt B x^T, y = S^T C + skip_h x with dt = softplus(z + dt_bias_h), over each
+    sequence's new rows in order.  xbc float32 [T, H*vdim + 2*groups*state]: x, then B, then C (head h uses group
+    h // (H/groups)); z [T, H] (a column view is fine); dt_bias, a_log, skip float32 [H]; memory float32 [slots, >=
+    H*state*vdim]: per slot every head's [state, vdim], read and updated.  Returns y float32 [T, H*vdim]."""
+    _need_cuda(xbc, z, dt_bias, a_log, skip, cu_new, slots, memory)
+    T, H, G, N, P = xbc.shape[0], int(n_heads), int(groups), int(state), int(vdim)
+    if xbc.dtype != torch.float32 or xbc.shape[1] != H * P + 2 * G * N or z.shape != (T, H):
+        raise KernelError(f"ssd_scan: float32 rows of {H * P + 2 * G * N} values and one step logit per head")
+    for t, what in ((dt_bias, "dt_bias"), (a_log, "a_log"), (skip, "skip")):
+        if t.dtype != torch.float32 or t.shape != (H,) or not t.is_contiguous():
+            raise KernelError(f"ssd_scan: {what} must be contiguous float32 [{H}]")
+    if memory.dtype != torch.float32 or memory.dim() != 2 or memory.stride(1) != 1 or memory.shape[1] < H * N * P:
+        raise KernelError(f"ssd_scan: a slot's memory must hold {H * N * P} float32 values")
+    _int32(cu_new, "ssd_scan cu_new")
+    _int32(slots, "ssd_scan slots")
+    out = torch.empty((T, H * P), dtype=torch.float32, device=xbc.device)
+    _library.call("dl_ssd_scan", _ptr(xbc), _rows_view(xbc, "ssd_scan xbc"), _ptr(z), _code(z.dtype), _rows_view(z, "ssd_scan z"),
+                  _ptr(dt_bias), _ptr(a_log), _ptr(skip), _ptr(cu_new), _ptr(slots), _ptr(memory), memory.stride(0), memory.shape[0],
+                  _ptr(out), out.stride(0), slots.numel(), T, H, G, N, P, _stream())
+    return out
+
+
+def _out_view(out, rows, width, dtype, device, what):
+    """``out`` (a [rows, width] view with contiguous rows) after checking it, or a new tensor."""
+    if out is None:
+        return torch.empty((rows, width), dtype=dtype, device=device)
+    if out.shape != (rows, width) or out.dtype != dtype:
+        raise KernelError(f"{what}: the output must be a {dtype} view [{rows}, {width}]")
+    return out
+
+
+def gated_group_norm(y, gate, gain, parts, eps, scale=1.0, out=None):
+    """v = y silu(gate); v divided by its root mean square over each of ``parts`` equal parts of the row, times gain and
+    ``scale``.  y float32 [T, W]; gate [T, W] of the step's dtype (a column view is fine); gain float32 [W].  Returns [T, W] in
+    the gate's dtype (``out``: a view to write instead)."""
+    _need_cuda(y, gate, gain, out)
+    T, W = y.shape
+    if y.dtype != torch.float32 or gate.shape != (T, W) or gain.dtype != torch.float32 or gain.shape != (W,) or W % parts:
+        raise KernelError(f"gated_group_norm: y float32 [T, W], a gate of its shape, gains [W], W a multiple of {parts} parts")
+    out = _out_view(out, T, W, gate.dtype, y.device, "gated_group_norm")
+    _library.call("dl_gated_group_norm", _ptr(y), _rows_view(y, "gated_group_norm y"), _ptr(gate), _rows_view(gate, "gated_group_norm gate"),
+                  _ptr(gain), _ptr(out), _rows_view(out, "gated_group_norm out"), _code(gate.dtype), T, W, int(parts), float(eps),
+                  float(scale), _stream())
+    return out
+
+
+# ------------------------------------------------------------ latent attention
+def _pair_tables(tables, what):
+    """(cos, sin, rotated channels, rows) of an interleaved rotation's tables, or of none."""
+    if tables is None:
+        return None, None, 0, 0
+    cos, sin = tables
+    if cos.dtype != torch.float32 or sin.dtype != torch.float32 or cos.shape != sin.shape or cos.dim() != 2 or not cos.is_contiguous() \
+            or not sin.is_contiguous():
+        raise KernelError(f"{what}: cos and sin must be contiguous float32 [positions, pairs]")
+    return cos, sin, 2 * cos.shape[1], cos.shape[0]
+
+
+def latent_rows(x, q_gain, kv_gain, eps, rot, tables, token_pos, lay):
+    """x [T, q_rank + kv_rank + rot] (a column view is fine) -> (query latent [T, q_rank] or None, cache rows [T, lay]): both
+    latents RMS-normalised with their gains (``q_gain`` None: no query latent), the last ``rot`` channels rotated by the token's
+    position (pairs 2i, 2i + 1 of as many channels as ``tables`` = (cos, sin) [positions, pairs] give) and put behind the second
+    latent, zeros behind them up to ``lay``."""
+    _need_cuda(x, q_gain, kv_gain, token_pos)
+    T, r = x.shape[0], kv_gain.numel()
+    rq = q_gain.numel() if q_gain is not None else 0
+    cos, sin, dims, rows = _pair_tables(tables, "latent_rows")
+    if x.shape[1] != rq + r + rot or dims > rot or lay < r + rot:
+        raise KernelError(f"latent_rows: rows of {rq} + {r} + {rot} channels into {lay}, {dims} of them rotated")
+    _int32(token_pos, "latent_rows positions")
+    cq = torch.empty((T, rq), dtype=x.dtype, device=x.device) if rq else None
+    kv = torch.empty((T, lay), dtype=x.dtype, device=x.device)
+    _library.call("dl_latent_rows", _ptr(x), _code(x.dtype), _rows_view(x, "latent_rows x"), rq, r, int(rot), dims, _ptr(q_gain), _ptr(kv_gain),
+                  float(eps), _ptr(cos), _ptr(sin), rows, _ptr(token_pos), _ptr(cq), _ptr(kv), int(lay), T, _stream())
+    return cq, kv
+
+
+def latent_queries(q, w_key, rot, tables, token_pos, lay):
+    """q [T, H*(dim + rot)] head by head -> [T, H*lay]: per head W_key[h] q[:dim] (w_key [H, rank, dim]), then the last ``rot``
+    channels rotated as in ``latent_rows``, then zeros."""
+    _need_cuda(q, w_key, token_pos)
+    H, r, d = w_key.shape
+    T = q.shape[0]
+    cos, sin, dims, rows = _pair_tables(tables, "latent_queries")
+    if q.shape[1] != H * (d + rot) or dims > rot or lay < r + rot:
+        raise KernelError(f"latent_queries: {H} heads of {d} + {rot} channels into {lay}")
+    _int32(token_pos, "latent_queries positions")
+    out = torch.empty((T, H * lay), dtype=q.dtype, device=q.device)
+    linear_per_head(q, w_key, x_head=d + rot, out=out, out_head=lay)
+    _library.call("dl_latent_query_tail", _ptr(q), _code(q.dtype), _rows_view(q, "latent_queries q"), d, int(rot), dims, _ptr(cos), _ptr(sin),
+                  rows, _ptr(token_pos), _ptr(out), out.stride(0), r, int(lay), H, T, _stream())
+    return out
+
+
+def channel_gate(o, gate, heads, width, lay=None, scale=1.0, out=None):
+    """out[t, h, c] = scale * o[t, h, c] * sigmoid(gate[t, h, c]) for o with its heads ``lay`` (default ``width``) apart and gate
+    [T, heads*width] (column views are fine; None: no gate, the scale alone).  Returns [T, heads*width] of o's dtype (``out``: a view to write instead)."""
+    _need_cuda(o, gate, out)
+    T, lay = o.shape[0], int(lay or width)
+    if o.shape[1] < (heads - 1) * lay + width or (gate is not None and (gate.shape != (T, heads * width) or gate.dtype != o.dtype)):
+        raise KernelError(f"channel_gate: o with {heads} heads {lay} apart and one gate logit per channel of o's dtype")
+    out = _out_view(out, T, heads * width, o.dtype, o.device, "channel_gate")
+    _library.call("dl_channel_gate", _ptr(o), _rows_view(o, "channel_gate o"), lay, _ptr(gate),
+                  _rows_view(gate, "channel_gate gate") if gate is not None else heads * width, _ptr(out),
+                  _rows_view(out, "channel_gate out"), _code(o.dtype), T, int(heads), int(width), float(scale), _stream())
     return out
 
 
@@ -909,25 +1108,33 @@ def experts_grouped(x, ids, weights, w_gate_up, w_down, kind, limit=0.0, alpha=1
 
 
 # --------------------------------------------------------------------- linear
-def linear_per_head(x, w):
+def linear_per_head(x, w, x_head=None, out=None, out_head=None):
     """y[t, h, :] = W[h] x[t, h, :] for x [T, H*a] (rows contiguous) and W [H, b, a]; returns [T, H*b] in x's dtype.
-    bfloat16: one batched library product with float32 accumulation; float32: the FFMA product head by head."""
-    _need_cuda(x, w)
-    if w.dim() != 3 or not w.is_contiguous() or x.dim() != 2 or x.shape[1] != w.shape[0] * w.shape[2] or x.dtype != w.dtype:
-        raise KernelError(f"linear_per_head: x {tuple(x.shape)} does not match W {tuple(w.shape)}")
+    bfloat16: one batched library product with float32 accumulation; float32: the FFMA product head by head.  ``x_head``: the
+    heads' distance in x (default a; the first a channels of each are read).  ``out`` (contiguous) and ``out_head``: heads that
+    distance apart are written into it, what lies between them stays as it is."""
+    _need_cuda(x, w, out)
     H, b, a = w.shape
+    xh, oh = int(x_head or a), int(out_head or b)
+    if w.dim() != 3 or not w.is_contiguous() or x.dim() != 2 or x.shape[1] != H * xh or xh < a or oh < b or x.dtype != w.dtype:
+        raise KernelError(f"linear_per_head: x {tuple(x.shape)} does not match W {tuple(w.shape)}")
     T = x.shape[0]
     xs = _rows_view(x, "linear_per_head x")
-    y = torch.empty((T, H * b), dtype=x.dtype, device=x.device)
+    if out is None:
+        y = torch.empty((T, H * oh), dtype=x.dtype, device=x.device)
+    else:
+        y = out
+        if y.shape != (T, H * oh) or y.dtype != x.dtype or not y.is_contiguous():
+            raise KernelError("linear_per_head: out must be contiguous [T, H*out_head] of x's dtype")
     if T == 0:
         return y
     if x.dtype == torch.float32:
         for h in range(H):
-            _library.call("dl_gemm_f32", x.data_ptr() + 4 * h * a, xs, w[h].data_ptr(), y.data_ptr() + 4 * h * b, H * b,
+            _library.call("dl_gemm_f32", x.data_ptr() + 4 * h * xh, xs, w[h].data_ptr(), y.data_ptr() + 4 * h * oh, H * oh,
                           T, b, a, _stream())
         return y
-    xv = x.as_strided((H, T, a), (a, xs, 1))
-    torch.bmm(xv, w.transpose(1, 2), out=y.view(T, H, b).transpose(0, 1))
+    xv = x.as_strided((H, T, a), (xh, xs, 1), x.storage_offset())
+    torch.bmm(xv, w.transpose(1, 2), out=y.as_strided((H, T, b), (oh, H * oh, 1), y.storage_offset()))
     return y
 
 

@@ -17,8 +17,9 @@ value projection); an RMS norm of every query and key head before the rotation, 
 the keys (``qk_norm``), or an RMS norm over the whole query projection and over the whole key projection, all heads at once,
 with a gain per channel (``qk_norm`` with ``over`` "projection"); a window that keeps a sequence's first tokens visible
 (``keep_first``); a learned number per head in the softmax's denominator, a sink without key or value (``sink``), or a sink
-of score zero without a tensor (``sink`` "zero": one is added to the denominator); and a rotation that pairs channel 2i
-with 2i + 1 (``pairing`` "interleaved").
+of score zero without a tensor (``sink`` "zero": one is added to the denominator); a rotation that pairs channel 2i
+with 2i + 1 (``pairing`` "interleaved"); and a gate per output channel (``gate`` "channel_sigmoid": the concatenated heads
+times sigmoid of a projection of the mixer's input as wide as they are, behind the attention).
 
 Interleaved pairs on kernels that pair channel i with i + r/2.  Scores do not change when the channels of q and k are
 permuted alike, so for a rotation of the first r channels in interleaved pairs the rows of the q and k projections (and
@@ -54,7 +55,7 @@ import torch
 from ..config.spec import PartSpec
 from ..errors import ConfigError
 from ..kernels import ops
-from .base import CacheNeed, Mixer, WeightSpec, make_part, register_mixer
+from .base import CacheNeed, Mixer, WeightSpec, make_part, pad_rows, register_mixer
 
 # Branch outputs are handed to the residual add in float32.
 BRANCH_DTYPE = torch.float32
@@ -65,7 +66,7 @@ class AttentionMixer(Mixer):
     ``position`` ({"kind", "params"} of a position encoding), optional ``scale``, optional ``score``
     ({"softcap": c, "slopes": [one per head]}: scores are capped and biased by distance before the
     softmax, which sends the mixer to the generic attention kernel); optional ``value_dim`` (per head, default
-    ``head_dim``), ``bias`` (True: q, k and v have biases), ``gate`` (None or "head_sigmoid"), ``own_kv`` (False: no key
+    ``head_dim``), ``bias`` (True: q, k and v have biases), ``gate`` (None, "head_sigmoid" or "channel_sigmoid"), ``own_kv`` (False: no key
     and value projections, the layer reads another's cache) and ``tensors``: the local names of ``q``, ``k``, ``v``,
     ``o``, ``gate`` and the bias suffix ``bias`` (appended to a projection's name); optional ``values`` ("own", or "keys":
     v is k as projected, there is no value projection and ``value_dim`` is ``head_dim``), ``qk_norm`` ({"eps"}: tensors
@@ -78,7 +79,8 @@ class AttentionMixer(Mixer):
     NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
              "gate": "g_proj.weight", "q_bias": "q_proj.bias", "k_bias": "k_proj.bias", "v_bias": "v_proj.bias",
              "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "sink": "sinks"}
-    GATES = (None, "head_sigmoid")
+    GATES = (None, "head_sigmoid", "channel_sigmoid")
+    stacks = True
     ROW_STEP = 16                # the stacked matrix's rows are a multiple of this: its product's rows stay 16-byte aligned
 
     def __init__(self, params, hidden_size, runtime):
@@ -104,6 +106,7 @@ class AttentionMixer(Mixer):
         self.value_dim = int(params.get("value_dim") or self.head_dim)
         self.bias = bool(params.get("bias", False))
         self.gate = params.get("gate")
+        self.channel_gate = self.gate == "channel_sigmoid"
         if self.gate not in self.GATES:
             raise ConfigError(f"attention: unknown gate {self.gate!r}; known: {list(self.GATES)}")
         self.own_kv = bool(params.get("own_kv", True))
@@ -135,11 +138,16 @@ class AttentionMixer(Mixer):
         self.plain = not self.bias and self.gate is None and self.value_dim == self.head_dim and self.own_kv \
             and self.values == "own" and self.qk_norm_eps is None and not self.sink and not self.keep_first \
             and params.get("pairing", "half") == "half"
-        # heads keep their own width and channel order where a norm runs over them or the keys double as values
-        as_stored = self.values == "keys" or self.qk_norm_eps is not None or params.get("pairing") == "interleaved"
         self.w_qkv = None
         self.w_o = None
         self.biases = None
+        fused = self.position.fused_rotary()         # (cos, sin, r)
+        rd = int(fused[2]) if fused is not None else 0
+        # a norm per head writes its result wherever the kernels want it: queries and keys that no rotation follows may be
+        # projected at their stored width and laid out by the norm
+        self.norm_lays = self.qk_norm_over == "head" and fused is not None and rd == 0 and self.values == "own"
+        # heads keep their own width and channel order where a norm runs over them or the keys double as values
+        as_stored = self.values == "keys" or (self.qk_norm_eps is not None and not self.norm_lays) or params.get("pairing") == "interleaved"
         # the width every head is laid out at (see the module's text); head_dim / value_dim stay the stored widths
         self.lay_k, self.lay_v = self.head_dim, self.value_dim
         if runtime.dtype == torch.bfloat16 and not self.plain and not as_stored and \
@@ -147,9 +155,7 @@ class AttentionMixer(Mixer):
             fits = [w for w in self.TENSOR_CORE_WIDTHS if w >= max(self.head_dim, self.value_dim)]
             if fits and self.n_heads // self.n_kv_heads <= 16:
                 self.lay_k = self.lay_v = fits[0]
-        # a partial rotation spread over the whole head (see the module's text): fused_rotary() gives (cos, sin, r)
-        fused = self.position.fused_rotary()
-        rd = int(fused[2]) if fused is not None else 0
+        # a partial rotation spread over the whole head (see the module's text)
         self.spread = bool(runtime.dtype == torch.bfloat16 and not self.plain and not as_stored and self.lay_k == self.lay_v
                            and self.lay_k in self.TENSOR_CORE_WIDTHS and 0 < rd < self.lay_k)
         self.rotation = None if fused is None else (self._wide_tables(fused[0], fused[1], rd, self.lay_k) + (self.lay_k,)
@@ -217,7 +223,7 @@ class AttentionMixer(Mixer):
                 specs[n["k_bias"]] = WeightSpec((self.kv_dim,), "precise", ("normal", 0.1))
                 specs[n["v_bias"]] = WeightSpec((self.v_width,), "precise", ("normal", 0.1))
         if self.gate:
-            specs[n["gate"]] = WeightSpec((self.n_heads, h), init=("normal", 0.1))
+            specs[n["gate"]] = WeightSpec((self.o_dim if self.channel_gate else self.n_heads, h), init=("normal", 0.1))
         if self.qk_norm_eps is not None:
             whole = self.qk_norm_over == "projection"
             specs[n["q_norm"]] = WeightSpec((self.q_dim if whole else self.head_dim,), "precise", ("one_plus_uniform", 0.1))
@@ -231,20 +237,17 @@ class AttentionMixer(Mixer):
     def bind(self, tensors):
         n = self.names
         H, G, hd, vd, lk, lv = self.n_heads, self.n_kv_heads, self.head_dim, self.value_dim, self.lay_k, self.lay_v
-        rows = [self._reorder(self._widen(tensors[n["q"]], H, hd, lk), H)]
+        pk = hd if self.norm_lays else lk                  # the width q and k leave the product at
+        rows = [self._reorder(self._widen(tensors[n["q"]], H, hd, pk), H)]
         if self.own_kv:
-            rows.append(self._reorder(self._widen(tensors[n["k"]], G, hd, lk), G))
+            rows.append(self._reorder(self._widen(tensors[n["k"]], G, hd, pk), G))
             if self.values == "own":
                 rows.append(self._widen(tensors[n["v"]], G, vd, lv))
         if self.gate:
             rows.append(tensors[n["gate"]])
-        if not self.plain:
-            total = sum(r.shape[0] for r in rows)
-            pad = -total % self.ROW_STEP
-            if pad:
-                rows.append(torch.zeros((pad, self.hidden_size), dtype=rows[0].dtype, device=rows[0].device))
-        self.w_qkv = torch.cat(rows, dim=0).contiguous()
-        self.w_o = self._widen(tensors[n["o"]], H, vd, lv, dim=1).contiguous()
+        self.w_qkv = torch.cat(rows, dim=0).contiguous() if self.plain else pad_rows(rows, self.ROW_STEP)
+        # (the gate per channel, and the sum of mixers, take the heads back to their stored width)
+        self.w_o = (tensors[n["o"]] if self.channel_gate or self.compact else self._widen(tensors[n["o"]], H, vd, lv, dim=1)).contiguous()
         if self.qk_norm_eps is not None and self.qk_norm_over == "projection":
             # one gain per channel of the projection: they follow their channels into the kernels' order
             self.q_gain = self._reorder(tensors[n["q_norm"]], H).contiguous()
@@ -273,6 +276,25 @@ class AttentionMixer(Mixer):
 
     takes_scaled_rows = True                    # x goes straight into the Q/K/V product
 
+    # As one side of a sum of mixers (``Mixer.stacks``): the stacked matrix under the interface's name.
+    compact = False                             # True: w_o takes the heads at their stored width whatever the gate
+
+    @property
+    def w_in(self):
+        return self.w_qkv
+
+    @w_in.setter
+    def w_in(self, value):
+        self.w_qkv = value
+
+    @property
+    def out_width(self):
+        return self.o_dim
+
+    def heads(self, proj, step, cache_view, scale=1.0, out=None):
+        a, g = self._attend(proj, step, cache_view)
+        return ops.channel_gate(a, g, self.n_heads, self.value_dim, lay=self.lay_v, scale=scale, out=out)
+
     def _forward_general(self, x, step, cache_view):
         """With biases, a gate, values of their own width or another layer's cache: one stacked product (q, then k and v
         where the layer has its own, then the gate's logits), one kernel that adds the biases, rotates and writes the
@@ -280,9 +302,18 @@ class AttentionMixer(Mixer):
         if cache_view.writes != self.own_kv:
             raise ConfigError("attention: a layer without key and value projections must read another layer's cache "
                               "(and one with them keeps its own)")
-        lk, lv = self.lay_k, self.lay_v
-        qd, kvd, vw = self.n_heads * lk, self.n_kv_heads * lk, self.n_kv_heads * lv
         y = ops.linear(x, self.w_qkv, resident=True)
+        if self.channel_gate:
+            a = self.heads(y, step, cache_view)
+        else:
+            a, _ = self._attend(y, step, cache_view)
+        return ops.linear(a, self.w_o, out_dtype=BRANCH_DTYPE, resident=True, lazy=True)
+
+    def _attend(self, y, step, cache_view):
+        """From the stacked product to the heads' outputs [T, n_heads * lay_v] and the logits of a gate per channel (or None)."""
+        lk, lv = self.lay_k, self.lay_v
+        pk = self.head_dim if self.norm_lays else lk
+        qd, kvd, vw = self.n_heads * pk, self.n_kv_heads * pk, self.n_kv_heads * lv
         q, at = y[:, :qd], qd
         k = v = None
         if self.own_kv and self.values == "keys":
@@ -290,7 +321,8 @@ class AttentionMixer(Mixer):
             v = k                                   # as projected: the norm below writes its result elsewhere
         elif self.own_kv:
             k, v, at = y[:, at:at + kvd], y[:, at + kvd:at + kvd + vw], at + kvd + vw
-        g = y[:, at:at + self.n_heads] if self.gate else None
+        g = y[:, at:at + self.n_heads] if self.gate == "head_sigmoid" else None
+        channel_g = y[:, at:at + self.o_dim] if self.channel_gate else None
         if self.qk_norm_eps is not None and self.qk_norm_over == "projection":
             if self.own_kv:
                 normed = ops.group_rmsnorm(y[:, :qd + kvd], self.qk_gain, qd, kvd, self.qk_norm_eps)
@@ -299,10 +331,10 @@ class AttentionMixer(Mixer):
                 q = ops.group_rmsnorm(q, self.qk_gain, qd, 0, self.qk_norm_eps)
         elif self.qk_norm_eps is not None:
             if self.own_kv:
-                normed = ops.head_rmsnorm(y[:, :qd + kvd], self.q_gain, self.n_heads, lk, self.qk_norm_eps, self.k_gain, self.n_kv_heads)
-                q, k = normed[:, :qd], normed[:, qd:]
+                normed = ops.head_rmsnorm(y[:, :qd + kvd], self.q_gain, self.n_heads, pk, self.qk_norm_eps, self.k_gain, self.n_kv_heads, lay=lk)
+                q, k = normed[:, :self.n_heads * lk], normed[:, self.n_heads * lk:]
             else:
-                q = ops.head_rmsnorm(q, self.q_gain, self.n_heads, lk, self.qk_norm_eps)
+                q = ops.head_rmsnorm(q, self.q_gain, self.n_heads, pk, self.qk_norm_eps, lay=lk)
         fused = self.rotation
         if fused is None:
             if self.biases is not None:
@@ -318,7 +350,7 @@ class AttentionMixer(Mixer):
                                      int(self.window or 0), plan=step.attention_plan,
                                      score_hook=self.score_hook if self.score_hook else None,
                                      value_dim=lv, biases=self.biases, gate=g, keep_first=self.keep_first, sinks=self.sinks)
-        return ops.linear(a, self.w_o, out_dtype=BRANCH_DTYPE, resident=True, lazy=True)
+        return a, channel_g
 
     def forward(self, x, step, cache_view):
         if not self.plain:

@@ -14,6 +14,7 @@ Kinds are registered by name:
     register_position_encoding("rotary", RotaryEncoding)
     register_arrangement("pre_norm", PreNormBlock)
     register_connection("stream_copies", StreamConnection)
+    register_mixer_input("causal_convolution", InputConvolution)
 
 and a ``PartSpec(kind, params, prefix)`` picks one per layer.
 """
@@ -138,6 +139,15 @@ class Norm(Part):
         raise NotImplementedError
 
 
+def pad_rows(rows, step=16):
+    """Matrices of one width stacked into one, with rows of zeros up to a multiple of ``step``: the rows of the stacked product
+    then stay 16-byte aligned."""
+    pad = -sum(r.shape[0] for r in rows) % step
+    if pad:
+        rows = list(rows) + [torch.zeros((pad, rows[0].shape[1]), dtype=rows[0].dtype, device=rows[0].device)]
+    return torch.cat(list(rows), dim=0).contiguous()
+
+
 def normalised_for(consumer, norm, residual, pending):
     """The stream, with the branch output ``pending`` (or None) added, normalised by ``norm`` for the
     part ``consumer``.  A part may return its last product unlaunched (``ops.linear(..., lazy=True)``);
@@ -183,6 +193,27 @@ class Mixer(Part):
 
         ``step`` is the engine's StepContext (token -> sequence map, positions, lengths);
         ``cache_view`` gives this execution's storage (``LayerCacheView``) or None."""
+        raise NotImplementedError
+
+    # A mixer that ``stacks`` is [one matrix of projections] -> heads -> [one output matrix], so that several mixers that read the
+    # same input can share the two products (``parts.paired``).  After ``bind``: ``w_in`` [rows, H], ``w_o`` [H, ``out_width``].
+    stacks = False
+
+    def heads(self, proj, step, cache_view, scale=1.0, out=None):
+        """What ``w_o`` is applied to, times ``scale``: [T, out_width] in the run dtype, from ``proj`` = x w_in^T (a column view of a
+        wider product is fine), written into ``out`` where given."""
+        raise NotImplementedError
+
+
+class MixerInput(Part):
+    """What a mixer reads, made from the stream: the stream as it is, or the stream mixed with its own past."""
+
+    def cache_need(self) -> Optional[CacheNeed]:
+        return None
+
+    def read(self, stream, pending, step, cache_view):
+        """Apply ``pending`` (an ``ops.PostNormed``, or None) to the float32 ``stream`` in place, then return the mixer's input
+        in the run dtype."""
         raise NotImplementedError
 
 
@@ -242,7 +273,7 @@ class Arrangement:
 
 
 _REGISTRIES = {"mixer": {}, "feed_forward": {}, "norm": {}, "position_encoding": {}, "arrangement": {},
-               "embedding": {}, "head": {}, "connection": {}}
+               "embedding": {}, "head": {}, "connection": {}, "mixer_input": {}}
 
 
 def _register(family, kind, cls):
@@ -274,6 +305,10 @@ def register_connection(kind, cls):
     return _register("connection", kind, cls)
 
 
+def register_mixer_input(kind, cls):
+    return _register("mixer_input", kind, cls)
+
+
 def register_embedding(kind, cls):
     return _register("embedding", kind, cls)
 
@@ -289,7 +324,7 @@ def registered(family):
 
 def _ensure_builtin():
     from . import (norms, rotary, attention, feed_forward, blocks, embedding, linear_attention,  # noqa: F401
-                   latent_attention, experts, delta_rule, connections, paired)
+                   latent_attention, experts, delta_rule, connections, paired, state_space, input_convolution)
 
 
 def make_part(family, spec, hidden_size, runtime):

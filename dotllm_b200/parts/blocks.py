@@ -97,7 +97,39 @@ class ConnectedBlock(Arrangement):
         return residual, self.feed_forward_connection.write(self.feed_forward.forward(n))
 
 
+class PostNormBlock(Arrangement):
+    """Sublayers that read the stream itself, with the norm behind the sum: x = norm1(a x + mixer(x)); x = norm2(a x + ff(x)).  The
+    norms (``parts.norms.PostRmsNorm``) own the factor a.  A ``mixer_input`` may stand before the mixer (``parts.input_convolution``);
+    what it keeps is part of the layer's cache, in front of the mixer's needs.  The feed-forward with its norm may be absent."""
+    needs = ("mixer", "mixer_norm")
+    narrows = True
+
+    def cache_need(self):
+        need = self.mixer.cache_need()
+        if "mixer_input" not in self.parts:
+            return need
+        return (self.mixer_input.cache_need(), *(need if isinstance(need, tuple) else (need,)))
+
+    def forward(self, residual, pending, step, cache_view, keep_rows=None):
+        from ..kernels import ops
+        if "mixer_input" in self.parts:
+            mixer_view = cache_view[1:] if isinstance(self.mixer.cache_need(), tuple) else cache_view[1]
+            h = self.mixer_input.read(residual, pending, step, cache_view[0])
+        else:
+            mixer_view = cache_view
+            h = ops.post_norm(residual, pending, self.mixer.runtime.dtype)
+        branch = self.mixer_norm.branch(self.mixer.forward(h, step, mixer_view))     # every token: the cache needs them all
+        if keep_rows is not None:
+            residual = ops.gather_rows(residual, keep_rows)
+            branch = ops.narrow_rows(branch, keep_rows)
+        if "feed_forward" not in self.parts:
+            return residual, branch
+        x = ops.post_norm(residual, branch, self.feed_forward.runtime.dtype)
+        return residual, self.feed_forward_norm.branch(self.feed_forward.forward(x))
+
+
 register_arrangement("pre_norm", PreNormBlock)
+register_arrangement("post_norm", PostNormBlock)
 register_arrangement("connected", ConnectedBlock)
 register_arrangement("parallel", ParallelBlock)
 register_arrangement("sandwich_norm", SandwichNormBlock)

@@ -1,4 +1,4 @@
-"""Dense gated feed-forward (SwiGLU): down(silu(gate(x)) * up(x)).
+"""Dense feed-forwards: gated (SwiGLU), down(silu(gate(x)) * up(x)), and plain, down(act(up(x))).
 
 src/DotLLM.Models/Architectures/TransformerModel.cs:342-382 with the activation of
 src/DotLLM.Cpu/Kernels/FusedOps.cs:33-78.  Gate and up are stacked into one matrix when the
@@ -24,8 +24,8 @@ class GatedFeedForward(FeedForward):
         super().__init__(params, hidden_size, runtime)
         self.intermediate_size = int(params["intermediate_size"])
         self.activation = params.get("activation", "silu")
-        if self.activation not in ops.GATINGS:
-            raise ConfigError(f"gated feed-forward: unsupported activation {self.activation!r}; known: {sorted(ops.GATINGS)}")
+        if self.activation not in ops.GATINGS or self.activation in ops.UNGATED:
+            raise ConfigError(f"gated feed-forward: unsupported activation {self.activation!r}; known: {sorted(set(ops.GATINGS) - ops.UNGATED)}")
         self.limit = float(params.get("limit", 0.0))
         self.alpha = float(params.get("alpha", 1.0))
         names = params.get("tensors") or ("gate_proj.weight", "up_proj.weight", "down_proj.weight")
@@ -52,4 +52,36 @@ class GatedFeedForward(FeedForward):
         return ops.linear(gated, self.w_down, out_dtype=BRANCH_DTYPE, resident=True, lazy=True)
 
 
+class PlainFeedForward(FeedForward):
+    """A dense feed-forward without a gate: down(act(up(x))), the activation in the first product's epilogue where it has one.
+
+    params: ``intermediate_size``; ``activation`` (one of ``ops.UNGATED``: "gelu", the exact form, or "relu2"); optional
+    ``tensors``: the local names of the up and down matrices."""
+
+    def __init__(self, params, hidden_size, runtime):
+        super().__init__(params, hidden_size, runtime)
+        self.intermediate_size = int(params["intermediate_size"])
+        self.activation = params["activation"]
+        if self.activation not in ops.UNGATED:
+            raise ConfigError(f"feed-forward: unsupported activation {self.activation!r}; known: {sorted(ops.UNGATED)}")
+        self.up_name, self.down_name = (str(n) for n in params.get("tensors") or ("up_proj.weight", "down_proj.weight"))
+        self.w_up = self.w_down = None
+
+    def weight_specs(self):
+        i, h = self.intermediate_size, self.hidden_size
+        return {self.up_name: WeightSpec((i, h)), self.down_name: WeightSpec((h, i))}
+
+    def bind(self, tensors):
+        self.w_up = tensors[self.up_name].contiguous()
+        self.w_down = tensors[self.down_name].contiguous()
+
+    def weight_bytes(self):
+        return (self.w_up.numel() + self.w_down.numel()) * self.w_down.element_size()
+
+    def forward(self, x):
+        u = ops.activated_linear(x, self.w_up, self.activation, resident=True)
+        return ops.linear(u, self.w_down, out_dtype=BRANCH_DTYPE, resident=True, lazy=True)
+
+
 register_feed_forward("gated_mlp", GatedFeedForward)
+register_feed_forward("plain_mlp", PlainFeedForward)

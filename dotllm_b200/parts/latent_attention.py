@@ -11,6 +11,17 @@ is therefore attention of H query heads of width r against ONE shared key/value 
 the paged cache of the layer holds c (as keys and, transposed, as values) and the library's own
 attention kernels (prefill on tcgen05, decode over pages, windows, page recycling) serve it unchanged.
 The two per-head changes of basis are batched products around the attention.
+
+A part of the keys may carry positions (``rot_dim`` R, ``position``): the queries then hold R more channels per head, one more
+projection of x gives R channels that all heads share as keys, and both are rotated (channel 2i with 2i + 1):
+
+    score = (q_h . k_h + rot(q'_h) . rot(k')) * scale
+
+The cached row is [c | rot(k')] (width r + R), the query against it [Wuk_h^T q_h | rot(q'_h)].  Options that go with it, each a
+parameter: a learned sink per head in the softmax's denominator (``sink``) and a gate per output channel (``gate``
+"channel_sigmoid").  In this form every projection of x - query latent, key/value latent with the shared key part, gate - is a row of
+one stacked matrix.  In a bfloat16 run whose r + R fits a width of the tensor-core attention kernels the row is laid out at that
+width, zeros behind it, and serves as key and value alike: the value's channels beyond r are read by nobody.
 """
 from __future__ import annotations
 
@@ -18,20 +29,24 @@ import math
 
 import torch
 
+from ..config.spec import PartSpec
 from ..errors import ConfigError
 from ..kernels import ops
-from .attention import BRANCH_DTYPE
-from .base import CacheNeed, Mixer, WeightSpec, register_mixer
+from .attention import BRANCH_DTYPE, AttentionMixer
+from .base import CacheNeed, Mixer, WeightSpec, make_part, pad_rows, register_mixer
 
 
 class LatentAttentionMixer(Mixer):
     """params: ``n_heads``, ``key_dim``, ``value_dim`` (per head), ``q_rank`` (None: queries without a latent), ``kv_rank`` (the latents),
     ``eps`` (of the latents' norms), optional ``scale`` (default key_dim^-1/2), ``window`` (None: every
-    earlier key; w: a query sees itself and the w - 1 tokens before it), ``tensors`` (local names)."""
+    earlier key; w: a query sees itself and the w - 1 tokens before it), ``tensors`` (local names); optional ``rot_dim`` with
+    ``position`` ({"kind": "rotary", "params"}), ``sink`` (True: tensor ``sink`` [n_heads]) and ``gate`` (None or "channel_sigmoid":
+    tensor ``gate`` [n_heads * value_dim, H])."""
 
     NAMES = {"q_down": "q_a_proj.weight", "q_norm": "q_a_norm.weight", "q_up": "q_b_proj.weight",
              "kv_down": "kv_a_proj.weight", "kv_norm": "kv_a_norm.weight", "k_up": "k_b_proj.weight",
-             "v_up": "v_b_proj.weight", "out": "o_proj.weight", "q": "q_proj.weight"}
+             "v_up": "v_b_proj.weight", "out": "o_proj.weight", "q": "q_proj.weight", "gate": "g_proj.weight", "sink": "sinks"}
+    GATES = (None, "channel_sigmoid")
 
     def __init__(self, params, hidden_size, runtime):
         super().__init__(params, hidden_size, runtime)
@@ -50,18 +65,45 @@ class LatentAttentionMixer(Mixer):
         if self.window is not None and self.window < 1:
             raise ConfigError("latent attention: a window holds at least the token itself")
         self.names = dict(self.NAMES, **(params.get("tensors") or {}))
+        self.rot_dim = int(params.get("rot_dim") or 0)
+        self.sink = bool(params.get("sink", False))
+        self.gate = params.get("gate")
+        if self.gate not in self.GATES or self.rot_dim < 0:
+            raise ConfigError(f"latent attention: unknown gate {self.gate!r} or a negative rotated width")
+        position = params.get("position")
+        self.position = make_part("position_encoding", PartSpec(position["kind"], position.get("params", {})), hidden_size, runtime) \
+            if position else None
+        self.tables = None
+        if self.position is not None:
+            fused = self.position.fused_rotary()
+            if fused is None or int(fused[2]) > self.rot_dim:
+                raise ConfigError("latent attention: positions are a rotation of at most the shared key part's channels")
+            self.tables = (fused[0], fused[1]) if fused[2] else None
+        self.stacked = bool(self.rot_dim or self.sink or self.gate)
+        # what the cache keeps of a token, and the width of the attention's keys and values
+        self.row = self.kv_rank + self.rot_dim
+        self.key_width, self.value_width = self.row, self.kv_rank
+        if self.stacked and runtime.dtype == torch.bfloat16:
+            fits = [w for w in AttentionMixer.TENSOR_CORE_WIDTHS if w >= self.row]
+            if fits:
+                self.key_width = self.value_width = fits[0]
+        self.w_in = self.w_gate = self.sinks = None
         self.w_dq = self.w_dkv = self.q_gain = self.kv_gain = self.w_uq = self.w_uk_t = self.w_uv = self.w_o = None
 
     def weight_specs(self):
         h, n, H = self.hidden_size, self.names, self.n_heads
         if self.q_rank is None:
-            queries = {n["q"]: WeightSpec((H * self.key_dim, h))}
+            queries = {n["q"]: WeightSpec((H * (self.key_dim + self.rot_dim), h))}
         else:
             queries = {n["q_down"]: WeightSpec((self.q_rank, h)),
                        n["q_norm"]: WeightSpec((self.q_rank,), "precise", ("one_plus_uniform", 0.1)),
-                       n["q_up"]: WeightSpec((H * self.key_dim, self.q_rank), init=("normal", 0.1))}
+                       n["q_up"]: WeightSpec((H * (self.key_dim + self.rot_dim), self.q_rank), init=("normal", 0.1))}
+        if self.sink:
+            queries[n["sink"]] = WeightSpec((H,), "precise", ("normal", 1.0))
+        if self.gate:
+            queries[n["gate"]] = WeightSpec((H * self.value_dim, h), init=("normal", 0.1))
         return {**queries,
-                n["kv_down"]: WeightSpec((self.kv_rank, h)),
+                n["kv_down"]: WeightSpec((self.row, h)),
                 n["kv_norm"]: WeightSpec((self.kv_rank,), "precise", ("one_plus_uniform", 0.1)),
                 n["k_up"]: WeightSpec((H * self.key_dim, self.kv_rank), init=("normal", 0.1)),
                 n["v_up"]: WeightSpec((H * self.value_dim, self.kv_rank), init=("normal", 0.1)),
@@ -81,16 +123,45 @@ class LatentAttentionMixer(Mixer):
         self.w_uk_t = tensors[n["k_up"]].view(H, self.key_dim, self.kv_rank).transpose(1, 2).contiguous()
         self.w_uv = tensors[n["v_up"]].view(H, self.value_dim, self.kv_rank).contiguous()
         self.w_o = tensors[n["out"]].contiguous()
+        self.sinks = tensors[n["sink"]].contiguous() if self.sink else None
+        if self.stacked:
+            rows = [m for m in (self.w_dq, self.w_dkv) if m is not None]
+            self.gate_at = -(-sum(m.shape[0] for m in rows) // 8) * 8             # the gate's columns start 16-byte aligned
+            self.w_in = pad_rows([pad_rows(rows, 8)] + ([tensors[n["gate"]]] if self.gate else []))
+            self.w_dq = self.w_dkv = None
 
     def weight_bytes(self):
-        mats = (self.w_dq, self.w_dkv, self.w_uq, self.w_uk_t, self.w_uv, self.w_o)
+        mats = (self.w_in, self.w_dq, self.w_dkv, self.w_uq, self.w_uk_t, self.w_uv, self.w_o)
         return sum(m.numel() for m in mats if m is not None) * self.w_o.element_size()
 
     def cache_need(self):
         # one shared head whose keys and values are both the latent
-        return CacheNeed("kv", n_kv_heads=1, head_dim=self.kv_rank, window=self.window)
+        return CacheNeed("kv", n_kv_heads=1, head_dim=self.key_width, window=self.window,
+                         v_dim=self.value_width if self.value_width != self.key_width else None)
+
+    def _forward_stacked(self, x, step, cache_view):
+        """One product of x, both latents' norms with the rotated key part in one kernel, the queries changed to the latent's basis,
+        attention over the cached rows, back to the values' basis, the gate, the output product."""
+        x = ops.resolve(x)
+        H, r, rq = self.n_heads, self.kv_rank, self.q_rank or 0
+        proj = ops.linear(x, self.w_in, resident=True)
+        cq, rows = ops.latent_rows(proj[:, :rq + self.row], self.q_gain if self.q_rank is not None else None, self.kv_gain, self.eps,
+                                   self.rot_dim, self.tables, step.token_pos, self.key_width)
+        q = ops.linear(cq if cq is not None else x, self.w_uq, resident=True)
+        q = ops.latent_queries(q, self.w_uk_t, self.rot_dim, self.tables, step.token_pos, self.key_width)
+        keys, values = (rows, rows[:, :self.value_width]) if cache_view.writes else (None, None)
+        a = ops.rope_cache_attention(q, keys, values, None, None, 0, step.token_seq, step.token_pos, cache_view.block_table,
+                                     cache_view.k, cache_view.v, H, 1, self.key_width, self.scale, int(self.window or 0),
+                                     plan=step.attention_plan, value_dim=self.value_width, sinks=self.sinks)
+        o = ops.linear_per_head(a, self.w_uv, x_head=self.value_width)                             # [T, H*dv]
+        if self.gate:
+            g = proj[:, self.gate_at:self.gate_at + H * self.value_dim]
+            o = ops.channel_gate(o, g, H, self.value_dim, out=o)
+        return ops.linear(o, self.w_o, out_dtype=BRANCH_DTYPE, resident=True, lazy=True)
 
     def forward(self, x, step, cache_view):
+        if self.stacked:
+            return self._forward_stacked(x, step, cache_view)
         dtype = self.runtime.dtype
         if self.q_rank is None:
             cq = x

@@ -96,5 +96,46 @@ class StreamNorm(Norm):
         return self.read_stream(residual, self.copies, delta, None)
 
 
+class PostRmsNorm(Norm):
+    """An RMS norm behind the sum: x <- u / sqrt(mean(u^2) + eps) * gain with u = alpha x + y, in place, float32.  A sublayer's output
+    y is handed on unadded (``branch`` -> ``ops.PostNormed``), and whoever reads the stream next applies it (``ops.post_norm``: a
+    feed-forward's copy, a mixer's input convolution, the model's last norm ride that kernel).  Without a sum (``forward``: the
+    model's last norm) it is the plain RMS norm.
+
+    params: ``eps``; ``alpha`` (default 1: the plain sum); ``gain`` "channel", or "scalar": one number for all channels (a tensor
+    without dimensions); optional ``tensor``: the gain's local name (default "weight"; "" when the prefix is the whole name)."""
+
+    def __init__(self, params, hidden_size, runtime):
+        super().__init__(params, hidden_size, runtime)
+        self.eps = float(params["eps"])
+        self.alpha = float(params.get("alpha", 1.0))
+        self.scalar = params.get("gain", "channel") == "scalar"
+        if params.get("gain", "channel") not in ("channel", "scalar"):
+            raise ConfigError("post-norm: a gain per 'channel' or a 'scalar' one")
+        self.tensor_name = str(params.get("tensor", "weight"))
+        self.gain = None
+
+    def weight_specs(self):
+        return {self.tensor_name: WeightSpec(() if self.scalar else (self.hidden_size,), "precise", ("one_plus_uniform", 0.1))}
+
+    def bind(self, tensors):
+        self.gain = tensors[self.tensor_name].reshape(-1).contiguous()
+
+    def weight_bytes(self):
+        return self.gain.numel() * self.gain.element_size()
+
+    def branch(self, data):
+        return ops.PostNormed(data, self.alpha, self.gain, self.eps)
+
+    def forward(self, x):
+        return ops.post_norm(x, None, self.runtime.dtype, last=(self.gain, self.eps))
+
+    def add_forward(self, residual, delta):
+        if not isinstance(delta, ops.PostNormed):
+            raise ConfigError("post-norm: what joins the stream must carry the norm behind its sum")
+        return ops.post_norm(residual, delta, self.runtime.dtype, last=(self.gain, self.eps))
+
+
+register_norm("post_rmsnorm", PostRmsNorm)
 register_norm("rmsnorm", RmsNorm)
 register_norm("stream_norm", StreamNorm)

@@ -9,10 +9,13 @@ pair of views.  The two norms and the sum are one kernel in float32.
 """
 from __future__ import annotations
 
+import torch
+
 from ..config.spec import PartSpec
 from ..errors import ConfigError
 from ..kernels import ops
-from .base import Mixer, WeightSpec, make_part, register_mixer
+from .attention import BRANCH_DTYPE
+from .base import Mixer, WeightSpec, make_part, pad_rows, register_mixer
 
 
 class PairedMixer(Mixer):
@@ -65,4 +68,66 @@ class PairedMixer(Mixer):
         return ops.pair_norm_sum(left, right, self.gains[0], self.gains[1], self.eps, self.weights[0], self.weights[1])
 
 
+class SummedMixer(Mixer):
+    """A weighted sum of mixers side by side without norms: y = w_l left(x) + w_r right(x).  Both sides ``stack`` (``Mixer.heads``), so
+    their projections are one product of the shared input, each side scales what it hands to its output matrix by its weight (in
+    float32, where it writes it), and one product with the two output matrices side by side is the sum.
+
+    params: ``left`` and ``right`` ({"kind", "params", "prefix"}), ``weights`` (one per side)."""
+
+    def __init__(self, params, hidden_size, runtime):
+        super().__init__(params, hidden_size, runtime)
+        self.weights = tuple(float(w) for w in params["weights"])
+        if len(self.weights) != 2:
+            raise ConfigError("summed mixer: one weight per side")
+        self.sides = []
+        for side in ("left", "right"):
+            d = params[side]
+            mixer = make_part("mixer", PartSpec(d["kind"], d.get("params", {})), hidden_size, runtime)
+            if not mixer.stacks:
+                raise ConfigError(f"summed mixer: a mixer of kind {d['kind']!r} does not share its products")
+            mixer.compact = True
+            self.sides.append((str(d.get("prefix", side + ".")), mixer))
+        self.graph_safe = all(getattr(m, "graph_safe", True) for _, m in self.sides)
+        self.w_in = self.w_o = None
+        self.at = ()                       # where each side's columns start: (in the stacked projection, in the stacked heads)
+
+    def weight_specs(self):
+        return {prefix + local: spec for prefix, mixer in self.sides for local, spec in mixer.weight_specs().items()}
+
+    def optional_names(self):
+        return {prefix + local for prefix, mixer in self.sides for local in mixer.optional_names()}
+
+    def bind(self, tensors):
+        for prefix, mixer in self.sides:
+            mixer.bind({local: tensors[prefix + local] for local in mixer.weight_specs()})
+        left, right = (m for _, m in self.sides)
+        self.at = ((0, 0), (left.w_in.shape[0], left.out_width))
+        self.w_in = pad_rows([left.w_in, right.w_in])
+        outs = [left.w_o, right.w_o]
+        pad = -(left.out_width + right.out_width) % 8                   # the products like whole eights of columns
+        if pad:
+            outs.append(torch.zeros((self.hidden_size, pad), dtype=left.w_o.dtype, device=left.w_o.device))
+        self.w_o = torch.cat(outs, dim=1).contiguous()
+        self.widths = tuple((m.w_in.shape[0], m.out_width) for _, m in self.sides)
+        self.padded = bool(pad)
+        left.w_in = right.w_in = left.w_o = right.w_o = None            # the stacked ones serve
+
+    def weight_bytes(self):
+        return (self.w_in.numel() + self.w_o.numel()) * self.w_in.element_size()
+
+    def cache_need(self):
+        return tuple(m.cache_need() for _, m in self.sides)
+
+    def forward(self, x, step, cache_view):
+        x = ops.resolve(x)
+        proj = ops.linear(x, self.w_in, resident=True)
+        make = torch.zeros if self.padded else torch.empty
+        y = make((x.shape[0], self.w_o.shape[1]), dtype=self.runtime.dtype, device=x.device)
+        for (_, mixer), weight, (p0, y0), (pn, yn), view in zip(self.sides, self.weights, self.at, self.widths, cache_view):
+            mixer.heads(proj[:, p0:p0 + pn], step, view, scale=weight, out=y[:, y0:y0 + yn])
+        return ops.linear(y, self.w_o, out_dtype=BRANCH_DTYPE, resident=True, lazy=True)
+
+
 register_mixer("paired", PairedMixer)
+register_mixer("summed", SummedMixer)

@@ -95,11 +95,12 @@ def head_norm_gate(o, g, gain, n_heads, vdim, eps, out_dtype, gate="silu"):
     return (y * act).reshape(T, n_heads * vdim).to(out_dtype)
 
 
-def head_rmsnorm(x, gain_a, heads_a, dim, eps, gain_b=None, heads_b=0):
+def head_rmsnorm(x, gain_a, heads_a, dim, eps, gain_b=None, heads_b=0, lay=None):
     T = x.shape[0]
     xf = x.to(torch.float32).reshape(T, heads_a + heads_b, dim)
     y = _rms(xf, eps)
     y = torch.cat([y[:, :heads_a] * gain_a] + ([y[:, heads_a:] * gain_b] if heads_b else []), dim=1)
+    y = torch.nn.functional.pad(y, (0, (lay or dim) - dim))
     return y.reshape(T, -1).to(x.dtype)
 
 
@@ -188,12 +189,117 @@ def scale_values(values, factor):
 
 
 def unary_activation(x, kind):
+    xf = x.to(torch.float32)
+    if kind == "gelu":
+        return (0.5 * xf * (1.0 + torch.erf(xf / 2.0 ** 0.5))).to(x.dtype)
     assert kind == "relu2"
-    return (torch.relu(x.to(torch.float32)) ** 2).to(x.dtype)
+    return (torch.relu(xf) ** 2).to(x.dtype)
 
 
 def activated_linear(x, w, kind, resident=False):
     return unary_activation(linear(x, w, torch.float32), kind).to(x.dtype)
+
+
+class PostNormed:
+    def __init__(self, data, alpha, gain, eps):
+        self.data, self.alpha, self.gain, self.eps = data, float(alpha), gain, float(eps)
+        self.shape = tuple(data.shape)
+
+    def narrowed(self, ids):
+        return PostNormed(self.data[ids.long()], self.alpha, self.gain, self.eps)
+
+
+def post_norm(x, write, out_dtype=None, last=None, conv=None):
+    if write is not None:
+        x.copy_(_rms(write.alpha * x + write.data.to(torch.float32), write.eps) * write.gain)
+    if last is not None:
+        return (_rms(x, last[1]) * last[0]).to(out_dtype)
+    if conv is not None:                                    # every row is the only new one of its sequence
+        taps, memory, slots = conv
+        cu = torch.arange(x.shape[0] + 1, dtype=torch.int32)
+        return causal_conv(x, taps, memory, cu, slots, 1, add_input=True, out_dtype=out_dtype)
+    return None if out_dtype is None else x if out_dtype == torch.float32 else x.to(out_dtype)
+
+
+def causal_conv(x, taps, memory, cu_new, slots, max_new, bias=None, activation=None, add_input=False, out_dtype=None):
+    T, C = x.shape
+    K = taps.shape[0]
+    out = torch.zeros((T, C), dtype=torch.float32)
+    for b in range(slots.numel()):
+        hist = memory[int(slots[b]), :(K - 1) * C].view(K - 1, C)
+        t0, t1 = int(cu_new[b]), int(cu_new[b + 1])
+        inputs = torch.cat([hist, x[t0:t1].to(torch.float32)], dim=0)
+        for j in range(t1 - t0):
+            y = (taps * inputs[j:j + K]).sum(0) + (bias if bias is not None else 0.0)
+            if activation == "silu":
+                y = y * torch.sigmoid(y)
+            out[t0 + j] = y + (inputs[j + K - 1] if add_input else 0.0)
+        if K > 1:
+            hist.copy_(inputs[inputs.shape[0] - (K - 1):].clone())
+    return out.to(out_dtype or torch.float32)
+
+
+def ssd_scan(xbc, z, dt_bias, a_log, skip, cu_new, slots, memory, n_heads, groups, state, vdim):
+    T, H, G, N, P = xbc.shape[0], n_heads, groups, state, vdim
+    x = xbc[:, :H * P].reshape(T, H, P)
+    B = xbc[:, H * P:H * P + G * N].reshape(T, G, N).repeat_interleave(H // G, dim=1)
+    C = xbc[:, H * P + G * N:].reshape(T, G, N).repeat_interleave(H // G, dim=1)
+    dt = torch.nn.functional.softplus(z.to(torch.float32) + dt_bias)
+    out = torch.zeros((T, H, P), dtype=torch.float32)
+    for b in range(slots.numel()):
+        S = memory[int(slots[b]), :H * N * P].view(H, N, P)
+        for t in range(int(cu_new[b]), int(cu_new[b + 1])):
+            S.mul_(torch.exp(-torch.exp(a_log) * dt[t])[:, None, None]).add_(dt[t][:, None, None] * B[t][:, :, None] * x[t][:, None, :])
+            out[t] = torch.einsum("hnp,hn->hp", S, C[t]) + skip[:, None] * x[t]
+    return out.reshape(T, H * P)
+
+
+def _into(out, value, dtype):
+    if out is None:
+        return value.to(dtype)
+    out.copy_(value.to(dtype))
+    return out
+
+
+def gated_group_norm(y, gate, gain, parts, eps, scale=1.0, out=None):
+    g = gate.to(torch.float32)
+    v = (y * g * torch.sigmoid(g)).reshape(y.shape[0], parts, -1)
+    return _into(out, _rms(v, eps).reshape(y.shape) * gain * scale, gate.dtype)
+
+
+def _rotated_pairs(x, tables, pos):
+    """x [T, ..., d]: channels 2i and 2i + 1 turned by the tables' angle of the row's position."""
+    if tables is None:
+        return x
+    cos, sin = (t[pos.long()].reshape(x.shape[0], *([1] * (x.dim() - 2)), -1) for t in tables)
+    dims = 2 * cos.shape[-1]
+    out = x.clone()
+    a, b = x[..., 0:dims:2], x[..., 1:dims:2]
+    out[..., 0:dims:2], out[..., 1:dims:2] = a * cos - b * sin, b * cos + a * sin
+    return out
+
+
+def latent_rows(x, q_gain, kv_gain, eps, rot, tables, token_pos, lay):
+    xf, rq, r = x.to(torch.float32), q_gain.numel() if q_gain is not None else 0, kv_gain.numel()
+    cq = (_rms(xf[:, :rq], eps) * q_gain).to(x.dtype) if rq else None
+    row = torch.cat([_rms(xf[:, rq:rq + r], eps) * kv_gain, _rotated_pairs(xf[:, rq + r:], tables, token_pos)], dim=1)
+    return cq, torch.nn.functional.pad(row, (0, lay - r - rot)).to(x.dtype)
+
+
+def latent_queries(q, w_key, rot, tables, token_pos, lay):
+    H, r, d = w_key.shape
+    qf = q.to(torch.float32).reshape(q.shape[0], H, d + rot)
+    head = torch.einsum("thd,hrd->thr", qf[..., :d], w_key.to(torch.float32))
+    y = torch.cat([head, _rotated_pairs(qf[..., d:], tables, token_pos)], dim=-1)
+    return torch.nn.functional.pad(y, (0, lay - r - rot)).reshape(q.shape[0], H * lay).to(q.dtype)
+
+
+def channel_gate(o, gate, heads, width, lay=None, scale=1.0, out=None):
+    lay = lay or width
+    y = torch.nn.functional.pad(o.to(torch.float32), (0, heads * lay - o.shape[1])).reshape(o.shape[0], heads, lay)[..., :width].reshape(o.shape[0], -1)
+    if gate is not None:
+        y = y * torch.sigmoid(gate.to(torch.float32))
+    return _into(out, y * scale, o.dtype)
 
 
 def softcap(values, cap):
@@ -272,11 +378,14 @@ def expert_down(h, ids, weights, w_down, addend=None, addend_gate=None, identity
     return out + (addend if addend_gate is None else addend * torch.sigmoid(addend_gate[:, :1]))
 
 
-def linear_per_head(x, w):
+def linear_per_head(x, w, x_head=None, out=None, out_head=None):
     H, b, a = w.shape
     T = x.shape[0]
-    y = torch.einsum("tha,hba->thb", x.to(torch.float32).reshape(T, H, a), w.to(torch.float32))
-    return y.reshape(T, H * b).to(x.dtype)
+    y = torch.einsum("tha,hba->thb", x.to(torch.float32).reshape(T, H, x_head or a)[..., :a], w.to(torch.float32)).to(x.dtype)
+    if out is None:
+        return torch.nn.functional.pad(y, (0, (out_head or b) - b)).reshape(T, -1)
+    out.view(T, H, out_head or b)[..., :b] = y
+    return out
 
 
 def _rotate(x, cos, sin, positions, n_heads, head_dim, rotary_dim):
