@@ -9,6 +9,7 @@
     python bench.py --workload komulorn [--shape 1b]  # the Komulorn design beside a Llama of equal width, heads and depth, and its kernels
     python bench.py --workload zemezen [--shape 1b]   # the Zemezen design beside a Kubedra of equal width and depth, and its kernels
     python bench.py --workload sopalorn [--shape 1b]  # the Sopalorn design beside a Zemezen of equal width and depth, and its kernels
+    python bench.py --workload semanex [--shape 1b]   # the Semanex design beside a Sopalorn and a Zemezen of equal width and depth, and its kernels
     python bench.py --impl plain-cpu                  # the plain implementation under tests/, timed on the CPU
 
 A "step" is one decode step: one new token for each of ``batch`` sequences that already hold
@@ -130,7 +131,7 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference", "plain-cpu"])
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"])
     ap.add_argument("--repeats", type=int, default=5, help="repetitions of every timed region (best and CV are reported)")
-    ap.add_argument("--workload", default="steady", choices=["steady", "unequal", "staggered", "short-prompts", "kubedra", "komulorn", "zemezen", "sopalorn"],
+    ap.add_argument("--workload", default="steady", choices=["steady", "unequal", "staggered", "short-prompts", "kubedra", "komulorn", "zemezen", "sopalorn", "semanex"],
                     help="unequal: 64 prompts of 16..2048 tokens in one prefill step, then 256 decode steps; "
                          "staggered: Model.generate on 64 prompts whose requests end five steps apart; "
                          "short-prompts: the time to the first token of single prompts of 20 to 1,024 tokens; "
@@ -138,7 +139,8 @@ def main():
                          "equal width and depth, and each of its kernels against its roofline; "
                          "komulorn: the same for the Komulorn design beside a Llama of equal width, heads and depth; "
                          "zemezen: the same for the Zemezen design beside a Kubedra of equal width and depth; "
-                         "sopalorn: the same for the Sopalorn design beside a Zemezen of equal width and depth")
+                         "sopalorn: the same for the Sopalorn design beside a Zemezen of equal width and depth; "
+                         "semanex: the same for the Semanex design beside a Sopalorn and a Zemezen")
     ap.add_argument("--no-generate", action="store_true", help="skip the Model.generate cells")
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--context", type=int, default=8192)
@@ -176,6 +178,8 @@ def main():
         return zemezen_workload(args)
     if args.workload == "sopalorn":
         return sopalorn_workload(args)
+    if args.workload == "semanex":
+        return semanex_workload(args)
     pk = peaks()
     shape_name, shape = SHAPES[args.shape]
     cfg_dict = dict(shape, num_hidden_layers=args.layers or shape["num_hidden_layers"])
@@ -1066,6 +1070,205 @@ def sopalorn_workload(args):
                       "n_gpus": 1, "steps": args.steps, "warmup": max(3, args.warmup), "higher_is_better": True, "dtype": "bf16",
                       "data": "synthetic", "vs_baseline": None, "clocks": sampler.stop(),
                       "config": {"model": "Sopalorn, four layers at the sizes named", "batch": 8, "context": ctx, "prefill_tokens": T,
+                                 "l2": "flushed between a kernel's timed launches"},
+                      "peaks": pk, "sizes": out}))
+    return 0
+
+
+SEMANEX_SIZES = {
+    # width, heads, state and feed-forward weights of the sizes above: a plain feed-forward of 1.5 ff has a gated one's bytes; the
+    # latent row (rank + shared rotated part) is as wide as the other designs' latent
+    "1b": dict(width=2048, heads=16, kv_heads=4, att_dim=128, q_rank=768, kv_rank=96, rot=32, ssm_heads=16, state=64, value=128, groups=1, conv=4,
+               taps=4, ff=12288, gated_ff=8192),
+    "8b": dict(width=4096, heads=32, kv_heads=8, att_dim=128, q_rank=1536, kv_rank=96, rot=32, ssm_heads=32, state=64, value=128, groups=1, conv=4,
+               taps=4, ff=21504, gated_ff=14336),
+}
+
+
+def semanex_workload(args):
+    """Prefill (one prompt of 2,048 tokens) and decode (batch 8 and 64 at context 2,048) tokens per second of a four-layer Semanex
+    model at a real model's layer sizes (parallel, latent attention, latent attention, parallel), beside a four-layer Sopalorn (the
+    closest design here: attention beside a recurrence in one layer) and a four-layer Zemezen (a recurrence, latent attention) of the
+    same width, heads, state, latent and feed-forward weights; then every kernel the design added or changed, alone, against its
+    roofline, beside the like kernel of the closest path.  Random weights, synthetic tokens, bfloat16, CUDA events, an L2 flush
+    between the timed launches of a kernel."""
+    import numpy as np
+    import torch
+    from dotllm_b200 import Model
+    from dotllm_b200.config import config_from_dict
+    from dotllm_b200.engine.step import AttentionPlan
+    from dotllm_b200.kernels import ops
+    tools = design_bench_tools(args)
+    pk, hbm, tflops, dev, T, ctx, sampler, timed, model_points = (tools.pk, tools.hbm, tools.tflops, tools.dev, tools.T, tools.ctx,
+                                                                  tools.sampler, tools.timed, tools.model_points)
+    sizes = ["1b", "8b"] if args.shape not in ("1b",) else ["1b"]
+
+    def kernel_table(z):
+        W, H, hd, nkv, r, rot, rq = z["width"], z["heads"], z["att_dim"], z["kv_heads"], z["kv_rank"], z["rot"], z["q_rank"]
+        S, N, P, G, K = z["ssm_heads"], z["state"], z["value"], z["groups"], z["conv"]
+        inner, C, lay = S * P, S * P + 2 * G * N, r + rot
+        bf = torch.bfloat16
+        rows = {}
+        i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+        rnd = lambda *s: torch.randn(*s, device=dev)
+
+        def row(name, fn, bytes_=0, flops=0):
+            us = timed(fn) * 1000.0
+            need = max(bytes_ / hbm, flops / tflops) * 1e6
+            rows[name] = {"us": round(us, 1), "roofline_us": round(need, 2), "frac": round(need / us, 4)}
+        for label, n, n_seqs in (("prefill", T, 1), ("decode", 64, 64)):
+            each = n // n_seqs
+            cu = torch.arange(0, n + 1, each, dtype=torch.int32, device=dev)
+            seq = torch.arange(n, dtype=torch.int32, device=dev) // each
+            slots = torch.arange(n_seqs, dtype=torch.int32, device=dev)
+            # the norm behind the sum and the input convolution, beside the residual add fused into an RMS norm
+            x, y, one, ones = rnd(n, W), rnd(n, W), torch.ones(1, device=dev), torch.ones(W, device=dev)
+            taps, hist = rnd(z["taps"], W) * 0.1, torch.zeros(n_seqs + 1, (z["taps"] - 1) * W, device=dev)
+            write = ops.PostNormed(y, 3.0, one, 1e-5)
+            row(f"post_norm {label}", lambda: ops.post_norm(x, write, bf), bytes_=n * W * (8 + 4 + 2))
+            if label == "decode":
+                row(f"post_norm + input convolution {label}", lambda: ops.post_norm(x, write, bf, conv=(taps, hist, slots)),
+                    bytes_=n * W * (8 + 4 + 2 + 8 * (z["taps"] - 1)))
+            else:
+                row(f"input convolution {label}", lambda: ops.causal_conv(x, taps, hist, cu, slots, each, add_input=True, out_dtype=bf),
+                    bytes_=n * W * (4 + 2))
+            row(f"llama add_rmsnorm {label}", lambda: ops.add_rmsnorm(x, y, ones, 1e-5, bf), bytes_=n * W * (8 + 4 + 2))
+            # the recurrence with its convolution and its gated norm, beside the delta rule's and the linear attention's
+            proj = rnd(n, 2 * inner + 2 * G * N + S).to(bf)
+            ctaps, cbias = rnd(K, C) * 0.5, torch.zeros(C, device=dev)
+            memory = torch.zeros(n_seqs + 1, S * N * P + (K - 1) * C, device=dev)
+            conv = lambda: ops.causal_conv(proj[:, :C], ctaps, memory[:, S * N * P:], cu, slots, each, bias=cbias, activation="silu")
+            zeros = torch.zeros(S, device=dev)
+            xbc = conv()
+            scan = lambda: ops.ssd_scan(xbc, proj[:, C + inner:C + inner + S], zeros, zeros, zeros, cu, slots, memory, S, G, N, P)
+            state_io = 2 * n_seqs * S * N * P * 4
+            row(f"causal_conv + silu {label}", conv, bytes_=n * C * (2 + 4))
+            row(f"ssd_scan {label}", scan, bytes_=n * (C + inner) * 4 + state_io, flops=6 * n * S * N * P)
+            row(f"causal_conv + ssd_scan {label}", lambda: (conv(), scan()), bytes_=n * (C * 2 + inner * 4) + state_io, flops=6 * n * S * N * P)
+            dq = rnd(n, 2 * S * N + S * P + S).to(bf)
+            dtaps = (rnd(2 * S * N + S * P, K) * 0.5).to(bf)
+            dmem = torch.zeros(n_seqs + 1, S * N * P + (K - 1) * (2 * S * N + S * P), device=dev)
+            zh = rnd(n, S)
+            row(f"sopalorn delta_rule (convolution + scan) {label}",
+                lambda: ops.delta_rule(dq, dtaps, dq[:, 2 * S * N + S * P:], zh, zeros, zeros, seq, cu, slots, dmem, S, S, N, P, N ** -0.5, 1e-6,
+                                       head_decay=True), bytes_=n * (dq.shape[1] * 2 + inner * 4) + state_io, flops=6 * n * S * N * P)
+            state = torch.zeros(n_seqs + 1, S, N, P, device=dev)
+            decay = torch.full((S,), 0.97, device=dev)
+            row(f"sopalorn gla_scan, constant decays {label}",
+                lambda: ops.gla_scan(dq[:, :S * N], dq[:, S * N:2 * S * N], dq[:, 2 * S * N:2 * S * N + S * P], None, decay, cu, slots, state, S, N, P, 1.0),
+                bytes_=n * (2 * S * N + S * P) * 2 + n * inner * 4 + state_io, flops=4 * n * S * N * P)
+            yy, gain = scan(), torch.ones(inner, device=dev)
+            gate = proj[:, C:C + inner]
+            row(f"gated_group_norm {label}", lambda: ops.gated_group_norm(yy, gate, gain, 1, 1e-5), bytes_=n * inner * (4 + 2 + 2))
+            g2 = gate.contiguous()
+            row(f"sopalorn head_norm_gate over all heads {label}", lambda: ops.head_norm_gate(yy, g2, gain, 1, inner, 1e-5, bf),
+                bytes_=n * inner * (4 + 2 + 2))
+            # attention with capped scores, a norm per head and a gate per channel
+            qkv = rnd(n, (H + 2 * nkv) * hd).to(bf)
+            gq = torch.ones(hd, device=dev)
+            row(f"head_rmsnorm (queries and keys) {label}", lambda: ops.head_rmsnorm(qkv[:, :(H + nkv) * hd], gq, H, hd, 1e-5, gq, nkv),
+                bytes_=n * (H + nkv) * hd * 4)
+            per = ctx if label == "decode" else n
+            pages = (per + 63) // 64
+            table = torch.arange(n_seqs * pages, dtype=torch.int32, device=dev).reshape(n_seqs, pages)
+            starts, news = ([0], [n]) if label == "prefill" else ([ctx - 1] * n_seqs, [1] * n_seqs)
+            totals = [s0 + s1 for s0, s1 in zip(starts, news)]
+            pos = i32([s0 + i for s0, s1 in zip(starts, news) for i in range(s1)])
+            seen = sum(p + 1 for p in pos.tolist())
+
+            def attend(name, q, heads, kv, width, **kw):
+                k_pool, v_pool = rnd(n_seqs * pages + 1, kv, 64, width).to(bf), rnd(n_seqs * pages + 1, kv, width, 64).to(bf)
+                plan = AttentionPlan(n_seqs, max(news), max(totals), label == "decode", i32(starts), i32(news),
+                                     i32([0] + list(np.cumsum(news))), i32(totals), list(starts), list(news))
+                row(f"{name} {label}", lambda: ops.attention(q, k_pool, v_pool, seq, pos, table, heads, kv, width, width ** -0.5, 0, plan=plan, **kw),
+                    bytes_=per * n_seqs * kv * width * 2 * 2 + n * heads * width * 4, flops=4 * seen * heads * width)
+            q = qkv[:, :H * hd]
+            attend("attention, capped scores", q, H, nkv, hd, score_hook=ops.ScoreHook(30.0))
+            attend("llama attention", q, H, nkv, hd)
+            o, cg = rnd(n, H * hd).to(bf), rnd(n, H * hd).to(bf)
+            row(f"channel_gate {label}", lambda: ops.channel_gate(o, cg, H, hd), bytes_=n * H * hd * 6)
+            hg = rnd(n, H).to(bf)
+            row(f"komulorn head_gate {label}", lambda: ops.head_gate(o, hg, H, hd), bytes_=n * H * hd * 4)
+            # latent attention: the rows, the queries, the attention over them with sinks, the way back
+            lp = rnd(n, rq + r + rot).to(bf)
+            ang = torch.arange(8192, device=dev)[:, None] * 1e-4 ** (torch.arange(rot // 2, device=dev) * 2.0 / rot)[None, :]
+            tables = (torch.cos(ang).contiguous(), torch.sin(ang).contiguous())
+            row(f"latent_rows {label}", lambda: ops.latent_rows(lp, torch.ones(rq, device=dev), torch.ones(r, device=dev), 1e-5, rot, tables, pos, lay),
+                bytes_=n * (rq + r + rot) * 4)
+            lat = rnd(n, rq)
+            row(f"kubedra norm of a query latent {label}", lambda: ops.add_rmsnorm(lat, None, torch.ones(rq, device=dev), 1e-5, bf), bytes_=n * rq * 6)
+            d_un = hd - rot
+            lq, wk = rnd(n, H * hd).to(bf), (rnd(H, r, d_un) * 0.1).to(bf)
+            row(f"latent_queries {label}", lambda: ops.latent_queries(lq, wk, rot, tables, pos, lay),
+                bytes_=n * H * (hd + lay) * 2 + H * r * d_un * 2, flops=2 * n * H * r * d_un)
+            wk2 = (rnd(H, lay, hd) * 0.1).to(bf)
+            row(f"kubedra queries to the latent {label}", lambda: ops.linear_per_head(lq, wk2), bytes_=n * H * (hd + lay) * 2 + H * lay * hd * 2,
+                flops=2 * n * H * lay * hd)
+            lqw = rnd(n, H * lay).to(bf)
+            attend("latent attention, sinks", lqw, H, 1, lay, sinks=torch.zeros(H, device=dev), split=True)
+            attend("kubedra latent attention", lqw, H, 1, lay)
+            wv = (rnd(H, hd, r) * 0.1).to(bf)
+            row(f"back from the latent, gate per channel {label}",
+                lambda: (lambda t: ops.channel_gate(t, cg, H, hd, out=t))(ops.linear_per_head(lqw, wv, x_head=lay)),
+                bytes_=n * H * (r + 2 * hd) * 2 + H * r * hd * 2, flops=2 * n * H * r * hd)
+            wv2 = (rnd(H, hd, lay) * 0.1).to(bf)
+            row(f"kubedra back from the latent {label}", lambda: ops.linear_per_head(lqw, wv2), bytes_=n * H * (lay + hd) * 2 + H * lay * hd * 2,
+                flops=2 * n * H * lay * hd)
+            # the plain feed-forward's first product with gelu in its epilogue, beside the gated one of equal weights
+            xb = rnd(n, W).to(bf)
+            wu, wgu = (rnd(z["ff"], W) * 0.02).to(bf), (rnd(2 * z["gated_ff"], W) * 0.02).to(bf)
+            row(f"product + exact gelu {label}", lambda: ops.activated_linear(xb, wu, "gelu", resident=True),
+                bytes_=z["ff"] * W * 2 + n * W * 2 + n * z["ff"] * 2, flops=2 * n * z["ff"] * W)
+            row(f"llama gated product {label}", lambda: ops.gated_linear(xb, wgu, resident=True),
+                bytes_=2 * z["gated_ff"] * W * 2 + n * W * 2 + n * z["gated_ff"] * 2, flops=2 * n * 2 * z["gated_ff"] * W)
+            del wu, wgu
+        return rows
+
+    out = {}
+    for name in sizes:
+        z = SEMANEX_SIZES[name]
+        vocab = 32000
+        scale, D = z["att_dim"] ** -0.5, z["att_dim"]
+        latent = {"type": "latent_attention", "mlp": {"kind": "dense", "ff": z["ff"]},
+                  "mixer": {"heads": z["heads"], "dim": D - z["rot"], "rot_dim": z["rot"], "vdim": D, "q_rank": z["q_rank"], "kv_rank": z["kv_rank"],
+                            "scale": scale, "rot": {"dims": z["rot"], "base": 10000.0}}}
+        left = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": D, "vdim": D, "scale": scale}
+        both = {"type": "parallel", "mlp": {"kind": "dense", "ff": z["ff"]},
+                "mixer": {"left": dict(left, softcap=30.0), "left_scale": 0.7, "right_scale": 0.7,
+                          "right": {"heads": z["ssm_heads"], "vdim": z["value"], "state": z["state"], "groups": z["groups"], "conv": z["conv"],
+                                    "norm_groups": 1}}}
+        xcfg = {"architecture": "Semanex", "vocab": vocab, "width": z["width"], "max_positions": 8192, "norm": {"eps": 1e-5}, "postln_alpha": 3.0,
+                "canon": {"taps": z["taps"]}, "embedding": {"scale": 1.0}, "layers": [both, latent, latent, both]}
+        dense = {"kind": "dense", "ff": z["gated_ff"], "limit": 7.0}
+        att = {"type": "attention", "mlp": dense, "mixer": dict(left, rot={"dims": 64, "base": 10000.0})}
+        pair = {"type": "parallel", "mlp": dense,
+                "mixer": {"left": left, "right": {"heads": z["ssm_heads"], "kv_heads": z["ssm_heads"], "dim": z["state"], "vdim": z["value"],
+                                                  "conv": z["conv"]}}}
+        scfg = {"architecture": "Sopalorn", "vocab": vocab, "width": z["width"], "max_positions": 8192, "norm": {"eps": 1e-5},
+                "embedding": {"scale": 1.0}, "logit_scale": 1.0, "layers": [pair, att, att, pair]}
+        zdense = {"kind": "dense", "ff": z["gated_ff"]}
+        delta = {"type": "channel_delta", "mlp": zdense, "mixer": {"heads": z["ssm_heads"], "kv_heads": z["ssm_heads"], "dim": z["state"],
+                                                                   "vdim": z["value"], "conv": z["conv"], "ranks": [64, 64]}}
+        zlat = {"type": "latent_attention", "mlp": zdense, "mixer": {"heads": z["heads"], "dim": D, "vdim": D, "kv_rank": z["kv_rank"] + z["rot"],
+                                                                     "scale": scale}}
+        zcfg = {"architecture": "Zemezen", "vocab": vocab, "width": z["width"], "max_positions": 8192, "norm": {"eps": 1e-5},
+                "layers": [delta, zlat, zlat, delta]}
+        point = {}
+        for label, cfg_dict in (("semanex", xcfg), ("sopalorn", scfg), ("zemezen", zcfg)):
+            model = Model.random(config_from_dict(cfg_dict), seed=0, dtype="bfloat16", device="cuda:0", on_device=True)
+            point[label] = model_points(model, vocab)
+            print(f"[bench] {name} {label}: {point[label]}", file=sys.stderr, flush=True)
+            del model
+            torch.cuda.empty_cache()
+        point["kernels"] = kernel_table(z)
+        for k, v in point["kernels"].items():
+            print(f"[bench] {name} {k}: {v}", file=sys.stderr, flush=True)
+        out[name] = point
+    first = out[sizes[0]]
+    print(json.dumps({"metric": "semanex_decode_tokens_per_second", "value": first["semanex"]["decode_b8_tok_s"], "unit": "tokens/s",
+                      "n_gpus": 1, "steps": args.steps, "warmup": max(3, args.warmup), "higher_is_better": True, "dtype": "bf16",
+                      "data": "synthetic", "vs_baseline": None, "clocks": sampler.stop(),
+                      "config": {"model": "Semanex, four layers at the sizes named", "batch": 8, "context": ctx, "prefill_tokens": T,
                                  "l2": "flushed between a kernel's timed launches"},
                       "peaks": pk, "sizes": out}))
     return 0

@@ -42,10 +42,13 @@ def decode_fits(group, head_dim):
     return 2 * 2 * 64 * head_dim * 2 + 4 * group * (head_dim + 4) * 4 + 4096 <= 227 * 1024
 
 
-def decode_tiles(n_heads, n_kv_heads):
+def decode_tiles(n_heads, n_kv_heads, split=True):
     """KV heads as the decode kernel counts them: a head of the pages whose group of query heads has more rows than a tile (16)
-    is walked by several tiles of query heads, each of equally many (a group of a prime number of heads: one head a tile)."""
+    is walked by several tiles of query heads, each of equally many (a group of a prime number of heads: one head a tile);
+    without ``split`` such a group is not taken (0)."""
     group = n_heads // n_kv_heads
+    if group > 16 and not split:
+        return 0
     return n_kv_heads * next(p for p in range(1, group + 1) if group % p == 0 and group // p <= 16)
 
 
@@ -91,14 +94,16 @@ FRESH_ROTATE_HEAD_DIMS = (64, 128)   # head sizes whose rotation the decode kern
 
 
 def decode_fresh(q, k, v, cos, sin, rotary_dim, block_table, k_pool, v_pool, n_heads, n_kv_heads, head_dim,
-                 scale, window, plan, biases=None, gate=None, sinks=None, softcap=0.0):
+                 scale, window, plan, biases=None, gate=None, sinks=None, softcap=0.0, split=False):
     """A decode step with the new token handled inside the attention kernel (rotation of q and k,
     cache write, attention): returns the output, or None when the sizes are not the kernel's.
     ``biases`` (q, k, v: float32 vectors or None) are added before the rotation and ``gate`` ([B, n_heads] logits of
     q's dtype, a column view is fine) multiplies each head's output by its sigmoid, both inside the kernel; with them
-    k and v may be None (a layer that reads another's cache: only the queries are biased and rotated).  ``sinks`` and
-    ``softcap`` as in ``run``."""
-    tiles = decode_tiles(n_heads, n_kv_heads)
+    k and v may be None (a layer that reads another's cache: only the queries are biased and rotated).  ``sinks``,
+    ``softcap`` and ``split`` as in ``run``."""
+    tiles = decode_tiles(n_heads, n_kv_heads, split)
+    if tiles == 0:
+        return None
     group = n_heads // tiles
     if not (plan.all_single and q.shape[0] == plan.n_seqs and head_dim in DECODE_HEAD_DIMS
             and decode_fits(group, head_dim) and (rotary_dim == 0 or (rotary_dim == head_dim
@@ -181,19 +186,21 @@ def _prefill(q, q_stride, out, k_pool, v_pool, n_pages, block_table, n_heads, n_
 
 
 def run(q, q_stride, out, k_pool, v_pool, n_pages, token_seq, token_pos, block_table,
-        n_heads, n_kv_heads, head_dim, scale, window, plan, keep_first=0, sinks=None, softcap=0.0):
+        n_heads, n_kv_heads, head_dim, scale, window, plan, keep_first=0, sinks=None, softcap=0.0, split=False):
     """Run a tensor-core kernel into ``out`` and return True, or return False to let the
     generic kernel take the call.  Kept first tokens and sinks are taken by the decode kernel (the kept pages join the
     step's list of pages; the sink's term enters where a head is normalised) and by both prefill kernels (the tcgen05 one
     walks the kept pages ahead of the window's, the mma.sync one lists them per tile).  ``softcap`` c > 0: scaled scores s
-    become c tanh(s / c), in all three."""
+    become c tanh(s / c), in all three.  ``split``: decode steps of more than 16 query heads a KV head run as several tiles of
+    query heads over the same pages (otherwise they are the generic kernel's)."""
     if q.dtype != torch.bfloat16 or q_stride % 8 or q.data_ptr() % 16 or head_dim not in DECODE_HEAD_DIMS:
         return False
     special = bool(keep_first) or sinks is not None
     if special and (out.stride(0) % 2 or out.data_ptr() % 4):
         return False
     if plan.all_single and q.shape[0] == plan.n_seqs and (DECODE_SPECIAL or not special):
-        if not decode_fits(n_heads // decode_tiles(n_heads, n_kv_heads), head_dim):
+        tiles = decode_tiles(n_heads, n_kv_heads, split)
+        if tiles == 0 or not decode_fits(n_heads // tiles, head_dim):
             return False
         return _decode(q, q_stride, out, k_pool, v_pool, n_pages, block_table, n_heads, n_kv_heads,
                        head_dim, scale, window, plan, keep_first, sinks, softcap)

@@ -579,7 +579,8 @@ class ScoreHook:
 
 
 def attention(q, k_pool, v_pool, token_seq, token_pos, block_table, n_heads, n_kv_heads,
-              head_dim, scale, window=0, plan=None, score_hook=None, value_dim=None, gate=None, keep_first=0, sinks=None):
+              head_dim, scale, window=0, plan=None, score_hook=None, value_dim=None, gate=None, keep_first=0, sinks=None,
+              split=False):
     """Causal attention of the step's tokens over their sequences' cached keys and values.
 
     q [T, nh*hd] (row-contiguous view); returns [T, nh*vd] of q's dtype (vd = ``value_dim``, default hd).
@@ -589,7 +590,9 @@ def attention(q, k_pool, v_pool, token_seq, token_pos, block_table, n_heads, n_k
     generic kernel runs.  ``gate`` [T, nh] of q's dtype (a column view is fine): head h's output is multiplied by
     sigmoid(gate[t, h]) - in the generic kernel's last step, or by ``head_gate`` behind a tensor-core kernel.
     ``keep_first`` n > 0 (with a window): a sequence's first n keys stay visible when the window has passed them.
-    ``sinks`` float32 [nh]: head h's softmax has one more term exp(sinks[h]) in its denominator, with no key and no value."""
+    ``sinks`` float32 [nh]: head h's softmax has one more term exp(sinks[h]) in its denominator, with no key and no value.
+    ``split``: let a bfloat16 decode step of more than 16 query heads a KV head run as several tiles of query heads over the same
+    pages on the tensor cores."""
     vd = int(value_dim or head_dim)
     _need_cuda(q, k_pool, v_pool, token_seq, token_pos, block_table, gate, sinks)
     if sinks is not None and (sinks.dtype != torch.float32 or sinks.shape != (n_heads,) or not sinks.is_contiguous()):
@@ -621,7 +624,7 @@ def attention(q, k_pool, v_pool, token_seq, token_pos, block_table, n_heads, n_k
     if plan is not None and q.dtype == torch.bfloat16 and slopes is None and vd == head_dim:
         if attention_fast.run(q, qs, out, k_pool, v_pool, n_pages, token_seq, token_pos, block_table,
                               n_heads, n_kv_heads, head_dim, float(scale), int(window), plan,
-                              keep_first=int(keep_first), sinks=sinks, softcap=softcap):
+                              keep_first=int(keep_first), sinks=sinks, softcap=softcap, split=split):
             return out if gate is None else head_gate(out, gate, n_heads, vd)
     _library.call("dl_attention_generic", _ptr(q), qs, _ptr(out), out.stride(0), _code(q.dtype),
                   _ptr(k_pool), _ptr(v_pool), n_pages, _ptr(token_seq), _ptr(token_pos),
@@ -632,7 +635,7 @@ def attention(q, k_pool, v_pool, token_seq, token_pos, block_table, n_heads, n_k
 
 def rope_cache_attention(q, k, v, cos, sin, rotary_dim, token_seq, token_pos, block_table, k_pool, v_pool,
                          n_heads, n_kv_heads, head_dim, scale, window=0, plan=None, score_hook=None,
-                         value_dim=None, biases=None, gate=None, keep_first=0, sinks=None):
+                         value_dim=None, biases=None, gate=None, keep_first=0, sinks=None, split=False):
     """``rope_cache_write`` followed by ``attention`` (same arguments, same result).  A bfloat16
     decode step (one new token per sequence) with a full-width rotation of head size 64 or 128, or
     with no rotation, runs as one kernel that adds the biases, rotates q, puts the new keys and values into the
@@ -641,14 +644,14 @@ def rope_cache_attention(q, k, v, cos, sin, rotary_dim, token_seq, token_pos, bl
             and (value_dim or head_dim) == head_dim and (k is not None or biases is not None or gate is not None) and not keep_first:
         out = attention_fast.decode_fresh(q, k, v, cos, sin, rotary_dim, block_table, k_pool, v_pool, n_heads,
                                           n_kv_heads, head_dim, float(scale), int(window), plan, biases=biases, gate=gate, sinks=sinks,
-                                          softcap=score_hook.softcap if score_hook else 0.0)
+                                          softcap=score_hook.softcap if score_hook else 0.0, split=split)
         if out is not None:
             return out
     rope_cache_write(q, k, v, cos, sin, rotary_dim, token_seq, token_pos, block_table, k_pool, v_pool,
                      n_heads, n_kv_heads, head_dim, write_cache=k is not None, value_dim=value_dim, biases=biases)
     return attention(q, k_pool, v_pool, token_seq, token_pos, block_table, n_heads, n_kv_heads, head_dim,
                      scale, window, plan=plan, score_hook=score_hook, value_dim=value_dim, gate=gate,
-                     keep_first=keep_first, sinks=sinks)
+                     keep_first=keep_first, sinks=sinks, split=split)
 
 
 def qkv_rope_cache(x, w_qkv, cos, sin, rotary_dim, token_seq, token_pos, block_table, k_pool, v_pool,

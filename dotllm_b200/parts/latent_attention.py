@@ -152,7 +152,7 @@ class LatentAttentionMixer(Mixer):
         keys, values = (rows, rows[:, :self.value_width]) if cache_view.writes else (None, None)
         a = ops.rope_cache_attention(q, keys, values, None, None, 0, step.token_seq, step.token_pos, cache_view.block_table,
                                      cache_view.k, cache_view.v, H, 1, self.key_width, self.scale, int(self.window or 0),
-                                     plan=step.attention_plan, value_dim=self.value_width, sinks=self.sinks)
+                                     plan=step.attention_plan, value_dim=self.value_width, sinks=self.sinks, split=True)
         o = ops.linear_per_head(a, self.w_uv, x_head=self.value_width)                             # [T, H*dv]
         if self.gate:
             g = proj[:, self.gate_at:self.gate_at + H * self.value_dim]

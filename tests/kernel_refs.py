@@ -439,7 +439,7 @@ def _gather_some(k_pool, v_pool, pages, positions):
 
 
 def attention(q, k_pool, v_pool, token_seq, token_pos, block_table, n_heads, n_kv_heads,
-              head_dim, scale, window=0, plan=None, score_hook=None, value_dim=None, gate=None, keep_first=0, sinks=None):
+              head_dim, scale, window=0, plan=None, score_hook=None, value_dim=None, gate=None, keep_first=0, sinks=None, split=False):
     vd = value_dim or head_dim
     if score_hook or vd != head_dim or gate is not None or keep_first or sinks is not None:
         return _attention_general(q, k_pool, v_pool, token_seq, token_pos, block_table, n_heads, n_kv_heads, head_dim,
