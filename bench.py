@@ -1137,13 +1137,13 @@ def semanex_workload(args):
             proj = rnd(n, 2 * inner + 2 * G * N + S).to(bf)
             ctaps, cbias = rnd(K, C) * 0.5, torch.zeros(C, device=dev)
             memory = torch.zeros(n_seqs + 1, S * N * P + (K - 1) * C, device=dev)
-            conv = lambda: ops.causal_conv(proj[:, :C], ctaps, memory[:, S * N * P:], cu, slots, each, bias=cbias, activation="silu")
+            conv = lambda: ops.causal_conv(proj[:, :C], ctaps, memory[:, S * N * P:], cu, slots, each, bias=cbias, activation="silu", out_dtype=bf)
             zeros = torch.zeros(S, device=dev)
             xbc = conv()
-            scan = lambda: ops.ssd_scan(xbc, proj[:, C + inner:C + inner + S], zeros, zeros, zeros, cu, slots, memory, S, G, N, P)
+            scan = lambda: ops.ssd_scan(xbc, proj[:, C + inner:C + inner + S], zeros, zeros, zeros, cu, slots, memory, S, G, N, P, max_new=each)
             state_io = 2 * n_seqs * S * N * P * 4
-            row(f"causal_conv + silu {label}", conv, bytes_=n * C * (2 + 4))
-            row(f"ssd_scan {label}", scan, bytes_=n * (C + inner) * 4 + state_io, flops=6 * n * S * N * P)
+            row(f"causal_conv + silu {label}", conv, bytes_=n * C * (2 + 2))
+            row(f"ssd_scan {label}", scan, bytes_=n * (C * 2 + inner * 4) + state_io, flops=6 * n * S * N * P)
             row(f"causal_conv + ssd_scan {label}", lambda: (conv(), scan()), bytes_=n * (C * 2 + inner * 4) + state_io, flops=6 * n * S * N * P)
             dq = rnd(n, 2 * S * N + S * P + S).to(bf)
             dtaps = (rnd(2 * S * N + S * P, K) * 0.5).to(bf)
@@ -1209,7 +1209,7 @@ def semanex_workload(args):
             attend("kubedra latent attention", lqw, H, 1, lay)
             wv = (rnd(H, hd, r) * 0.1).to(bf)
             row(f"back from the latent, gate per channel {label}",
-                lambda: (lambda t: ops.channel_gate(t, cg, H, hd, out=t))(ops.linear_per_head(lqw, wv, x_head=lay)),
+                lambda: ops.latent_values(lqw, wv, lay, gate=cg),
                 bytes_=n * H * (r + 2 * hd) * 2 + H * r * hd * 2, flops=2 * n * H * r * hd)
             wv2 = (rnd(H, hd, lay) * 0.1).to(bf)
             row(f"kubedra back from the latent {label}", lambda: ops.linear_per_head(lqw, wv2), bytes_=n * H * (lay + hd) * 2 + H * lay * hd * 2,

@@ -15,13 +15,30 @@ __device__ __forceinline__ void lt_pair(float u, float v, float c, float s, floa
     b = v * c + u * s;
 }
 
-#define LT_THREADS 128
-
+// Channel c of a part of `rot` channels, its first rot_dims rotated; zeros beyond.
 template <typename T>
+__device__ __forceinline__ float lt_tail(const T* __restrict__ src, int c, int rot, int rot_dims, const float* __restrict__ cos_t,
+                                         const float* __restrict__ sin_t, int pos) {
+    if (c >= rot) return 0.f;
+    const float v = dl_to_f32<T>(src[c]);
+    if (c >= rot_dims) return v;
+    const size_t at = (size_t)pos * (rot_dims / 2) + (c >> 1);
+    const float other = dl_to_f32<T>(src[c ^ 1]), cs = cos_t[at], sn = sin_t[at];
+    float a, b;
+    lt_pair(c & 1 ? other : v, c & 1 ? v : other, cs, sn, a, b);
+    return c & 1 ? b : a;
+}
+
+#define LT_THREADS 128
+#define LT_KEEP 16                       // values of a latent a thread keeps in registers
+
+// Eight (bfloat16) or four (float32) neighbours at a time where everything is aligned for it (VEC), else one.
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(LT_THREADS)
 latent_rows_kernel(const T* __restrict__ x, int ld, int q_rank, int kv_rank, int rot, int rot_dims, const float* __restrict__ q_gain,
                    const float* __restrict__ kv_gain, float eps, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                    int table_rows, const int32_t* __restrict__ token_pos, T* __restrict__ q_out, T* __restrict__ kv_out, int lay) {
+    constexpr int V = VEC ? 16 / (int)sizeof(T) : 1;
     __shared__ float scratch[33];
     dl_launch_dependents();
     dl_grid_dependency_wait();
@@ -31,25 +48,52 @@ latent_rows_kernel(const T* __restrict__ x, int ld, int q_rank, int kv_rank, int
     const T* src = x + t * ld + (is_q ? 0 : q_rank);
     T* dst = is_q ? q_out + t * q_rank : kv_out + t * lay;
     const float* gain = is_q ? q_gain : kv_gain;
+    const bool keep = rank <= LT_THREADS * LT_KEEP;
+    float v[LT_KEEP];
     float ss = 0.f;
-    for (int c = threadIdx.x; c < rank; c += LT_THREADS) { const float v = dl_to_f32<T>(src[c]); ss += v * v; }
+    if (keep) {
+#pragma unroll
+        for (int i = 0; i < LT_KEEP / V; ++i) {
+            const int c = (threadIdx.x + i * LT_THREADS) * V;
+            if (VEC) {
+                uint4 raw = make_uint4(0u, 0u, 0u, 0u);
+                if (c < rank) raw = *reinterpret_cast<const uint4*>(src + c);
+                const T* r8 = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+                for (int e = 0; e < V; ++e) v[i * V + e] = dl_to_f32<T>(r8[e]);
+            } else {
+                v[i] = c < rank ? dl_to_f32<T>(src[c]) : 0.f;
+            }
+#pragma unroll
+            for (int e = 0; e < V; ++e) ss += v[i * V + e] * v[i * V + e];
+        }
+    } else {
+        for (int c = threadIdx.x; c < rank; c += LT_THREADS) { const float w = dl_to_f32<T>(src[c]); ss += w * w; }
+    }
     ss = dl_block_sum(ss, scratch);
     const float r = 1.0f / sqrtf(ss / (float)rank + eps);
-    for (int c = threadIdx.x; c < rank; c += LT_THREADS) dst[c] = dl_from_f32<T>(dl_to_f32<T>(src[c]) * r * gain[c]);
+    if (keep) {
+#pragma unroll
+        for (int i = 0; i < LT_KEEP / V; ++i) {
+            const int c = (threadIdx.x + i * LT_THREADS) * V;
+            if (c >= rank) continue;
+            if (VEC) {
+                uint4 raw;
+                T* r8 = reinterpret_cast<T*>(&raw);
+#pragma unroll
+                for (int e = 0; e < V; ++e) r8[e] = dl_from_f32<T>(v[i * V + e] * r * gain[c + e]);
+                *reinterpret_cast<uint4*>(dst + c) = raw;
+            } else {
+                dst[c] = dl_from_f32<T>(v[i] * r * gain[c]);
+            }
+        }
+    } else {
+        for (int c = threadIdx.x; c < rank; c += LT_THREADS) dst[c] = dl_from_f32<T>(dl_to_f32<T>(src[c]) * r * gain[c]);
+    }
     if (is_q) return;
     const int pos = rot_dims > 0 ? min(token_pos[t], table_rows - 1) : 0;    // host-validated
-    for (int c = threadIdx.x; c < lay - kv_rank; c += LT_THREADS) {
-        float v = c < rot ? dl_to_f32<T>(src[kv_rank + c]) : 0.f;
-        if (c < rot_dims) {
-            const int i = c >> 1;
-            const float other = dl_to_f32<T>(src[kv_rank + (c ^ 1)]);
-            const float cs = cos_t[(size_t)pos * (rot_dims / 2) + i], sn = sin_t[(size_t)pos * (rot_dims / 2) + i];
-            float a, b;
-            lt_pair(c & 1 ? other : v, c & 1 ? v : other, cs, sn, a, b);
-            v = c & 1 ? b : a;
-        }
-        dst[kv_rank + c] = dl_from_f32<T>(v);
-    }
+    for (int c = threadIdx.x; c < lay - kv_rank; c += LT_THREADS)
+        dst[kv_rank + c] = dl_from_f32<T>(lt_tail<T>(src + kv_rank, c, rot, rot_dims, cos_t, sin_t, pos));
 }
 
 // x [tokens, q_rank + kv_rank + rot] of dtype (rows ld apart; q_rank 0: no query latent); gains float32; cos, sin float32
@@ -64,14 +108,18 @@ extern "C" int dl_latent_rows(const void* x, int dtype, int ld, int q_rank, int 
                "latent_rows: a tensor is missing");
     if (n_tokens == 0) return DL_OK;
     const dim3 grid(n_tokens, q_rank > 0 ? 2 : 1), block(LT_THREADS);
+    const int v = dtype == DL_BF16 ? 8 : 4;
+    const bool vec = q_rank % v == 0 && kv_rank % v == 0 && ld % v == 0 && lay % v == 0 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)kv_out % 16) == 0 &&
+                     ((uintptr_t)q_out % 16) == 0;
     cudaError_t e;
-    if (dtype == DL_F32)
-        e = dl_launch_dependent(latent_rows_kernel<float>, grid, block, 0, (cudaStream_t)stream, (const float*)x, ld, q_rank, kv_rank, rot,
-                                rot_dims, q_gain, kv_gain, eps, cos_t, sin_t, table_rows, token_pos, (float*)q_out, (float*)kv_out, lay);
-    else if (dtype == DL_BF16)
-        e = dl_launch_dependent(latent_rows_kernel<__nv_bfloat16>, grid, block, 0, (cudaStream_t)stream, (const __nv_bfloat16*)x, ld, q_rank,
-                                kv_rank, rot, rot_dims, q_gain, kv_gain, eps, cos_t, sin_t, table_rows, token_pos, (__nv_bfloat16*)q_out,
-                                (__nv_bfloat16*)kv_out, lay);
+#define LR_GO(T, VEC)                                                                                                                    \
+    e = dl_launch_dependent(latent_rows_kernel<T, VEC>, grid, block, 0, (cudaStream_t)stream, (const T*)x, ld, q_rank, kv_rank, rot, rot_dims, \
+                            q_gain, kv_gain, eps, cos_t, sin_t, table_rows, token_pos, (T*)q_out, (T*)kv_out, lay)
+    if (dtype == DL_F32 && vec) LR_GO(float, true);
+    else if (dtype == DL_F32) LR_GO(float, false);
+    else if (dtype == DL_BF16 && vec) LR_GO(__nv_bfloat16, true);
+    else if (dtype == DL_BF16) LR_GO(__nv_bfloat16, false);
+#undef LR_GO
     else
         return dl_fail(DL_ERR_UNSUPPORTED, "latent_rows: dtype %d", dtype);
     if (e != cudaSuccess) return dl_fail(DL_ERR_LAUNCH, "latent_rows: %s", cudaGetErrorString(e));
@@ -91,16 +139,7 @@ latent_query_tail_kernel(const T* __restrict__ q, int q_ld, int dim, int rot, in
     for (int e = threadIdx.x; e < H * tail; e += 256) {
         const int h = e / tail, c = e - h * tail;
         const T* src = q + t * q_ld + (size_t)h * (dim + rot) + dim;
-        float v = c < rot ? dl_to_f32<T>(src[c]) : 0.f;
-        if (c < rot_dims) {
-            const int i = c >> 1;
-            const float other = dl_to_f32<T>(src[c ^ 1]);
-            const float cs = cos_t[(size_t)pos * (rot_dims / 2) + i], sn = sin_t[(size_t)pos * (rot_dims / 2) + i];
-            float a, b;
-            lt_pair(c & 1 ? other : v, c & 1 ? v : other, cs, sn, a, b);
-            v = c & 1 ? b : a;
-        }
-        out[t * out_ld + (size_t)h * lay + rank + c] = dl_from_f32<T>(v);
+        out[t * out_ld + (size_t)h * lay + rank + c] = dl_from_f32<T>(lt_tail<T>(src, c, rot, rot_dims, cos_t, sin_t, pos));
     }
 }
 
@@ -181,5 +220,108 @@ extern "C" int dl_channel_gate(const void* o, int o_ld, int lay, const void* g, 
     else if (dtype == DL_BF16) e = gate_launch<__nv_bfloat16>(o, o_ld, lay, g, g_ld, out, out_ld, rows, heads, width, scale, (cudaStream_t)stream);
     else return dl_fail(DL_ERR_UNSUPPORTED, "channel_gate: dtype %d", dtype);
     if (e != cudaSuccess) return dl_fail(DL_ERR_LAUNCH, "channel_gate: %s", cudaGetErrorString(e));
+    return DL_OK;
+}
+
+// ---------------------------------------------------------------------------------------------------------------------
+// The change of basis per head for a few rows (a decode step), with what stands beside it in one kernel:
+//
+//   out[t, h * out_head + j] = f(sum_k W[h][j][k] x[t, h * x_head + k]),   f: nothing, or times sigmoid(gate[t, h * J + j])
+//
+// and, for queries on their way to the latent (`rot` >= 0), the rotated part of every head behind its J channels (rot channels of x
+// behind its K, zeros up to out_head).  A warp owns 16 rows of W and 8 NT tokens: mma.sync m16n8k16 with W as A, the operands
+// straight from memory, 16 bytes a lane (a lane's 8 neighbouring k of 32 are a permutation that both operands share).
+#define PH_WARPS 4
+
+__device__ __forceinline__ void ph_mma(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+    asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+        : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+        : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+template <int NT>
+__global__ void __launch_bounds__(32 * PH_WARPS)
+per_head_rows_kernel(const __nv_bfloat16* __restrict__ x, int x_ld, int x_head, const __nv_bfloat16* __restrict__ w, int J, int K,
+                     __nv_bfloat16* __restrict__ out, int out_ld, int out_head, const __nv_bfloat16* __restrict__ gate, int gate_ld, int rot,
+                     int rot_dims, const float* __restrict__ cos_t, const float* __restrict__ sin_t, int table_rows,
+                     const int32_t* __restrict__ token_pos, int n_tokens) {
+    dl_launch_dependents();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
+    const int h = blockIdx.y, tok0 = blockIdx.z * 8 * NT;
+    const int j_lo = (blockIdx.x * PH_WARPS + warp) * 16 + g, j_hi = j_lo + 8;
+    const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+    const __nv_bfloat16* w_lo = w + ((size_t)h * J + j_lo) * K + 8 * t;
+    const __nv_bfloat16* w_hi = w_lo + (size_t)8 * K;
+    uint4 a_lo = j_lo < J && 8 * t < K ? *reinterpret_cast<const uint4*>(w_lo) : zero;      // weights: no kernel of the stream writes them
+    uint4 a_hi = j_hi < J && 8 * t < K ? *reinterpret_cast<const uint4*>(w_hi) : zero;
+    dl_grid_dependency_wait();
+    float acc[NT][4];
+#pragma unroll
+    for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[n][e] = 0.f;
+    for (int k0 = 0; k0 < K; k0 += 32) {
+        const int k = k0 + 8 * t, kn = k + 32;
+        uint4 b[NT];
+#pragma unroll
+        for (int n = 0; n < NT; ++n) {
+            const int tok = tok0 + 8 * n + g;
+            b[n] = tok < n_tokens && k < K ? *reinterpret_cast<const uint4*>(x + (size_t)tok * x_ld + (size_t)h * x_head + k) : zero;
+        }
+        const uint4 n_lo = j_lo < J && kn < K ? *reinterpret_cast<const uint4*>(w_lo + k0 + 32) : zero;
+        const uint4 n_hi = j_hi < J && kn < K ? *reinterpret_cast<const uint4*>(w_hi + k0 + 32) : zero;
+#pragma unroll
+        for (int n = 0; n < NT; ++n) {
+            ph_mma(acc[n], a_lo.x, a_hi.x, a_lo.y, a_hi.y, b[n].x, b[n].y);
+            ph_mma(acc[n], a_lo.z, a_hi.z, a_lo.w, a_hi.w, b[n].z, b[n].w);
+        }
+        a_lo = n_lo;
+        a_hi = n_hi;
+    }
+#pragma unroll
+    for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int tok = tok0 + 8 * n + 2 * t + (e & 1), j = e < 2 ? j_lo : j_hi;
+            if (tok >= n_tokens || j >= J) continue;
+            float v = acc[n][e];
+            if (gate != nullptr) v /= 1.0f + expf(-__bfloat162float(gate[(size_t)tok * gate_ld + (size_t)h * J + j]));
+            out[(size_t)tok * out_ld + (size_t)h * out_head + j] = __float2bfloat16_rn(v);
+        }
+    if (rot < 0 || blockIdx.x != 0) return;
+    const int tail = out_head - J, mine = min(8 * NT, n_tokens - tok0);
+    for (int e = threadIdx.x; e < mine * tail; e += 32 * PH_WARPS) {
+        const int tok = tok0 + e / tail, c = e % tail;
+        const int pos = rot_dims > 0 ? min(token_pos[tok], table_rows - 1) : 0;
+        out[(size_t)tok * out_ld + (size_t)h * out_head + J + c] = __float2bfloat16_rn(
+            lt_tail<__nv_bfloat16>(x + (size_t)tok * x_ld + (size_t)h * x_head + K, c, rot, rot_dims, cos_t, sin_t, pos));
+    }
+}
+
+// x bf16 [tokens, H * x_head] (rows x_ld apart), w bf16 [H, J, K], out bf16 [tokens, H * out_head] (rows out_ld apart); K, x_ld and
+// x_head multiples of 8, x and w 16-byte aligned.  gate bf16 [tokens, H * J] (rows gate_ld apart) or NULL; rot -1: nothing behind the
+// J channels, else as in dl_latent_query_tail.
+extern "C" int dl_per_head_rows(const void* x, int x_ld, int x_head, const void* w, int H, int J, int K, void* out, int out_ld, int out_head,
+                                const void* gate, int gate_ld, int rot, int rot_dims, const float* cos_t, const float* sin_t, int table_rows,
+                                const int32_t* token_pos, int n_tokens, void* stream) {
+    DL_REQUIRE(n_tokens >= 0 && H > 0 && J > 0 && K > 0 && H <= 65535, "per_head_rows: bad sizes");
+    DL_REQUIRE(K % 8 == 0 && x_ld % 8 == 0 && x_head % 8 == 0 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)w % 16) == 0, "per_head_rows: operands come in aligned eights");
+    DL_REQUIRE(x_head >= K + (rot > 0 ? rot : 0) && out_head >= J + (rot > 0 ? rot : 0) && x_ld >= H * x_head && out_ld >= H * out_head &&
+                   (gate == nullptr || gate_ld >= H * J), "per_head_rows: rows overlap");
+    DL_REQUIRE(rot_dims >= 0 && rot_dims <= (rot > 0 ? rot : 0) && rot_dims % 2 == 0 && (rot_dims == 0 || (cos_t && sin_t && token_pos && table_rows > 0)),
+               "per_head_rows: a rotation needs tables and positions");
+    if (n_tokens == 0) return DL_OK;
+    const int nt = n_tokens <= 8 ? 1 : n_tokens <= 16 ? 2 : 4;
+    const dim3 grid((J + 16 * PH_WARPS - 1) / (16 * PH_WARPS), H, (n_tokens + 8 * nt - 1) / (8 * nt)), block(32 * PH_WARPS);
+    cudaError_t e;
+#define PH_GO(NT)                                                                                                                          \
+    e = dl_launch_dependent(per_head_rows_kernel<NT>, grid, block, 0, (cudaStream_t)stream, (const __nv_bfloat16*)x, x_ld, x_head,         \
+                            (const __nv_bfloat16*)w, J, K, (__nv_bfloat16*)out, out_ld, out_head, (const __nv_bfloat16*)gate, gate_ld, rot, \
+                            rot_dims, cos_t, sin_t, table_rows, token_pos, n_tokens)
+    if (nt == 1) PH_GO(1);
+    else if (nt == 2) PH_GO(2);
+    else PH_GO(4);
+#undef PH_GO
+    if (e != cudaSuccess) return dl_fail(DL_ERR_LAUNCH, "per_head_rows: %s", cudaGetErrorString(e));
     return DL_OK;
 }

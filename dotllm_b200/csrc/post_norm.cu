@@ -13,6 +13,7 @@
 #include "common.cuh"
 
 #define PN_THREADS 256
+#define PN_BIG 1024
 #define PN_MAX 8
 
 struct PnArgs {
@@ -66,22 +67,43 @@ __device__ __forceinline__ float4 pn_gain4(const float* gain, int step, int c) {
     return *reinterpret_cast<const float4*>(gain + c);
 }
 
-// The row in registers: NV pieces of four per thread.
-template <int NV>
-__global__ void __launch_bounds__(PN_THREADS) post_norm_kernel(const PnArgs a) {
+// The row in registers: NV pieces of four per thread.  KT > 0: a convolution of up to KT taps whose taps and history are asked for
+// together with the row, ahead of the norm's barriers; KT 0: none, or one of more taps, read where it is used.
+template <int THREADS, int NV, int KT>
+__global__ void __launch_bounds__(THREADS) post_norm_kernel(const PnArgs a) {
     __shared__ float scratch[33];
     dl_launch_dependents();
-    dl_grid_dependency_wait();
     const size_t row = blockIdx.x, base = row * a.width;
     const int tid = threadIdx.x;
+    float4 tap[NV][KT > 0 ? KT : 1], past[NV][KT > 1 ? KT - 1 : 1];
+    if (KT > 0) {                                            // weights: no kernel of the stream writes them
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+#pragma unroll
+            for (int j = 0; j < KT; ++j) {                   // place KT - 1 - lag meets the input `lag` rows back
+                const int c = (tid + i * THREADS) * 4, at = a.K - KT + j;
+                tap[i][j] = at >= 0 && c < a.width ? *reinterpret_cast<const float4*>(a.taps + (size_t)at * a.width + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+    }
+    dl_grid_dependency_wait();
+    const int slot = a.hist != nullptr ? a.slots[row] : -1;
+    const bool conv = slot >= 0 && slot < a.n_slots;
+    float* hs = conv ? a.hist + (size_t)slot * a.hist_stride : nullptr;
     float4 u[NV];
     float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-        const int c = (tid + i * PN_THREADS) * 4;
+        const int c = (tid + i * THREADS) * 4;
         u[i] = make_float4(0.f, 0.f, 0.f, 0.f);
         if (c < a.width) {
             u[i] = *reinterpret_cast<const float4*>(a.x + base + c);
+            if (KT > 1) {
+#pragma unroll
+                for (int j = 0; j + 1 < KT; ++j) {
+                    const int at = a.K - KT + j;
+                    past[i][j] = conv && at >= 0 ? *reinterpret_cast<const float4*>(hs + (size_t)at * a.width + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+                }
+            }
             if (a.y != nullptr) {
                 const float4 y = pn_load_y(a, row, c);
                 u[i] = make_float4(fmaf(a.alpha, u[i].x, y.x), fmaf(a.alpha, u[i].y, y.y), fmaf(a.alpha, u[i].z, y.z), fmaf(a.alpha, u[i].w, y.w));
@@ -95,7 +117,7 @@ __global__ void __launch_bounds__(PN_THREADS) post_norm_kernel(const PnArgs a) {
         ss = 0.f;
 #pragma unroll
         for (int i = 0; i < NV; ++i) {
-            const int c = (tid + i * PN_THREADS) * 4;
+            const int c = (tid + i * THREADS) * 4;
             if (c < a.width) {
                 const float4 g = pn_gain4(a.gain, a.gain_step, c);
                 u[i] = make_float4(u[i].x * r * g.x, u[i].y * r * g.y, u[i].z * r * g.z, u[i].w * r * g.w);
@@ -109,7 +131,7 @@ __global__ void __launch_bounds__(PN_THREADS) post_norm_kernel(const PnArgs a) {
         const float r = 1.0f / sqrtf(ss / (float)a.width + a.eps2);
 #pragma unroll
         for (int i = 0; i < NV; ++i) {
-            const int c = (tid + i * PN_THREADS) * 4;
+            const int c = (tid + i * THREADS) * 4;
             if (c < a.width) {
                 const float4 g = pn_gain4(a.gain2, a.gain2_step, c);
                 pn_store4(a, base + c, make_float4(u[i].x * r * g.x, u[i].y * r * g.y, u[i].z * r * g.z, u[i].w * r * g.w));
@@ -118,21 +140,28 @@ __global__ void __launch_bounds__(PN_THREADS) post_norm_kernel(const PnArgs a) {
         return;
     }
     if (a.out == nullptr) return;
-    const int slot = a.hist != nullptr ? a.slots[row] : -1;
-    const bool conv = slot >= 0 && slot < a.n_slots;
-    float* hs = conv ? a.hist + (size_t)slot * a.hist_stride : nullptr;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-        const int c = (tid + i * PN_THREADS) * 4;
+        const int c = (tid + i * THREADS) * 4;
         if (c >= a.width) continue;
         float4 h = u[i];
         if (conv) {
             float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-            for (int j = 0; j < a.K; ++j) {                      // oldest first; a history row moves to the place before it
-                const float4 w = *reinterpret_cast<const float4*>(a.taps + (size_t)j * a.width + c);
-                const float4 in = j + 1 < a.K ? *reinterpret_cast<const float4*>(hs + (size_t)j * a.width + c) : u[i];
-                if (j > 0) *reinterpret_cast<float4*>(hs + (size_t)(j - 1) * a.width + c) = in;
-                acc = make_float4(fmaf(w.x, in.x, acc.x), fmaf(w.y, in.y, acc.y), fmaf(w.z, in.z, acc.z), fmaf(w.w, in.w, acc.w));
+            if (KT > 0) {
+#pragma unroll
+                for (int j = 0; j < KT; ++j) {                   // oldest first; a history row moves to the place before it
+                    const float4 w = tap[i][j], in = j + 1 < KT ? past[i][j] : u[i];
+                    const int at = a.K - KT + j;
+                    if (at > 0) *reinterpret_cast<float4*>(hs + (size_t)(at - 1) * a.width + c) = in;
+                    acc = make_float4(fmaf(w.x, in.x, acc.x), fmaf(w.y, in.y, acc.y), fmaf(w.z, in.z, acc.z), fmaf(w.w, in.w, acc.w));
+                }
+            } else {
+                for (int j = 0; j < a.K; ++j) {
+                    const float4 w = *reinterpret_cast<const float4*>(a.taps + (size_t)j * a.width + c);
+                    const float4 in = j + 1 < a.K ? *reinterpret_cast<const float4*>(hs + (size_t)j * a.width + c) : u[i];
+                    if (j > 0) *reinterpret_cast<float4*>(hs + (size_t)(j - 1) * a.width + c) = in;
+                    acc = make_float4(fmaf(w.x, in.x, acc.x), fmaf(w.y, in.y, acc.y), fmaf(w.z, in.z, acc.z), fmaf(w.w, in.w, acc.w));
+                }
             }
             h = make_float4(h.x + acc.x, h.y + acc.y, h.z + acc.z, h.w + acc.w);
         }
@@ -212,15 +241,24 @@ extern "C" int dl_post_norm(float* x, const void* y, int y_dtype, int y_stride, 
     const bool vec = width % 4 == 0 && width <= PN_THREADS * 4 * PN_MAX && al16(x) && (y == nullptr || (al16(y) && y_stride % 4 == 0)) &&
                      (out == nullptr || al16(out)) && (hist == nullptr || (al16(hist) && hist_stride % 4 == 0 && al16(taps))) &&
                      (y == nullptr || gain_n == 1 || al16(gain)) && (gain2 == nullptr || gain2_n == 1 || al16(gain2));
-    const int pieces = (width / 4 + PN_THREADS - 1) / PN_THREADS;
+    // few rows (a decode step): as many threads as a row has pieces, up to 1,024
+    const bool big = rows <= 2 * dl_sm_count() && width > PN_THREADS * 4;
+    const int threads = big ? PN_BIG : PN_THREADS, pieces = (width / 4 + threads - 1) / threads;
+    const bool short_conv = hist != nullptr && K <= 4;
     cudaStream_t s = (cudaStream_t)stream;
     cudaError_t e;
-    const dim3 grid(rows), block(PN_THREADS);
+    const dim3 grid(rows), block(vec ? threads : PN_THREADS);
+#define PN_GO(T, NV, KT) e = dl_launch_dependent(post_norm_kernel<T, NV, KT>, grid, block, 0, s, a)
     if (!vec) e = dl_launch_dependent(post_norm_wide_kernel, grid, block, 0, s, a);
-    else if (pieces <= 1) e = dl_launch_dependent(post_norm_kernel<1>, grid, block, 0, s, a);
-    else if (pieces <= 2) e = dl_launch_dependent(post_norm_kernel<2>, grid, block, 0, s, a);
-    else if (pieces <= 4) e = dl_launch_dependent(post_norm_kernel<4>, grid, block, 0, s, a);
-    else e = dl_launch_dependent(post_norm_kernel<PN_MAX>, grid, block, 0, s, a);
+    else if (big && pieces <= 1 && short_conv) PN_GO(PN_BIG, 1, 4);
+    else if (big && pieces <= 1) PN_GO(PN_BIG, 1, 0);
+    else if (big) PN_GO(PN_BIG, 2, 0);
+    else if (pieces <= 1 && short_conv) PN_GO(PN_THREADS, 1, 4);
+    else if (pieces <= 1) PN_GO(PN_THREADS, 1, 0);
+    else if (pieces <= 2) PN_GO(PN_THREADS, 2, 0);
+    else if (pieces <= 4) PN_GO(PN_THREADS, 4, 0);
+    else PN_GO(PN_THREADS, PN_MAX, 0);
+#undef PN_GO
     if (e != cudaSuccess) return dl_fail(DL_ERR_LAUNCH, "post_norm: %s", cudaGetErrorString(e));
     return DL_OK;
 }

@@ -27,10 +27,12 @@ _library.register_signatures({
     "dl_head_rmsnorm": [_P, _I, _P, _I, _I, _P, _P, _I, _I, _I, _I, _I, _F, _P],
     "dl_post_norm": [_P, _P, _I, _I, _F, _P, _I, _F, _P, _I, _F, _P, _I, _I, _I, _P, ctypes.c_long, _I, _P, _P, _I, _P],
     "dl_causal_conv": [_P, _I, _I, _P, _I, _P, _I, _I, _P, ctypes.c_long, _I, _P, _P, _P, _I, _I, _I, _I, _I, _P],
-    "dl_ssd_scan": [_P, _I, _P, _I, _I, _P, _P, _P, _P, _P, _P, ctypes.c_long, _I, _P, _I, _I, _I, _I, _I, _I, _I, _P],
+    "dl_ssd_scan": [_P, _I, _I, _P, _I, _P, _P, _P, _P, _P, _P, ctypes.c_long, _I, _P, _I, _I, _I, _I, _I, _I, _I, _P],
+    "dl_ssd_chunk": [_P, _I, _P, _I, _P, _P, _P, _P, _P, _P, ctypes.c_long, _I, _P, _I, _I, _I, _I, _I, _I, _P],
     "dl_gated_group_norm": [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _F, _P],
     "dl_latent_rows": [_P, _I, _I, _I, _I, _I, _I, _P, _P, _F, _P, _P, _I, _P, _P, _P, _I, _I, _P],
     "dl_latent_query_tail": [_P, _I, _I, _I, _I, _I, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P],
+    "dl_per_head_rows": [_P, _I, _I, _P, _I, _I, _I, _P, _I, _I, _P, _I, _I, _I, _P, _P, _I, _P, _I, _P],
     "dl_channel_gate": [_P, _I, _I, _P, _I, _P, _I, _I, _I, _I, _I, _F, _P],
     "dl_delta_rule": [_P, _I, _P, _I, _I, _P, _I, _P, _I, _P, _P, _P, _P, _P, _P, _P, ctypes.c_long, _I,
                       _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _F, _I, _P],
@@ -784,15 +786,21 @@ def head_rmsnorm(x, gain_a, heads_a, dim, eps, gain_b=None, heads_b=0, lay=None)
 
 
 # --------------------------------------------------- state-space recurrence
-def ssd_scan(xbc, z, dt_bias, a_log, skip, cu_new, slots, memory, n_heads, groups, state, vdim):
+SSD_CHUNKED = True              # False: always the token-by-token scan (tests compare the two)
+SSD_CHUNK_MIN_TOKENS = 12       # steps whose longest sequence brings fewer tokens walk them one by one
+SSD_CHUNK_MAX_STATE = 256       # SC_MAX_STATE in csrc/ssd.cu
+
+
+def ssd_scan(xbc, z, dt_bias, a_log, skip, cu_new, slots, memory, n_heads, groups, state, vdim, max_new=1):
     """The recurrence S <- exp(-exp(a_log_h) dt) S + dt B x^T, y = S^T C + skip_h x with dt = softplus(z + dt_bias_h), over each
-    sequence's new rows in order.  xbc float32 [T, H*vdim + 2*groups*state]: x, then B, then C (head h uses group
-    h // (H/groups)); z [T, H] (a column view is fine); dt_bias, a_log, skip float32 [H]; memory float32 [slots, >=
+    sequence's new rows in order.  xbc [T, H*vdim + 2*groups*state]: x, then B, then C (head h uses group h // (H/groups));
+    z [T, H] of xbc's dtype (a column view is fine); ``max_new``: the most tokens a sequence brings - prompts of a bfloat16 run are
+    walked a chunk at a time on the tensor cores, with float32 products; dt_bias, a_log, skip float32 [H]; memory float32 [slots, >=
     H*state*vdim]: per slot every head's [state, vdim], read and updated.  Returns y float32 [T, H*vdim]."""
     _need_cuda(xbc, z, dt_bias, a_log, skip, cu_new, slots, memory)
     T, H, G, N, P = xbc.shape[0], int(n_heads), int(groups), int(state), int(vdim)
-    if xbc.dtype != torch.float32 or xbc.shape[1] != H * P + 2 * G * N or z.shape != (T, H):
-        raise KernelError(f"ssd_scan: float32 rows of {H * P + 2 * G * N} values and one step logit per head")
+    if xbc.dtype != z.dtype or xbc.shape[1] != H * P + 2 * G * N or z.shape != (T, H):
+        raise KernelError(f"ssd_scan: rows of {H * P + 2 * G * N} values and one step logit per head, of one dtype")
     for t, what in ((dt_bias, "dt_bias"), (a_log, "a_log"), (skip, "skip")):
         if t.dtype != torch.float32 or t.shape != (H,) or not t.is_contiguous():
             raise KernelError(f"ssd_scan: {what} must be contiguous float32 [{H}]")
@@ -801,7 +809,13 @@ def ssd_scan(xbc, z, dt_bias, a_log, skip, cu_new, slots, memory, n_heads, group
     _int32(cu_new, "ssd_scan cu_new")
     _int32(slots, "ssd_scan slots")
     out = torch.empty((T, H * P), dtype=torch.float32, device=xbc.device)
-    _library.call("dl_ssd_scan", _ptr(xbc), _rows_view(xbc, "ssd_scan xbc"), _ptr(z), _code(z.dtype), _rows_view(z, "ssd_scan z"),
+    ld, zld = _rows_view(xbc, "ssd_scan xbc"), _rows_view(z, "ssd_scan z")
+    if SSD_CHUNKED and xbc.dtype == torch.bfloat16 and max_new >= SSD_CHUNK_MIN_TOKENS and N % 8 == 0 and P % 8 == 0 and N <= SSD_CHUNK_MAX_STATE \
+            and ld % 8 == 0 and xbc.data_ptr() % 16 == 0:
+        _library.call("dl_ssd_chunk", _ptr(xbc), ld, _ptr(z), zld, _ptr(dt_bias), _ptr(a_log), _ptr(skip), _ptr(cu_new), _ptr(slots), _ptr(memory),
+                      memory.stride(0), memory.shape[0], _ptr(out), out.stride(0), slots.numel(), H, G, N, P, _stream())
+        return out
+    _library.call("dl_ssd_scan", _ptr(xbc), _code(xbc.dtype), ld, _ptr(z), zld,
                   _ptr(dt_bias), _ptr(a_log), _ptr(skip), _ptr(cu_new), _ptr(slots), _ptr(memory), memory.stride(0), memory.shape[0],
                   _ptr(out), out.stride(0), slots.numel(), T, H, G, N, P, _stream())
     return out
@@ -862,6 +876,32 @@ def latent_rows(x, q_gain, kv_gain, eps, rot, tables, token_pos, lay):
     return cq, kv
 
 
+PER_HEAD_ROWS = 128             # rows up to which the products per head run in the few-rows kernel (more: batched library products)
+
+
+def _per_head_rows_takes(x, w, x_head):
+    return (x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and 0 < x.shape[0] <= PER_HEAD_ROWS and w.shape[2] % 8 == 0 and x_head % 8 == 0
+            and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0 and w.is_contiguous())
+
+
+def latent_values(a, w_value, lay, gate=None):
+    """a [T, H*lay] (the attention's outputs in the latent's basis, the first rank channels of each head) -> [T, H*vdim]: per head
+    W_value[h] a (w_value [H, vdim, rank]), times sigmoid(gate) per channel where ``gate`` [T, H*vdim] (a column view is fine) is
+    given."""
+    _need_cuda(a, w_value, gate)
+    H, vd, r = w_value.shape
+    T = a.shape[0]
+    if a.shape[1] != H * lay or lay < r or (gate is not None and (gate.shape != (T, H * vd) or gate.dtype != a.dtype)):
+        raise KernelError(f"latent_values: {H} heads of {r} in {lay} channels and a gate [T, {H * vd}]")
+    if _per_head_rows_takes(a, w_value, lay):
+        out = torch.empty((T, H * vd), dtype=a.dtype, device=a.device)
+        _library.call("dl_per_head_rows", _ptr(a), _rows_view(a, "latent_values a"), int(lay), _ptr(w_value), H, vd, r, _ptr(out), out.stride(0), vd,
+                      _ptr(gate), _rows_view(gate, "latent_values gate") if gate is not None else 0, -1, 0, None, None, 0, None, T, _stream())
+        return out
+    o = linear_per_head(a, w_value, x_head=lay)
+    return o if gate is None else channel_gate(o, gate, H, vd, out=o)
+
+
 def latent_queries(q, w_key, rot, tables, token_pos, lay):
     """q [T, H*(dim + rot)] head by head -> [T, H*lay]: per head W_key[h] q[:dim] (w_key [H, rank, dim]), then the last ``rot``
     channels rotated as in ``latent_rows``, then zeros."""
@@ -873,6 +913,10 @@ def latent_queries(q, w_key, rot, tables, token_pos, lay):
         raise KernelError(f"latent_queries: {H} heads of {d} + {rot} channels into {lay}")
     _int32(token_pos, "latent_queries positions")
     out = torch.empty((T, H * lay), dtype=q.dtype, device=q.device)
+    if _per_head_rows_takes(q, w_key, d + rot):
+        _library.call("dl_per_head_rows", _ptr(q), _rows_view(q, "latent_queries q"), d + rot, _ptr(w_key), H, r, d, _ptr(out), out.stride(0),
+                      int(lay), None, 0, int(rot), dims, _ptr(cos), _ptr(sin), rows, _ptr(token_pos), T, _stream())
+        return out
     linear_per_head(q, w_key, x_head=d + rot, out=out, out_head=lay)
     _library.call("dl_latent_query_tail", _ptr(q), _code(q.dtype), _rows_view(q, "latent_queries q"), d, int(rot), dims, _ptr(cos), _ptr(sin),
                   rows, _ptr(token_pos), _ptr(out), out.stride(0), r, int(lay), H, T, _stream())

@@ -153,10 +153,8 @@ class LatentAttentionMixer(Mixer):
         a = ops.rope_cache_attention(q, keys, values, None, None, 0, step.token_seq, step.token_pos, cache_view.block_table,
                                      cache_view.k, cache_view.v, H, 1, self.key_width, self.scale, int(self.window or 0),
                                      plan=step.attention_plan, value_dim=self.value_width, sinks=self.sinks, split=True)
-        o = ops.linear_per_head(a, self.w_uv, x_head=self.value_width)                             # [T, H*dv]
-        if self.gate:
-            g = proj[:, self.gate_at:self.gate_at + H * self.value_dim]
-            o = ops.channel_gate(o, g, H, self.value_dim, out=o)
+        g = proj[:, self.gate_at:self.gate_at + H * self.value_dim] if self.gate else None
+        o = ops.latent_values(a, self.w_uv, self.value_width, gate=g)                             # [T, H*dv]
         return ops.linear(o, self.w_o, out_dtype=BRANCH_DTYPE, resident=True, lazy=True)
 
     def forward(self, x, step, cache_view):

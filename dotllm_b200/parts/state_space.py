@@ -7,8 +7,8 @@
     out = W_o (rms over equal parts of (y * silu(z)) * gain)               (the gate comes before the norm)
 
 What a sequence carries - every head's state and the convolution's last K - 1 inputs - is the layer execution's fixed-size
-cache entry, one float32 vector per slot, zero when a sequence opens.  From the convolution's sum on everything up to the
-gate is float32 in either run dtype.  The kernels walk a sequence's new tokens in order from that entry, so prompts, parts of
+cache entry, one float32 vector per slot, zero when a sequence opens.  The convolution leaves x, B and C in the run dtype (its sums
+are float32); steps, decays, the recurrence and everything up to the gate are float32 in either run dtype.  The kernels walk a sequence's new tokens in order from that entry, so prompts, parts of
 prompts and decoded tokens are one code path.
 """
 from __future__ import annotations
@@ -83,9 +83,9 @@ class StateSpaceMixer(Mixer):
         C, W, memory = self.channels, self.inner, cache_view.state
         z, dt = proj[:, C:C + W], proj[:, C + W:C + W + self.n_heads]
         xbc = ops.causal_conv(proj[:, :C], self.conv, memory[:, self.state_size:], step.cu_new, cache_view.slots,
-                              step.attention_plan.max_new, bias=self.conv_bias, activation="silu")
+                              step.attention_plan.max_new, bias=self.conv_bias, activation="silu", out_dtype=self.runtime.dtype)
         y = ops.ssd_scan(xbc, dt, self.dt_bias, self.rate, self.skip, step.cu_new, cache_view.slots, memory, self.n_heads, self.groups,
-                         self.state, self.value_dim)
+                         self.state, self.value_dim, max_new=step.attention_plan.max_new)
         return ops.gated_group_norm(y, z, self.norm_gain, self.norm_parts, self.eps, scale=scale, out=out)
 
     def forward(self, x, step, cache_view):

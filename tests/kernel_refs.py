@@ -239,7 +239,8 @@ def causal_conv(x, taps, memory, cu_new, slots, max_new, bias=None, activation=N
     return out.to(out_dtype or torch.float32)
 
 
-def ssd_scan(xbc, z, dt_bias, a_log, skip, cu_new, slots, memory, n_heads, groups, state, vdim):
+def ssd_scan(xbc, z, dt_bias, a_log, skip, cu_new, slots, memory, n_heads, groups, state, vdim, max_new=1):
+    xbc = xbc.to(torch.float32)
     T, H, G, N, P = xbc.shape[0], n_heads, groups, state, vdim
     x = xbc[:, :H * P].reshape(T, H, P)
     B = xbc[:, H * P:H * P + G * N].reshape(T, G, N).repeat_interleave(H // G, dim=1)
@@ -292,6 +293,11 @@ def latent_queries(q, w_key, rot, tables, token_pos, lay):
     head = torch.einsum("thd,hrd->thr", qf[..., :d], w_key.to(torch.float32))
     y = torch.cat([head, _rotated_pairs(qf[..., d:], tables, token_pos)], dim=-1)
     return torch.nn.functional.pad(y, (0, lay - r - rot)).reshape(q.shape[0], H * lay).to(q.dtype)
+
+
+def latent_values(a, w_value, lay, gate=None):
+    o = linear_per_head(a.to(torch.float32), w_value.to(torch.float32), x_head=lay)
+    return (o if gate is None else o * torch.sigmoid(gate.to(torch.float32))).to(a.dtype)
 
 
 def channel_gate(o, gate, heads, width, lay=None, scale=1.0, out=None):

@@ -142,21 +142,22 @@ def test_causal_convolution_alone(C, K, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("H,G,N,P", [(4, 2, 40, 48), (3, 3, 1, 5), (6, 1, 19, 7), (8, 2, 128, 64), (2, 1, 64, 24), (2, 2, 200, 10), (1, 1, 400, 9),
+@pytest.mark.parametrize("H,G,N,P", [(4, 2, 40, 48), (2, 1, 16, 8), (3, 1, 256, 40), (2, 2, 128, 128), (3, 3, 1, 5), (6, 1, 19, 7), (8, 2, 128, 64), (2, 1, 64, 24), (2, 2, 200, 10), (1, 1, 400, 9),
                                      (5, 5, 32, 33)])
 def test_state_space_scan_alone(H, G, N, P, dtype):
     """Unequal prompts, then portions and single tokens from the states they left, in slots that are not neighbours; the step
-    logits (in the projection's type) span decays from almost one to almost nothing."""
+    logits span decays from almost one to almost nothing.  bfloat16 prompts go a chunk at a time through the tensor cores where
+    the sizes allow, and give the scan's float32 results."""
     bias, a_log, skip = g32(H, seed=1), g32(H, seed=2, scale=0.7), g32(H, seed=3)
     memory = torch.zeros((6, H * N * P + 12), dtype=torch.float32, device=DEV)
     rmem = memory.cpu().clone()
     slots = i32([4, 0, 2])
-    for n, sizes in enumerate(([1, 37, 70], [5, 1, 2], [1, 1, 1])):
+    for n, sizes in enumerate(([1, 37, 70], [5, 1, 2], [1, 1, 1], [130, 64, 65])):
         T = sum(sizes)
-        xbc = g32(T, H * P + 2 * G * N + 4, seed=10 + n, scale=0.7)[:, :H * P + 2 * G * N]
+        xbc = g32(T, H * P + 2 * G * N + 8, seed=10 + n, scale=0.7).to(dtype)[:, :H * P + 2 * G * N]
         z = g32(T, H + 3, seed=20 + n, scale=3.0).to(dtype)[:, 1:H + 1]
         cu = i32([0] + list(np.cumsum(sizes)))
-        got = ops.ssd_scan(xbc, z, bias, a_log, skip, cu, slots, memory, H, G, N, P)
+        got = ops.ssd_scan(xbc, z, bias, a_log, skip, cu, slots, memory, H, G, N, P, max_new=max(sizes))
         want = kernel_refs.ssd_scan(xbc.cpu(), z.cpu(), bias.cpu(), a_log.cpu(), skip.cpu(), cu.cpu(), slots.cpu(), rmem, H, G, N, P)
         close(got, want, torch.float32), close(memory, rmem, torch.float32)
 
@@ -179,11 +180,11 @@ def test_gates_and_the_norm_over_parts_alone(dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("H,dim,rot,dims,rq,r,lay", [(4, 20, 8, 8, 28, 40, 64), (3, 7, 6, 0, 11, 13, 19), (6, 32, 32, 32, 96, 96, 128), (5, 16, 24, 12, 0, 40, 64)])
-def test_latent_rows_and_queries_alone(H, dim, rot, dims, rq, r, lay, dtype):
-    T = 9
+@pytest.mark.parametrize("T", [9, 3, 40, 150])
+@pytest.mark.parametrize("H,dim,rot,dims,rq,r,lay", [(4, 20, 8, 8, 28, 40, 64), (4, 24, 8, 8, 1536, 104, 128), (2, 72, 64, 64, 32, 64, 128), (3, 7, 6, 0, 11, 13, 19), (6, 32, 32, 32, 96, 96, 128), (5, 16, 24, 12, 0, 40, 64)])
+def test_latent_rows_and_queries_alone(H, dim, rot, dims, rq, r, lay, T, dtype):
     x = g32(T, rq + r + rot + 8, seed=1).to(dtype)[:, :rq + r + rot]
-    pos = i32([0, 1, 5, 63, 64, 99, 2, 2, 7])
+    pos = i32(([0, 1, 5, 63, 64, 99, 2, 2, 7] * 20)[:T])
     angle = torch.arange(100)[:, None] * 0.37 ** torch.arange(max(1, dims // 2))[None, :]
     tables = (torch.cos(angle).to(DEV).float().contiguous(), torch.sin(angle).to(DEV).float().contiguous()) if dims else None
     rtables = tuple(t.cpu() for t in tables) if dims else None
@@ -197,6 +198,9 @@ def test_latent_rows_and_queries_alone(H, dim, rot, dims, rq, r, lay, dtype):
     close(got, kernel_refs.latent_queries(q.cpu(), w.cpu(), rot, rtables, pos.cpu(), lay), dtype)
     assert not got.view(T, H, lay)[:, :, r + rot:].any()
     wo = g32(H, 12, r, seed=6, scale=0.3).to(dtype)
+    gate = g32(T, H * 12 + 8, seed=7).to(dtype)[:, 8:]
+    for gt in (gate, None):
+        close(ops.latent_values(got, wo, lay, gate=gt), kernel_refs.latent_values(got.cpu(), wo.cpu(), lay, gate=None if gt is None else gt.cpu()), dtype)
     close(ops.linear_per_head(got, wo, x_head=lay), kernel_refs.linear_per_head(got.cpu(), wo.cpu(), x_head=lay), dtype)
 
 
