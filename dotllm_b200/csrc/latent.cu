@@ -48,6 +48,11 @@ latent_rows_kernel(const T* __restrict__ x, int ld, int q_rank, int kv_rank, int
     const T* src = x + t * ld + (is_q ? 0 : q_rank);
     T* dst = is_q ? q_out + t * q_rank : kv_out + t * lay;
     const float* gain = is_q ? q_gain : kv_gain;
+    if (!is_q) {                                             // the part behind the latent: it waits for no sum
+        const int pos = rot_dims > 0 ? min(token_pos[t], table_rows - 1) : 0;    // host-validated
+        for (int c = threadIdx.x; c < lay - kv_rank; c += LT_THREADS)
+            dst[kv_rank + c] = dl_from_f32<T>(lt_tail<T>(src + kv_rank, c, rot, rot_dims, cos_t, sin_t, pos));
+    }
     const bool keep = rank <= LT_THREADS * LT_KEEP;
     float v[LT_KEEP];
     float ss = 0.f;
@@ -90,10 +95,6 @@ latent_rows_kernel(const T* __restrict__ x, int ld, int q_rank, int kv_rank, int
     } else {
         for (int c = threadIdx.x; c < rank; c += LT_THREADS) dst[c] = dl_from_f32<T>(dl_to_f32<T>(src[c]) * r * gain[c]);
     }
-    if (is_q) return;
-    const int pos = rot_dims > 0 ? min(token_pos[t], table_rows - 1) : 0;    // host-validated
-    for (int c = threadIdx.x; c < lay - kv_rank; c += LT_THREADS)
-        dst[kv_rank + c] = dl_from_f32<T>(lt_tail<T>(src + kv_rank, c, rot, rot_dims, cos_t, sin_t, pos));
 }
 
 // x [tokens, q_rank + kv_rank + rot] of dtype (rows ld apart; q_rank 0: no query latent); gains float32; cos, sin float32
@@ -231,7 +232,8 @@ extern "C" int dl_channel_gate(const void* o, int o_ld, int lay, const void* g, 
 // and, for queries on their way to the latent (`rot` >= 0), the rotated part of every head behind its J channels (rot channels of x
 // behind its K, zeros up to out_head).  A warp owns 16 rows of W and 8 NT tokens: mma.sync m16n8k16 with W as A, the operands
 // straight from memory, 16 bytes a lane (a lane's 8 neighbouring k of 32 are a permutation that both operands share).
-#define PH_WARPS 4
+#define PH_WARPS 2
+#define PH_K 4                           // pieces of 32 channels whose operands are in flight together
 
 __device__ __forceinline__ void ph_mma(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
     asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
@@ -252,31 +254,44 @@ per_head_rows_kernel(const __nv_bfloat16* __restrict__ x, int x_ld, int x_head, 
     const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
     const __nv_bfloat16* w_lo = w + ((size_t)h * J + j_lo) * K + 8 * t;
     const __nv_bfloat16* w_hi = w_lo + (size_t)8 * K;
-    uint4 a_lo = j_lo < J && 8 * t < K ? *reinterpret_cast<const uint4*>(w_lo) : zero;      // weights: no kernel of the stream writes them
-    uint4 a_hi = j_hi < J && 8 * t < K ? *reinterpret_cast<const uint4*>(w_hi) : zero;
+    // PH_K x 32 channels at a time: every operand of a run is asked for before the first product
+    uint4 a_lo[PH_K], a_hi[PH_K];
+    auto load_w = [&](int k0) {
+#pragma unroll
+        for (int i = 0; i < PH_K; ++i) {
+            const bool in = k0 + 32 * i + 8 * t < K;
+            a_lo[i] = in && j_lo < J ? *reinterpret_cast<const uint4*>(w_lo + k0 + 32 * i) : zero;
+            a_hi[i] = in && j_hi < J ? *reinterpret_cast<const uint4*>(w_hi + k0 + 32 * i) : zero;
+        }
+    };
+    load_w(0);                                               // weights: no kernel of the stream writes them
     dl_grid_dependency_wait();
-    float acc[NT][4];
+    float acc[NT][4], gv[NT][4];
 #pragma unroll
     for (int n = 0; n < NT; ++n)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) acc[n][e] = 0.f;
-    for (int k0 = 0; k0 < K; k0 += 32) {
-        const int k = k0 + 8 * t, kn = k + 32;
-        uint4 b[NT];
-#pragma unroll
-        for (int n = 0; n < NT; ++n) {
-            const int tok = tok0 + 8 * n + g;
-            b[n] = tok < n_tokens && k < K ? *reinterpret_cast<const uint4*>(x + (size_t)tok * x_ld + (size_t)h * x_head + k) : zero;
+        for (int e = 0; e < 4; ++e) {
+            const int tok = tok0 + 8 * n + 2 * t + (e & 1), j = e < 2 ? j_lo : j_hi;
+            acc[n][e] = 0.f;
+            gv[n][e] = gate != nullptr && tok < n_tokens && j < J ? __bfloat162float(gate[(size_t)tok * gate_ld + (size_t)h * J + j]) : 0.f;
         }
-        const uint4 n_lo = j_lo < J && kn < K ? *reinterpret_cast<const uint4*>(w_lo + k0 + 32) : zero;
-        const uint4 n_hi = j_hi < J && kn < K ? *reinterpret_cast<const uint4*>(w_hi + k0 + 32) : zero;
+    for (int k0 = 0; k0 < K; k0 += 32 * PH_K) {
+        uint4 b[NT][PH_K];
 #pragma unroll
-        for (int n = 0; n < NT; ++n) {
-            ph_mma(acc[n], a_lo.x, a_hi.x, a_lo.y, a_hi.y, b[n].x, b[n].y);
-            ph_mma(acc[n], a_lo.z, a_hi.z, a_lo.w, a_hi.w, b[n].z, b[n].w);
-        }
-        a_lo = n_lo;
-        a_hi = n_hi;
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+            for (int i = 0; i < PH_K; ++i) {
+                const int tok = tok0 + 8 * n + g, k = k0 + 32 * i + 8 * t;
+                b[n][i] = tok < n_tokens && k < K ? *reinterpret_cast<const uint4*>(x + (size_t)tok * x_ld + (size_t)h * x_head + k) : zero;
+            }
+        if (k0 > 0) load_w(k0);
+#pragma unroll
+        for (int i = 0; i < PH_K; ++i)
+#pragma unroll
+            for (int n = 0; n < NT; ++n) {
+                ph_mma(acc[n], a_lo[i].x, a_hi[i].x, a_lo[i].y, a_hi[i].y, b[n][i].x, b[n][i].y);
+                ph_mma(acc[n], a_lo[i].z, a_hi[i].z, a_lo[i].w, a_hi[i].w, b[n][i].z, b[n][i].w);
+            }
     }
 #pragma unroll
     for (int n = 0; n < NT; ++n)
@@ -284,8 +299,7 @@ per_head_rows_kernel(const __nv_bfloat16* __restrict__ x, int x_ld, int x_head, 
         for (int e = 0; e < 4; ++e) {
             const int tok = tok0 + 8 * n + 2 * t + (e & 1), j = e < 2 ? j_lo : j_hi;
             if (tok >= n_tokens || j >= J) continue;
-            float v = acc[n][e];
-            if (gate != nullptr) v /= 1.0f + expf(-__bfloat162float(gate[(size_t)tok * gate_ld + (size_t)h * J + j]));
+            const float v = gate != nullptr ? acc[n][e] / (1.0f + expf(-gv[n][e])) : acc[n][e];
             out[(size_t)tok * out_ld + (size_t)h * out_head + j] = __float2bfloat16_rn(v);
         }
     if (rot < 0 || blockIdx.x != 0) return;
@@ -311,7 +325,7 @@ extern "C" int dl_per_head_rows(const void* x, int x_ld, int x_head, const void*
     DL_REQUIRE(rot_dims >= 0 && rot_dims <= (rot > 0 ? rot : 0) && rot_dims % 2 == 0 && (rot_dims == 0 || (cos_t && sin_t && token_pos && table_rows > 0)),
                "per_head_rows: a rotation needs tables and positions");
     if (n_tokens == 0) return DL_OK;
-    const int nt = n_tokens <= 8 ? 1 : n_tokens <= 16 ? 2 : 4;
+    const int nt = n_tokens <= 8 ? 1 : 2;
     const dim3 grid((J + 16 * PH_WARPS - 1) / (16 * PH_WARPS), H, (n_tokens + 8 * nt - 1) / (8 * nt)), block(32 * PH_WARPS);
     cudaError_t e;
 #define PH_GO(NT)                                                                                                                          \
@@ -319,8 +333,7 @@ extern "C" int dl_per_head_rows(const void* x, int x_ld, int x_head, const void*
                             (const __nv_bfloat16*)w, J, K, (__nv_bfloat16*)out, out_ld, out_head, (const __nv_bfloat16*)gate, gate_ld, rot, \
                             rot_dims, cos_t, sin_t, table_rows, token_pos, n_tokens)
     if (nt == 1) PH_GO(1);
-    else if (nt == 2) PH_GO(2);
-    else PH_GO(4);
+    else PH_GO(2);
 #undef PH_GO
     if (e != cudaSuccess) return dl_fail(DL_ERR_LAUNCH, "per_head_rows: %s", cudaGetErrorString(e));
     return DL_OK;

@@ -248,12 +248,18 @@ __device__ __forceinline__ void sc_split(float v0, float v1, uint32_t (&p)[3]) {
     }
 }
 
-template <int NT>
+// Where the walk would leave most of the machine idle (one prompt), the chunks run side by side in three launches instead:
+// SC_STATES, every chunk's own contribution to the state, sum_j B_j (exp(c_L - c_j) dt_j x_j)^T, and its whole decay c_L, into
+// scratch; ssd_pass_kernel, the states before every chunk one after the other, elementwise, in place; SC_OUTPUTS, every chunk's
+// outputs from the state before it.  SC_WALK is the walk in one launch.
+enum { SC_WALK = 0, SC_STATES = 1, SC_OUTPUTS = 2 };
+
+template <int NT, int MODE>
 __global__ void __launch_bounds__(SC_THREADS)
 ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, int ld, const __nv_bfloat16* __restrict__ z, int z_ld, const float* __restrict__ dt_bias,
                  const float* __restrict__ a_log, const float* __restrict__ skip, const int32_t* __restrict__ cu_new,
                  const int32_t* __restrict__ slots, float* __restrict__ state, long slot_stride, int n_slots, float* __restrict__ y, int y_ld,
-                 int H, int G, int N, int P) {
+                 int H, int G, int N, int P, int n_chunks, float* __restrict__ part_state, float* __restrict__ part_decay) {
     constexpr int LDN = NT + 8, LDP = SC_P + 8;               // rows of shared memory, shifted so that ldmatrix misses its own banks
     constexpr int MT = (NT / 16 + SC_WARPS - 1) / SC_WARPS;   // row tiles of the state per warp
     extern __shared__ __align__(128) unsigned char sc_raw[];
@@ -264,14 +270,16 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, int ld, const __nv_bfloa
     __nv_bfloat16* sX = sS + 3 * NT * LDP;                                        // [3][SC_L][LDP]: x_j weighted for the new state
     __shared__ float s_cum[2][SC_L], s_dt[2][SC_L];           // running log2 decay up to and with the token, step size
     dl_launch_dependents();
-    const int b = blockIdx.z, h = blockIdx.y, g_ = h / (H / G);
+    const int b = MODE == SC_WALK ? blockIdx.z : blockIdx.z / n_chunks, h = blockIdx.y, g_ = h / (H / G);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
     const int col0 = blockIdx.x * SC_P;
     const float rate2 = expf(a_log[h]) * 1.4426950408889634f, bias = dt_bias[h], d_skip = skip[h];
     dl_grid_dependency_wait();
     const int t0 = cu_new[b], n = cu_new[b + 1] - t0;
     const int slot = slots[b];
-    if (slot < 0 || slot >= n_slots || n <= 0) return;        // uniform over the block
+    const int begin = MODE == SC_WALK ? 0 : (blockIdx.z % n_chunks) * SC_L;
+    const int end = MODE == SC_WALK ? n : min(n, begin + SC_L);
+    if (slot < 0 || slot >= n_slots || begin >= n) return;    // uniform over the block
     const __nv_bfloat16* x_in = xbc + (size_t)t0 * ld + (size_t)h * P + col0;
     const __nv_bfloat16* b_in = xbc + (size_t)t0 * ld + (size_t)H * P + (size_t)g_ * N;
     const __nv_bfloat16* c_in = b_in + (size_t)G * N;
@@ -281,7 +289,7 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, int ld, const __nv_bfloa
             const bool live = first + j < n && ch < N;
             const size_t at = live ? (size_t)(first + j) * ld + ch : 0;
             sc_copy16(sB + (size_t)(buf * SC_L + j) * LDN + ch, b_in + at, live);
-            sc_copy16(sC + (size_t)(buf * SC_L + j) * LDN + ch, c_in + at, live);
+            if (MODE != SC_STATES) sc_copy16(sC + (size_t)(buf * SC_L + j) * LDN + ch, c_in + at, live);
         }
         for (int e = tid; e < SC_L * (SC_P / 8); e += SC_THREADS) {
             const int j = e / (SC_P / 8), ch = (e - j * (SC_P / 8)) * 8;
@@ -311,10 +319,10 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, int ld, const __nv_bfloa
         s_dt[buf][2 * lane] = dt[0];
         s_dt[buf][2 * lane + 1] = dt[1];
     };
-    bring(0, 0);
-    if (warp == 0) scalars(0, 0);
+    bring(begin, 0);
+    if (warp == 0) scalars(begin, 0);
     // the state: this warp's row tiles, SC_P columns
-    float* S = state + (size_t)slot * slot_stride + (size_t)h * N * P;
+    float* S = MODE == SC_WALK ? state + (size_t)slot * slot_stride + (size_t)h * N * P : part_state + ((size_t)blockIdx.z * H + h) * N * P;
     float st[MT][SC_P / 8][4];
 #pragma unroll
     for (int i = 0; i < MT; ++i)
@@ -323,7 +331,7 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, int ld, const __nv_bfloa
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int row = (warp + SC_WARPS * i) * 16 + g + 8 * (e >> 1), col = col0 + c * 8 + 2 * t + (e & 1);
-                st[i][c][e] = row < N && col < P ? S[(size_t)row * P + col] : 0.f;
+                st[i][c][e] = MODE != SC_STATES && row < N && col < P ? S[(size_t)row * P + col] : 0.f;
             }
     auto put_state = [&]() {                                  // the three parts of this warp's rows into shared memory
 #pragma unroll
@@ -341,20 +349,20 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, int ld, const __nv_bfloa
                 }
         }
     };
-    put_state();
+    if (MODE != SC_STATES) put_state();
     // a lane's row and column of the 16 x 16 tile that ldmatrix reads (A as stored; B and the transposed forms share the pattern)
     const int lrow = lane & 15, lcol = (lane >> 4) * 8;
     int buf = 0;
-    for (int first = 0; first < n; first += SC_L, buf ^= 1) {
+    for (int first = begin; first < end; first += SC_L, buf ^= 1) {
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();                                      // the chunk, its scalars and the state's parts are there; the other buffer is free
-        if (first + SC_L < n) bring(first + SC_L, buf ^ 1);
+        if (first + SC_L < end) bring(first + SC_L, buf ^ 1);
         const __nv_bfloat16* cB = sB + (size_t)buf * SC_L * LDN;
         const __nv_bfloat16* cC = sC + (size_t)buf * SC_L * LDN;
         const __nv_bfloat16* cx = sx + (size_t)buf * SC_L * LDP;
         const float cum_l = s_cum[buf][SC_L - 1];
         // x weighted by what is left of its step at the chunk's end, in three parts
-        for (int e = tid; e < SC_L * SC_P / 2; e += SC_THREADS) {
+        for (int e = tid; MODE != SC_OUTPUTS && e < SC_L * SC_P / 2; e += SC_THREADS) {
             const int j = e / (SC_P / 2), c = (e - j * (SC_P / 2)) * 2;
             const float w = exp2f(cum_l - s_cum[buf][j]) * s_dt[buf][j];
             const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162*>(cx + (size_t)j * LDP + c);
@@ -363,6 +371,7 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, int ld, const __nv_bfloa
 #pragma unroll
             for (int q = 0; q < 3; ++q) *reinterpret_cast<uint32_t*>(sX + (size_t)(q * SC_L + j) * LDP + c) = part[q];
         }
+        if (MODE != SC_STATES) {
         // ---- the read-out of the state before the chunk: rows 16 warp .. of C against the state's parts
         float yo[SC_P / 8][4];
 #pragma unroll
@@ -438,6 +447,8 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, int ld, const __nv_bfloa
                         make_float2(fmaf(d_skip, __low2float(v), yo[c][2 * hf]), fmaf(d_skip, __high2float(v), yo[c][2 * hf + 1]));
                 }
             }
+        }
+        if (MODE == SC_OUTPUTS) return;
         __syncthreads();                                      // the weighted x is there; everyone is done with the state's parts
         // ---- the new state
         const float keep = exp2f(cum_l);
@@ -464,11 +475,12 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, int ld, const __nv_bfloa
                     }
             }
         }
-        if (first + SC_L < n) {
+        if (first + SC_L < end) {
             put_state();
             if (warp == 0) scalars(first + SC_L, buf ^ 1);
         }
     }
+    if (MODE == SC_STATES && tid == 0 && blockIdx.x == 0) part_decay[(size_t)blockIdx.z * H + h] = s_cum[0][SC_L - 1];
 #pragma unroll
     for (int i = 0; i < MT; ++i)
 #pragma unroll
@@ -480,36 +492,97 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, int ld, const __nv_bfloa
             }
 }
 
-template <int NT>
-static int ssd_chunk_launch(const void* xbc, int ld, const void* z, int z_ld, const float* dt_bias, const float* a_log, const float* skip,
-                            const int32_t* cu_new, const int32_t* slots, float* state, long slot_stride, int n_slots, float* y, int y_ld,
-                            int n_seqs, int H, int G, int N, int P, cudaStream_t s) {
+// The state before every chunk, in place of the chunk's contribution: four neighbouring values of one (sequence, head) a thread.
+__global__ void __launch_bounds__(256)
+ssd_pass_kernel(float* __restrict__ part_state, const float* __restrict__ part_decay, const int32_t* __restrict__ cu_new,
+                const int32_t* __restrict__ slots, float* __restrict__ state, long slot_stride, int n_slots, int H, int NP, int n_chunks) {
+    dl_launch_dependents();
+    dl_grid_dependency_wait();
+    const int b = blockIdx.z, h = blockIdx.y, at = (blockIdx.x * 256 + threadIdx.x) * 4;
+    const int n = cu_new[b + 1] - cu_new[b], slot = slots[b];
+    if (at >= NP || n <= 0 || slot < 0 || slot >= n_slots) return;
+    const int chunks = (n + SC_L - 1) / SC_L;
+    float4* S = reinterpret_cast<float4*>(state + (size_t)slot * slot_stride + (size_t)h * NP + at);
+    float4 s = *S;
+    float* p = part_state + ((size_t)b * n_chunks * H + h) * NP + at;
+    const float* d = part_decay + (size_t)b * n_chunks * H + h;
+    const size_t step = (size_t)H * NP;
+    constexpr int AHEAD = 8;                                 // chunks whose contributions are asked for together
+    for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
+        float4 v[AHEAD];
+        float k[AHEAD];
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i) {
+            const int c = min(c0 + i, chunks - 1);
+            v[i] = *reinterpret_cast<const float4*>(p + (size_t)c * step);
+            k[i] = d[(size_t)c * H];
+        }
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i) {
+            if (c0 + i >= chunks) break;
+            *reinterpret_cast<float4*>(p + (size_t)(c0 + i) * step) = s;
+            const float keep = exp2f(k[i]);
+            s = make_float4(fmaf(keep, s.x, v[i].x), fmaf(keep, s.y, v[i].y), fmaf(keep, s.z, v[i].z), fmaf(keep, s.w, v[i].w));
+        }
+    }
+    *S = s;
+}
+
+template <int NT, int MODE>
+static cudaError_t ssd_chunk_go(dim3 grid, const void* xbc, int ld, const void* z, int z_ld, const float* dt_bias, const float* a_log,
+                                const float* skip, const int32_t* cu_new, const int32_t* slots, float* state, long slot_stride, int n_slots,
+                                float* y, int y_ld, int H, int G, int N, int P, int n_chunks, float* part_state, float* part_decay,
+                                cudaStream_t s) {
     const size_t smem = (size_t)(4 * SC_L * (NT + 8) + 2 * SC_L * (SC_P + 8) + 3 * NT * (SC_P + 8) + 3 * SC_L * (SC_P + 8)) * 2;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(ssd_chunk_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        if (e != cudaSuccess) return dl_fail(DL_ERR_LAUNCH, "ssd_chunk: shared memory %zu: %s", smem, cudaGetErrorString(e));
+        cudaError_t e = cudaFuncSetAttribute(ssd_chunk_kernel<NT, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return e;
         configured = true;
     }
-    const dim3 grid((P + SC_P - 1) / SC_P, H, n_seqs), block(SC_THREADS);
     const bool early = (long)grid.x * grid.y * grid.z > 2L * dl_sm_count();
-    cudaError_t e = dl_launch_dependent_if(early, ssd_chunk_kernel<NT>, grid, block, smem, s, (const __nv_bfloat16*)xbc, ld, (const __nv_bfloat16*)z,
-                                           z_ld, dt_bias, a_log, skip, cu_new, slots, state, slot_stride, n_slots, y, y_ld, H, G, N, P);
+    return dl_launch_dependent_if(early, ssd_chunk_kernel<NT, MODE>, grid, dim3(SC_THREADS), smem, s, (const __nv_bfloat16*)xbc, ld,
+                                  (const __nv_bfloat16*)z, z_ld, dt_bias, a_log, skip, cu_new, slots, state, slot_stride, n_slots, y, y_ld, H, G, N, P,
+                                  n_chunks, part_state, part_decay);
+}
+
+template <int NT>
+static int ssd_chunk_launch(const void* xbc, int ld, const void* z, int z_ld, const float* dt_bias, const float* a_log, const float* skip,
+                            const int32_t* cu_new, const int32_t* slots, float* state, long slot_stride, int n_slots, float* y, int y_ld,
+                            int n_seqs, int H, int G, int N, int P, int n_chunks, float* part_state, float* part_decay, cudaStream_t s) {
+    const dim3 walk((P + SC_P - 1) / SC_P, H, n_seqs), side(walk.x, H, n_seqs * n_chunks);
+    cudaError_t e;
+#define SC_ARGS xbc, ld, z, z_ld, dt_bias, a_log, skip, cu_new, slots, state, slot_stride, n_slots, y, y_ld, H, G, N, P, n_chunks, part_state, part_decay, s
+    if (part_state == nullptr) {
+        e = ssd_chunk_go<NT, SC_WALK>(walk, SC_ARGS);
+    } else {
+        e = ssd_chunk_go<NT, SC_STATES>(side, SC_ARGS);
+        if (e == cudaSuccess)
+            e = dl_launch_dependent(ssd_pass_kernel, dim3((N * P / 4 + 255) / 256, H, n_seqs), dim3(256), 0, s, part_state, (const float*)part_decay,
+                                    cu_new, slots, state, slot_stride, n_slots, H, N * P, n_chunks);
+        if (e == cudaSuccess) e = ssd_chunk_go<NT, SC_OUTPUTS>(side, SC_ARGS);
+    }
+#undef SC_ARGS
     if (e != cudaSuccess) return dl_fail(DL_ERR_LAUNCH, "ssd_chunk: %s", cudaGetErrorString(e));
     return DL_OK;
 }
 
 // As dl_ssd_scan, a chunk at a time on the tensor cores: xbc and z bfloat16, rows and their parts 16-byte aligned (ld, N and P
-// multiples of 8), N up to SC_MAX_STATE.
+// multiples of 8), N up to SC_MAX_STATE.  part_state float32 [n_seqs * n_chunks, H, N, P] and part_decay float32 [n_seqs * n_chunks, H]
+// (n_chunks: SC_L-token chunks of the longest sequence): the chunks run side by side; both NULL: a block walks its sequence's chunks.
 extern "C" int dl_ssd_chunk(const void* xbc, int ld, const void* z, int z_ld, const float* dt_bias, const float* a_log, const float* skip,
                             const int32_t* cu_new, const int32_t* slots, float* state, long slot_stride, int n_slots, float* y, int y_ld,
-                            int n_seqs, int H, int G, int N, int P, void* stream) {
+                            int n_seqs, int H, int G, int N, int P, int n_chunks, float* part_state, float* part_decay, void* stream) {
     DL_REQUIRE(n_seqs >= 0 && H > 0 && G > 0 && N > 0 && P > 0 && n_slots > 0 && H % G == 0 && H <= 65535 && n_seqs <= 65535, "ssd_chunk: bad sizes");
+    DL_REQUIRE((part_state == nullptr) == (part_decay == nullptr) &&
+                   (part_state == nullptr || (n_chunks >= 1 && (long)n_seqs * n_chunks <= 65535 && slot_stride % 4 == 0 && ((uintptr_t)state % 16) == 0 &&
+                                              ((uintptr_t)part_state % 16) == 0)),
+               "ssd_chunk: chunks side by side need scratch for at most 65,535 of them and aligned states");
     DL_REQUIRE(N % 8 == 0 && P % 8 == 0 && ld % 8 == 0 && ((uintptr_t)xbc % 16) == 0 && N <= SC_MAX_STATE && y_ld % 2 == 0 && ((uintptr_t)y % 8) == 0,
                "ssd_chunk: state and value channels come in aligned eights, the state up to %d", SC_MAX_STATE);
     DL_REQUIRE(ld >= H * P + 2 * G * N && z_ld >= H && y_ld >= H * P && slot_stride >= (long)H * N * P, "ssd_chunk: rows overlap");
     if (n_seqs == 0) return DL_OK;
-#define SC_GO(NT) return ssd_chunk_launch<NT>(xbc, ld, z, z_ld, dt_bias, a_log, skip, cu_new, slots, state, slot_stride, n_slots, y, y_ld, n_seqs, H, G, N, P, (cudaStream_t)stream)
+#define SC_GO(NT) return ssd_chunk_launch<NT>(xbc, ld, z, z_ld, dt_bias, a_log, skip, cu_new, slots, state, slot_stride, n_slots, y, y_ld, n_seqs, H, G, N, P, n_chunks, part_state, part_decay, (cudaStream_t)stream)
     if (N <= 32) SC_GO(32);
     if (N <= 64) SC_GO(64);
     if (N <= 128) SC_GO(128);

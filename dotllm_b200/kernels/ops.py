@@ -28,7 +28,7 @@ _library.register_signatures({
     "dl_post_norm": [_P, _P, _I, _I, _F, _P, _I, _F, _P, _I, _F, _P, _I, _I, _I, _P, ctypes.c_long, _I, _P, _P, _I, _P],
     "dl_causal_conv": [_P, _I, _I, _P, _I, _P, _I, _I, _P, ctypes.c_long, _I, _P, _P, _P, _I, _I, _I, _I, _I, _P],
     "dl_ssd_scan": [_P, _I, _I, _P, _I, _P, _P, _P, _P, _P, _P, ctypes.c_long, _I, _P, _I, _I, _I, _I, _I, _I, _I, _P],
-    "dl_ssd_chunk": [_P, _I, _P, _I, _P, _P, _P, _P, _P, _P, ctypes.c_long, _I, _P, _I, _I, _I, _I, _I, _I, _P],
+    "dl_ssd_chunk": [_P, _I, _P, _I, _P, _P, _P, _P, _P, _P, ctypes.c_long, _I, _P, _I, _I, _I, _I, _I, _I, _I, _P, _P, _P],
     "dl_gated_group_norm": [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _F, _P],
     "dl_latent_rows": [_P, _I, _I, _I, _I, _I, _I, _P, _P, _F, _P, _P, _I, _P, _P, _P, _I, _I, _P],
     "dl_latent_query_tail": [_P, _I, _I, _I, _I, _I, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P],
@@ -789,6 +789,9 @@ def head_rmsnorm(x, gain_a, heads_a, dim, eps, gain_b=None, heads_b=0, lay=None)
 SSD_CHUNKED = True              # False: always the token-by-token scan (tests compare the two)
 SSD_CHUNK_MIN_TOKENS = 12       # steps whose longest sequence brings fewer tokens walk them one by one
 SSD_CHUNK_MAX_STATE = 256       # SC_MAX_STATE in csrc/ssd.cu
+SSD_CHUNK, SSD_CHUNK_COLS = 64, 32      # SC_L, SC_P in csrc/ssd.cu
+SSD_SIDE_BLOCKS = 592           # a walk of at least this many blocks fills the machine by itself: its chunks need not run side by side
+SSD_SIDE_BYTES = 512 << 20      # most scratch that chunks side by side may take
 
 
 def ssd_scan(xbc, z, dt_bias, a_log, skip, cu_new, slots, memory, n_heads, groups, state, vdim, max_new=1):
@@ -812,8 +815,14 @@ def ssd_scan(xbc, z, dt_bias, a_log, skip, cu_new, slots, memory, n_heads, group
     ld, zld = _rows_view(xbc, "ssd_scan xbc"), _rows_view(z, "ssd_scan z")
     if SSD_CHUNKED and xbc.dtype == torch.bfloat16 and max_new >= SSD_CHUNK_MIN_TOKENS and N % 8 == 0 and P % 8 == 0 and N <= SSD_CHUNK_MAX_STATE \
             and ld % 8 == 0 and xbc.data_ptr() % 16 == 0:
+        B, chunks = slots.numel(), (int(max_new) + SSD_CHUNK - 1) // SSD_CHUNK
+        part = decay = None
+        if chunks > 1 and B * H * ((P + SSD_CHUNK_COLS - 1) // SSD_CHUNK_COLS) < SSD_SIDE_BLOCKS and B * chunks <= 65535 \
+                and B * chunks * H * N * P * 4 <= SSD_SIDE_BYTES and memory.stride(0) % 4 == 0 and memory.data_ptr() % 16 == 0:
+            part = torch.empty((B * chunks, H, N, P), dtype=torch.float32, device=xbc.device)
+            decay = torch.empty((B * chunks, H), dtype=torch.float32, device=xbc.device)
         _library.call("dl_ssd_chunk", _ptr(xbc), ld, _ptr(z), zld, _ptr(dt_bias), _ptr(a_log), _ptr(skip), _ptr(cu_new), _ptr(slots), _ptr(memory),
-                      memory.stride(0), memory.shape[0], _ptr(out), out.stride(0), slots.numel(), H, G, N, P, _stream())
+                      memory.stride(0), memory.shape[0], _ptr(out), out.stride(0), B, H, G, N, P, chunks, _ptr(part), _ptr(decay), _stream())
         return out
     _library.call("dl_ssd_scan", _ptr(xbc), _code(xbc.dtype), ld, _ptr(z), zld,
                   _ptr(dt_bias), _ptr(a_log), _ptr(skip), _ptr(cu_new), _ptr(slots), _ptr(memory), memory.stride(0), memory.shape[0],

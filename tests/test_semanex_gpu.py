@@ -141,13 +141,14 @@ def test_causal_convolution_alone(C, K, dtype):
         close(memory, rmem, torch.float32)
 
 
-@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("dtype,side", [(torch.float32, 0), (torch.bfloat16, 592), (torch.bfloat16, 0)])
 @pytest.mark.parametrize("H,G,N,P", [(4, 2, 40, 48), (2, 1, 16, 8), (3, 1, 256, 40), (2, 2, 128, 128), (3, 3, 1, 5), (6, 1, 19, 7), (8, 2, 128, 64), (2, 1, 64, 24), (2, 2, 200, 10), (1, 1, 400, 9),
                                      (5, 5, 32, 33)])
-def test_state_space_scan_alone(H, G, N, P, dtype):
+def test_state_space_scan_alone(monkeypatch, H, G, N, P, dtype, side):
     """Unequal prompts, then portions and single tokens from the states they left, in slots that are not neighbours; the step
     logits span decays from almost one to almost nothing.  bfloat16 prompts go a chunk at a time through the tensor cores where
-    the sizes allow, and give the scan's float32 results."""
+    the sizes allow - the chunks side by side in three launches, or walked in one - and give the scan's float32 results."""
+    monkeypatch.setattr(ops, "SSD_SIDE_BLOCKS", side)
     bias, a_log, skip = g32(H, seed=1), g32(H, seed=2, scale=0.7), g32(H, seed=3)
     memory = torch.zeros((6, H * N * P + 12), dtype=torch.float32, device=DEV)
     rmem = memory.cpu().clone()
