@@ -145,7 +145,7 @@ struct AdCut {
     int total, share;        // pages in the step, pages per block
 };
 
-__device__ __forceinline__ AdCut ad_cut(const int32_t* seq_len, int n_seqs, int nkv, AdWin window, int n_blocks, int lane) {
+__device__ __forceinline__ AdCut ad_cut(const int32_t* seq_len, int n_seqs, int nkv, AdWin window, int n_blocks, int min_share, int lane) {
     int sum = 0;
     for (int b0 = 0; b0 < n_seqs; b0 += 32)
         if (b0 + lane < n_seqs) sum += ad_pages_of(seq_len[b0 + lane], window);
@@ -153,7 +153,7 @@ __device__ __forceinline__ AdCut ad_cut(const int32_t* seq_len, int n_seqs, int 
     for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
     AdCut c;
     c.total = sum * nkv;
-    c.share = max(1, (c.total + n_blocks - 1) / n_blocks);
+    c.share = max(min_share, (c.total + n_blocks - 1) / n_blocks);
     return c;
 }
 
@@ -422,6 +422,9 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int g = lane >> 2, t = lane & 3;
     const AdWin window = {window_size, window_size > 0 ? fresh.keep_first : 0};
+    // A page is one warp's work: a share of fewer pages than the block has warps takes no less time, and a group of many heads is
+    // merged from more segments, which does take time.
+    const int min_share = WIDE ? n_stages : 1;
     const int pkv = fresh.pool_heads, per_pool = nkv / pkv;      // heads of the pages, heads of the launch that share one
     // The kernel checks its own shared-memory layout: if the launch gave it less dynamic shared
     // memory than the stages and merge buffers need, it records status 11 and touches nothing.
@@ -457,7 +460,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_
         int n = 0;                                           // pages issued so far, over all runs
         bool stop = false, waited = false;
         const uint64_t policy = ad_stream_policy();
-        const AdCut cut = ad_cut(seq_len, n_seqs, nkv, window, gridDim.x, lane);
+        const AdCut cut = ad_cut(seq_len, n_seqs, nkv, window, gridDim.x, min_share, lane);
         AdWalk walk = ad_walk_begin(cut, seq_len, n_seqs, nkv, window, blockIdx.x, lane);
         AdSeg w;
         while (!stop && ad_walk_next(walk, w, seq_len, n_seqs, nkv, window)) {
@@ -509,7 +512,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_
         const bool capped = fresh.cap.post > 0.f;
         const float scale2 = capped ? 1.f : scale * 1.4426950408889634f;    // scores in units of log2 (capped ones come in them)
         int n0 = 0;                                          // pages of the runs before this one
-        const AdCut cut = ad_cut(seq_len, n_seqs, nkv, window, gridDim.x, lane);
+        const AdCut cut = ad_cut(seq_len, n_seqs, nkv, window, gridDim.x, min_share, lane);
         AdWalk walk = ad_walk_begin(cut, seq_len, n_seqs, nkv, window, blockIdx.x, lane);
         AdSeg w;
         dl_grid_dependency_wait();       // q comes from the kernel before this one; out and the scratch may be in use by it
@@ -716,7 +719,7 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_
 #pragma unroll
                         for (int j = 0; j < 4; ++j)
 #pragma unroll
-                            for (int e = 0; e < (WIDE ? 4 : 2); ++e) sc[h][j][e] = dl_capped_score(sc[h][j][e], fresh.cap);
+                            for (int e = 0; e < (WIDE ? 4 : 2); e += 2) dl_cap_scores(sc[h][j][e], sc[h][j][e + 1], fresh.cap);
                 }
                 // ---- mask (ragged pages only; lane holds keys base + 32h + 8t + 2j + {0,1}) and row maximum
                 if (ragged) {

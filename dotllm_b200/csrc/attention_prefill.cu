@@ -232,7 +232,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
 #pragma unroll
                         for (int j = 0; j < 4; ++j)
 #pragma unroll
-                            for (int e = 0; e < 4; ++e) sc[hh][j][e] = dl_capped_score(sc[hh][j][e], cap);
+                            for (int e = 0; e < 4; e += 2) dl_cap_scores(sc[hh][j][e], sc[hh][j][e + 1], cap);
                 }
                 if (ragged) {
                     // lane holds keys base + 32hh + 8t + 2j + {0,1} of rows g (lo) and g+8 (hi).  Masked

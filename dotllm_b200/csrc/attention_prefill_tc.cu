@@ -338,7 +338,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
 
             if (CAP) {                                          // before the mask: a hidden key's score is replaced, not capped
 #pragma unroll
-                for (int i = 0; i < 64; ++i) sc[i] = dl_capped_score(sc[i], cap);
+                for (int i = 0; i < 64; i += 2) dl_cap_scores(sc[i], sc[i + 1], cap);
             }
             const int key0 = page_of(j) * DL_PAGE;
             // pages wholly visible to every row of the tile need no mask

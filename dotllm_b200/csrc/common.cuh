@@ -111,11 +111,18 @@ static inline DlScoreCap dl_score_cap(float softcap, float scale) {
     if (softcap > 0.f) c.pre = 2.f * 1.4426950408889634f * scale / softcap, c.post = softcap * 1.4426950408889634f;
     return c;
 }
-__device__ __forceinline__ float dl_capped_score(float raw, DlScoreCap cap) {
-    float e, r;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(raw * cap.pre));
-    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(e + 1.f));
-    return fmaf(-2.f * cap.post, r, cap.post);
+// Two scores in place, with one reciprocal between them.  The argument is held to where tanh is 1 in float32 anyway, so that the
+// product of the two denominators stays finite; a score that is no number (a key that was never written; the mask comes after
+// this) becomes the cap and leaves its neighbour alone.
+__device__ __forceinline__ void dl_cap_scores(float& a, float& b, DlScoreCap cap) {
+    float ea, eb, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(ea) : "f"(fminf(a * cap.pre, 62.f)));
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(eb) : "f"(fminf(b * cap.pre, 62.f)));
+    ea += 1.f;
+    eb += 1.f;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(ea * eb));
+    a = fmaf(-2.f * cap.post, r * eb, cap.post);
+    b = fmaf(-2.f * cap.post, r * ea, cap.post);
 }
 
 // Sum over a block of up to 1024 threads; every thread gets the result.  The order of

@@ -97,6 +97,63 @@ latent_rows_kernel(const T* __restrict__ x, int ld, int q_rank, int kv_rank, int
     }
 }
 
+// The same with a warp per (token, latent) and no block barrier: latents of up to 32 lanes x NP pieces of 16 bytes, aligned.
+template <typename T, int NP>
+__global__ void __launch_bounds__(LT_THREADS)
+latent_rows_warp_kernel(const T* __restrict__ x, int ld, int q_rank, int kv_rank, int rot, int rot_dims, const float* __restrict__ q_gain,
+                        const float* __restrict__ kv_gain, float eps, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
+                        int table_rows, const int32_t* __restrict__ token_pos, T* __restrict__ q_out, T* __restrict__ kv_out, int lay, int n_tokens) {
+    constexpr int V = 16 / (int)sizeof(T);
+    dl_launch_dependents();
+    const int lane = threadIdx.x & 31, which = blockIdx.y;   // 0: the key/value latent and what lies behind it, 1: the query latent
+    const int t = blockIdx.x * (LT_THREADS / 32) + (threadIdx.x >> 5);
+    if (t >= n_tokens) return;
+    const int rank = which ? q_rank : kv_rank;
+    const float* gain = which ? q_gain : kv_gain;
+    float gg[NP <= 4 ? NP * V : 1];
+    if (NP <= 4) {                                           // weights: no kernel of the stream writes them
+#pragma unroll
+        for (int i = 0; i < NP; ++i)
+#pragma unroll
+            for (int e = 0; e < V; e += 4) {
+                const int c = (lane + 32 * i) * V + e;
+                const float4 w = c < rank ? *reinterpret_cast<const float4*>(gain + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+                gg[(i * V + e) % (NP * V)] = w.x, gg[(i * V + e + 1) % (NP * V)] = w.y, gg[(i * V + e + 2) % (NP * V)] = w.z, gg[(i * V + e + 3) % (NP * V)] = w.w;
+            }
+    }
+    dl_grid_dependency_wait();
+    const T* src = x + (size_t)t * ld + (which ? 0 : q_rank);
+    T* dst = which ? q_out + (size_t)t * q_rank : kv_out + (size_t)t * lay;
+    uint4 raw[NP];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+        const int c = (lane + 32 * i) * V;
+        raw[i] = c < rank ? *reinterpret_cast<const uint4*>(src + c) : make_uint4(0u, 0u, 0u, 0u);
+    }
+    if (which == 0) {                                        // the part behind the latent: it waits for no sum
+        const int pos = rot_dims > 0 ? min(token_pos[t], table_rows - 1) : 0;    // host-validated
+        for (int c = lane; c < lay - kv_rank; c += 32)
+            dst[kv_rank + c] = dl_from_f32<T>(lt_tail<T>(src + kv_rank, c, rot, rot_dims, cos_t, sin_t, pos));
+    }
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+        const T* v = reinterpret_cast<const T*>(&raw[i]);
+#pragma unroll
+        for (int e = 0; e < V; ++e) { const float f = dl_to_f32<T>(v[e]); ss += f * f; }
+    }
+    const float r = 1.0f / sqrtf(dl_warp_sum(ss) / (float)rank + eps);
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+        const int c = (lane + 32 * i) * V;
+        if (c >= rank) continue;
+        T* v = reinterpret_cast<T*>(&raw[i]);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[e] = dl_from_f32<T>(dl_to_f32<T>(v[e]) * r * (NP <= 4 ? gg[(i * V + e) % (NP <= 4 ? NP * V : 1)] : gain[c + e]));
+        *reinterpret_cast<uint4*>(dst + c) = raw[i];
+    }
+}
+
 // x [tokens, q_rank + kv_rank + rot] of dtype (rows ld apart; q_rank 0: no query latent); gains float32; cos, sin float32
 // [table_rows, rot_dims / 2]; q_out [tokens, q_rank], kv_out [tokens, lay] contiguous of dtype, lay >= kv_rank + rot.
 extern "C" int dl_latent_rows(const void* x, int dtype, int ld, int q_rank, int kv_rank, int rot, int rot_dims, const float* q_gain,
@@ -105,6 +162,7 @@ extern "C" int dl_latent_rows(const void* x, int dtype, int ld, int q_rank, int 
     DL_REQUIRE(n_tokens >= 0 && q_rank >= 0 && kv_rank > 0 && rot >= 0 && rot_dims >= 0 && rot_dims <= rot && rot_dims % 2 == 0 && eps > 0.f,
                "latent_rows: bad sizes");
     DL_REQUIRE(ld >= q_rank + kv_rank + rot && lay >= kv_rank + rot, "latent_rows: rows too short");
+    DL_REQUIRE(dtype == DL_F32 || dtype == DL_BF16, "latent_rows: dtype %d", dtype);
     DL_REQUIRE(kv_gain && kv_out && (q_rank == 0 || (q_gain && q_out)) && (rot_dims == 0 || (cos_t && sin_t && token_pos && table_rows > 0)),
                "latent_rows: a tensor is missing");
     if (n_tokens == 0) return DL_OK;
@@ -113,6 +171,18 @@ extern "C" int dl_latent_rows(const void* x, int dtype, int ld, int q_rank, int 
     const bool vec = q_rank % v == 0 && kv_rank % v == 0 && ld % v == 0 && lay % v == 0 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)kv_out % 16) == 0 &&
                      ((uintptr_t)q_out % 16) == 0;
     cudaError_t e;
+    const int longest = q_rank > kv_rank ? q_rank : kv_rank;
+    if (vec && longest <= 32 * 8 * v && ((uintptr_t)q_gain % 16) == 0 && ((uintptr_t)kv_gain % 16) == 0) {
+        const dim3 wgrid((n_tokens + LT_THREADS / 32 - 1) / (LT_THREADS / 32), grid.y);
+#define LW_GO(T, NP)                                                                                                                       \
+    e = dl_launch_dependent(latent_rows_warp_kernel<T, NP>, wgrid, block, 0, (cudaStream_t)stream, (const T*)x, ld, q_rank, kv_rank, rot,    \
+                            rot_dims, q_gain, kv_gain, eps, cos_t, sin_t, table_rows, token_pos, (T*)q_out, (T*)kv_out, lay, n_tokens)
+        if (dtype == DL_F32) { if (longest <= 32 * 4 * v) LW_GO(float, 4); else LW_GO(float, 8); }
+        else { if (longest <= 32 * 4 * v) LW_GO(__nv_bfloat16, 4); else LW_GO(__nv_bfloat16, 8); }
+#undef LW_GO
+        if (e != cudaSuccess) return dl_fail(DL_ERR_LAUNCH, "latent_rows: %s", cudaGetErrorString(e));
+        return DL_OK;
+    }
 #define LR_GO(T, VEC)                                                                                                                    \
     e = dl_launch_dependent(latent_rows_kernel<T, VEC>, grid, block, 0, (cudaStream_t)stream, (const T*)x, ld, q_rank, kv_rank, rot, rot_dims, \
                             q_gain, kv_gain, eps, cos_t, sin_t, table_rows, token_pos, (T*)q_out, (T*)kv_out, lay)
@@ -251,6 +321,17 @@ per_head_rows_kernel(const __nv_bfloat16* __restrict__ x, int x_ld, int x_head, 
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
     const int h = blockIdx.y, tok0 = blockIdx.z * 8 * NT;
     const int j_lo = (blockIdx.x * PH_WARPS + warp) * 16 + g, j_hi = j_lo + 8;
+    if (rot >= 0 && blockIdx.x == gridDim.x - 1) {           // a block of its own for what stands behind the J channels
+        dl_grid_dependency_wait();
+        const int tail = out_head - J, mine = min(8 * NT, n_tokens - tok0);
+        for (int e = threadIdx.x; e < mine * tail; e += 32 * PH_WARPS) {
+            const int tok = tok0 + e / tail, c = e % tail;
+            const int pos = rot_dims > 0 ? min(token_pos[tok], table_rows - 1) : 0;       // host-validated
+            out[(size_t)tok * out_ld + (size_t)h * out_head + J + c] = __float2bfloat16_rn(
+                lt_tail<__nv_bfloat16>(x + (size_t)tok * x_ld + (size_t)h * x_head + K, c, rot, rot_dims, cos_t, sin_t, pos));
+        }
+        return;
+    }
     const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
     const __nv_bfloat16* w_lo = w + ((size_t)h * J + j_lo) * K + 8 * t;
     const __nv_bfloat16* w_hi = w_lo + (size_t)8 * K;
@@ -302,14 +383,6 @@ per_head_rows_kernel(const __nv_bfloat16* __restrict__ x, int x_ld, int x_head, 
             const float v = gate != nullptr ? acc[n][e] / (1.0f + expf(-gv[n][e])) : acc[n][e];
             out[(size_t)tok * out_ld + (size_t)h * out_head + j] = __float2bfloat16_rn(v);
         }
-    if (rot < 0 || blockIdx.x != 0) return;
-    const int tail = out_head - J, mine = min(8 * NT, n_tokens - tok0);
-    for (int e = threadIdx.x; e < mine * tail; e += 32 * PH_WARPS) {
-        const int tok = tok0 + e / tail, c = e % tail;
-        const int pos = rot_dims > 0 ? min(token_pos[tok], table_rows - 1) : 0;
-        out[(size_t)tok * out_ld + (size_t)h * out_head + J + c] = __float2bfloat16_rn(
-            lt_tail<__nv_bfloat16>(x + (size_t)tok * x_ld + (size_t)h * x_head + K, c, rot, rot_dims, cos_t, sin_t, pos));
-    }
 }
 
 // x bf16 [tokens, H * x_head] (rows x_ld apart), w bf16 [H, J, K], out bf16 [tokens, H * out_head] (rows out_ld apart); K, x_ld and
@@ -326,7 +399,7 @@ extern "C" int dl_per_head_rows(const void* x, int x_ld, int x_head, const void*
                "per_head_rows: a rotation needs tables and positions");
     if (n_tokens == 0) return DL_OK;
     const int nt = n_tokens <= 8 ? 1 : 2;
-    const dim3 grid((J + 16 * PH_WARPS - 1) / (16 * PH_WARPS), H, (n_tokens + 8 * nt - 1) / (8 * nt)), block(32 * PH_WARPS);
+    const dim3 grid((J + 16 * PH_WARPS - 1) / (16 * PH_WARPS) + (rot >= 0 ? 1 : 0), H, (n_tokens + 8 * nt - 1) / (8 * nt)), block(32 * PH_WARPS);
     cudaError_t e;
 #define PH_GO(NT)                                                                                                                          \
     e = dl_launch_dependent(per_head_rows_kernel<NT>, grid, block, 0, (cudaStream_t)stream, (const __nv_bfloat16*)x, x_ld, x_head,         \

@@ -790,7 +790,7 @@ SSD_CHUNKED = True              # False: always the token-by-token scan (tests c
 SSD_CHUNK_MIN_TOKENS = 12       # steps whose longest sequence brings fewer tokens walk them one by one
 SSD_CHUNK_MAX_STATE = 256       # SC_MAX_STATE in csrc/ssd.cu
 SSD_CHUNK, SSD_CHUNK_COLS = 64, 32      # SC_L, SC_P in csrc/ssd.cu
-SSD_SIDE_BLOCKS = 592           # a walk of at least this many blocks fills the machine by itself: its chunks need not run side by side
+SSD_SIDE_BLOCKS = 112           # a walk of at least this many blocks fills most of the machine by itself: its chunks need not run side by side
 SSD_SIDE_BYTES = 512 << 20      # most scratch that chunks side by side may take
 
 
