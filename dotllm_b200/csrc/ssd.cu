@@ -263,11 +263,12 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, int ld, const __nv_bfloa
     constexpr int LDN = NT + 8, LDP = SC_P + 8;               // rows of shared memory, shifted so that ldmatrix misses its own banks
     constexpr int MT = (NT / 16 + SC_WARPS - 1) / SC_WARPS;   // row tiles of the state per warp
     extern __shared__ __align__(128) unsigned char sc_raw[];
-    __nv_bfloat16* sB = reinterpret_cast<__nv_bfloat16*>(sc_raw);                 // [2][SC_L][LDN]
-    __nv_bfloat16* sC = sB + 2 * SC_L * LDN;                                      // [2][SC_L][LDN]
-    __nv_bfloat16* sx = sC + 2 * SC_L * LDN;                                      // [2][SC_L][LDP]
-    __nv_bfloat16* sS = sx + 2 * SC_L * LDP;                                      // [3][NT][LDP]: the state before the chunk
-    __nv_bfloat16* sX = sS + 3 * NT * LDP;                                        // [3][SC_L][LDP]: x_j weighted for the new state
+    constexpr int BUFS = MODE == SC_WALK ? 2 : 1;             // a walk brings the next chunk while it works on one
+    __nv_bfloat16* sB = reinterpret_cast<__nv_bfloat16*>(sc_raw);                 // [BUFS][SC_L][LDN]
+    __nv_bfloat16* sC = sB + BUFS * SC_L * LDN;                                   // [BUFS][SC_L][LDN] (not where only states are made)
+    __nv_bfloat16* sx = sC + (MODE == SC_STATES ? 0 : BUFS * SC_L * LDN);         // [BUFS][SC_L][LDP]
+    __nv_bfloat16* sS = sx + BUFS * SC_L * LDP;                                   // [3][NT][LDP]: the state before the chunk (likewise)
+    __nv_bfloat16* sX = sS + (MODE == SC_STATES ? 0 : 3 * NT * LDP);              // [3][SC_L][LDP]: x_j weighted for the new state (not for outputs)
     __shared__ float s_cum[2][SC_L], s_dt[2][SC_L];           // running log2 decay up to and with the token, step size
     dl_launch_dependents();
     const int b = MODE == SC_WALK ? blockIdx.z : blockIdx.z / n_chunks, h = blockIdx.y, g_ = h / (H / G);
@@ -533,7 +534,9 @@ static cudaError_t ssd_chunk_go(dim3 grid, const void* xbc, int ld, const void* 
                                 const float* skip, const int32_t* cu_new, const int32_t* slots, float* state, long slot_stride, int n_slots,
                                 float* y, int y_ld, int H, int G, int N, int P, int n_chunks, float* part_state, float* part_decay,
                                 cudaStream_t s) {
-    const size_t smem = (size_t)(4 * SC_L * (NT + 8) + 2 * SC_L * (SC_P + 8) + 3 * NT * (SC_P + 8) + 3 * SC_L * (SC_P + 8)) * 2;
+    constexpr int bufs = MODE == SC_WALK ? 2 : 1;
+    const size_t smem = (size_t)(bufs * SC_L * ((MODE == SC_STATES ? 1 : 2) * (NT + 8) + SC_P + 8) + (MODE == SC_STATES ? 0 : 3 * NT * (SC_P + 8)) +
+                                 (MODE == SC_OUTPUTS ? 0 : 3 * SC_L * (SC_P + 8))) * 2;
     static bool configured = false;
     if (!configured) {
         cudaError_t e = cudaFuncSetAttribute(ssd_chunk_kernel<NT, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);

@@ -790,7 +790,7 @@ SSD_CHUNKED = True              # False: always the token-by-token scan (tests c
 SSD_CHUNK_MIN_TOKENS = 12       # steps whose longest sequence brings fewer tokens walk them one by one
 SSD_CHUNK_MAX_STATE = 256       # SC_MAX_STATE in csrc/ssd.cu
 SSD_CHUNK, SSD_CHUNK_COLS = 64, 32      # SC_L, SC_P in csrc/ssd.cu
-SSD_SIDE_BLOCKS = 112           # a walk of at least this many blocks fills most of the machine by itself: its chunks need not run side by side
+SSD_SIDE_BLOCKS = 296           # a walk of at least this many blocks fills the machine by itself: its chunks need not run side by side
 SSD_SIDE_BYTES = 512 << 20      # most scratch that chunks side by side may take
 
 
@@ -817,7 +817,7 @@ def ssd_scan(xbc, z, dt_bias, a_log, skip, cu_new, slots, memory, n_heads, group
             and ld % 8 == 0 and xbc.data_ptr() % 16 == 0:
         B, chunks = slots.numel(), (int(max_new) + SSD_CHUNK - 1) // SSD_CHUNK
         part = decay = None
-        if chunks > 1 and B * H * ((P + SSD_CHUNK_COLS - 1) // SSD_CHUNK_COLS) < SSD_SIDE_BLOCKS and B * chunks <= 65535 \
+        if chunks > 2 and B * H * ((P + SSD_CHUNK_COLS - 1) // SSD_CHUNK_COLS) < SSD_SIDE_BLOCKS and B * chunks <= 65535 \
                 and B * chunks * H * N * P * 4 <= SSD_SIDE_BYTES and memory.stride(0) % 4 == 0 and memory.data_ptr() % 16 == 0:
             part = torch.empty((B * chunks, H, N, P), dtype=torch.float32, device=xbc.device)
             decay = torch.empty((B * chunks, H), dtype=torch.float32, device=xbc.device)
