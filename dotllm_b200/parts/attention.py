@@ -65,7 +65,7 @@ class AttentionMixer(Mixer):
     """params: ``n_heads``, ``n_kv_heads``, ``head_dim``, ``window`` (None = all keys),
     ``position`` ({"kind", "params"} of a position encoding), optional ``scale``, optional ``score``
     ({"softcap": c, "slopes": [one per head]}: scores are capped and biased by distance before the
-    softmax, which sends the mixer to the generic attention kernel); optional ``value_dim`` (per head, default
+    softmax; slopes send the mixer to the generic attention kernel); optional ``value_dim`` (per head, default
     ``head_dim``), ``bias`` (True: q, k and v have biases), ``gate`` (None, "head_sigmoid" or "channel_sigmoid"), ``own_kv`` (False: no key
     and value projections, the layer reads another's cache) and ``tensors``: the local names of ``q``, ``k``, ``v``,
     ``o``, ``gate`` and the bias suffix ``bias`` (appended to a projection's name); optional ``values`` ("own", or "keys":
