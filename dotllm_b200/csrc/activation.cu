@@ -40,21 +40,23 @@ extern "C" int dl_swiglu(const void* gate, const void* up, int in_stride, void* 
 // Other gatings of a feed-forward's two products, float32 arithmetic, chosen by `kind`:
 //   1  gelu_tanh(g) * u,  gelu_tanh(z) = 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))
 //   2  g' sigmoid(alpha g') (u' + 1)  with g' = min(g, limit), u' = clamp(u, -limit, limit)
-// (kind 0 is the SwiGLU above.)  `limit` and `alpha` are parameters of kind 2.
+// (kind 0 is the SwiGLU above.)  `limit` and `alpha` are parameters of kind 2.  `bias` (float32 [2 width], the gate's and then
+// the up product's, or NULL) is added first.
 template <typename T>
 __global__ void __launch_bounds__(256)
 gated_activation_kernel(const T* __restrict__ gate, const T* __restrict__ up, int in_stride, T* __restrict__ out,
-                        int rows, int width, int kind, float limit, float alpha) {
+                        int rows, int width, int kind, float limit, float alpha, const float* __restrict__ bias) {
     const size_t n = (size_t)rows * width;
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
         const size_t r = i / width, c = i - r * width;
-        out[i] = dl_from_f32<T>(dl_gate_value(kind, dl_to_f32<T>(gate[r * in_stride + c]), dl_to_f32<T>(up[r * in_stride + c]),
-                                              limit, alpha));
+        float g = dl_to_f32<T>(gate[r * in_stride + c]), u = dl_to_f32<T>(up[r * in_stride + c]);
+        if (bias != nullptr) g += bias[c], u += bias[width + c];
+        out[i] = dl_from_f32<T>(dl_gate_value(kind, g, u, limit, alpha));
     }
 }
 
 extern "C" int dl_gated_activation(const void* gate, const void* up, int in_stride, void* out, int dtype, int rows,
-                                   int width, int kind, float limit, float alpha, void* stream) {
+                                   int width, int kind, float limit, float alpha, const float* bias, void* stream) {
     DL_REQUIRE(rows >= 0 && width > 0 && in_stride >= width && kind >= 0 && kind < GATE_KINDS && dl_gate_is_gated(kind), "gated_activation: bad arguments");
     if (rows == 0) return DL_OK;
     cudaStream_t s = (cudaStream_t)stream;
@@ -62,10 +64,10 @@ extern "C" int dl_gated_activation(const void* gate, const void* up, int in_stri
     const int blocks = (int)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
     if (dtype == DL_F32)
         gated_activation_kernel<float><<<blocks, 256, 0, s>>>((const float*)gate, (const float*)up, in_stride, (float*)out,
-                                                              rows, width, kind, limit, alpha);
+                                                              rows, width, kind, limit, alpha, bias);
     else if (dtype == DL_BF16)
         gated_activation_kernel<__nv_bfloat16><<<blocks, 256, 0, s>>>((const __nv_bfloat16*)gate, (const __nv_bfloat16*)up,
-                                                                      in_stride, (__nv_bfloat16*)out, rows, width, kind, limit, alpha);
+                                                                      in_stride, (__nv_bfloat16*)out, rows, width, kind, limit, alpha, bias);
     else
         return dl_fail(DL_ERR_UNSUPPORTED, "gated_activation: dtype %d", dtype);
     DL_CHECK_LAUNCH("gated_activation");

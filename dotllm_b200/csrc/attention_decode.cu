@@ -280,6 +280,7 @@ struct AdFresh {
     // two options of the mask and of the softmax that travel with the others
     int keep_first;                  // with a window: the sequence's first keys that stay visible behind it
     const float* sinks;              // [nh] float32 or NULL: one more term exp(sinks[head]) in the head's denominator, no key, no value
+    const float* slopes;             // [nh] float32 or NULL: slopes[head] * (key position - query position) is added to the head's scores
     DlScoreCap cap;                  // post > 0: scaled scores s become c tanh(s / c) before the softmax
     int pool_heads;                  // KV heads of the pages; nkv is a multiple of it: neighbouring KV heads of the launch then read
                                      // (and, for the step's own token, write) the same head of the pages, so that more query heads
@@ -510,7 +511,9 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_
         // while that kernel finishes, and q is waited for after it.
         float* my_o = merge_o + (size_t)warp * group * (HD + 4);
         const bool capped = fresh.cap.post > 0.f;
-        const float scale2 = capped ? 1.f : scale * 1.4426950408889634f;    // scores in units of log2 (capped ones come in them)
+        const bool sloped = fresh.slopes != nullptr;
+        const float to_log2 = capped ? 1.f : scale * 1.4426950408889634f;   // scores in units of log2 (capped ones come in them)
+        const float scale2 = sloped ? 1.f : to_log2;                        // ... and so do those that took a distance penalty
         int n0 = 0;                                          // pages of the runs before this one
         const AdCut cut = ad_cut(seq_len, n_seqs, nkv, window, gridDim.x, min_share, lane);
         AdWalk walk = ad_walk_begin(cut, seq_len, n_seqs, nkv, window, blockIdx.x, lane);
@@ -554,6 +557,8 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_
                     }
                 }
             }
+            const float slope_lo = sloped && g < group ? fresh.slopes[w.kvh * group + g] * 1.4426950408889634f : 0.f;
+            const float slope_hi = WIDE && sloped && g + 8 < group ? fresh.slopes[w.kvh * group + g + 8] * 1.4426950408889634f : 0.f;
             float o[DT][4];
 #pragma unroll
             for (int i = 0; i < DT; ++i)
@@ -720,6 +725,19 @@ attention_decode_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv_
                         for (int j = 0; j < 4; ++j)
 #pragma unroll
                             for (int e = 0; e < (WIDE ? 4 : 2); e += 2) dl_cap_scores(sc[h][j][e], sc[h][j][e + 1], fresh.cap);
+                }
+                if (sloped) {                                 // slope * (key - query), the same places as the masks below
+                    const float from = (float)(base + 8 * t - (w.len - 1));
+#pragma unroll
+                    for (int h = 0; h < 2; ++h)
+#pragma unroll
+                        for (int j = 0; j < 4; ++j)
+#pragma unroll
+                            for (int e = 0; e < 2; ++e) {
+                                const float off = from + (float)(32 * h + 2 * j + e);
+                                sc[h][j][e] = fmaf(sc[h][j][e], to_log2, slope_lo * off);
+                                if (WIDE) sc[h][j][2 + e] = fmaf(sc[h][j][2 + e], to_log2, slope_hi * off);
+                            }
                 }
                 // ---- mask (ragged pages only; lane holds keys base + 32h + 8t + 2j + {0,1}) and row maximum
                 if (ragged) {
@@ -959,7 +977,9 @@ static int ad_launch(cudaStream_t s, const void* q, int q_stride, void* out, int
 // q: bf16 [B, nh*hd] rows q_stride apart (one token per sequence); out likewise.
 // seq_len[b]: keys of sequence b including the new token; block_table: int32 [B, bt_stride] page ids.
 // blocks: persistent blocks to use (<= 0: one per multiprocessor).
-// sinks: float32 [nh] or NULL; softcap: 0 for none, else scaled scores s become softcap * tanh(s / softcap).
+// sinks: float32 [nh] or NULL; softcap: 0 for none, else scaled scores s become softcap * tanh(s / softcap); slopes: float32 [nh]
+// or NULL, slopes[h] * (key position - query position) is added to head h's scores after that; gate: bfloat16, one logit per
+// (sequence, query head) in rows gate_stride apart, or NULL: a head's output is multiplied by its sigmoid.
 // pool_heads: KV heads of the pages (usually nkv); a divisor of nkv lets neighbouring KV heads of the launch share one.
 // part_o: float32 [part_slots, group, hd]; part_ml: float32 [part_slots, group, 2]: scratch for the
 // segments of (sequence, head) pairs that the cut spreads over several blocks, two per block.
@@ -1015,14 +1035,17 @@ static int ad_dispatch(const void* q, int q_stride, void* out, int out_stride, v
 extern "C" int dl_attention_decode_bf16(const void* q, int q_stride, void* out, int out_stride, const void* k_pool,
                                         const void* v_pool, int n_pages, const int32_t* seq_len,
                                         const int32_t* block_table, int bt_stride, int n_seqs, int nh, int nkv,
-                                        int hd, float scale, int window, int keep_first, const float* sinks, float softcap, int pool_heads,
-                                        int blocks,
+                                        int hd, float scale, int window, int keep_first, const float* sinks, float softcap,
+                                        const float* slopes, const void* gate, int gate_stride, int pool_heads, int blocks,
                                         float* part_o, float* part_ml, int part_slots, int* pair_counters, int n_counters,
                                         int* status, void* stream) {
     DL_REQUIRE(keep_first >= 0 && (keep_first == 0 || window > 0), "attention_decode: kept first keys need a window");
     AdFresh none = {};
     none.keep_first = keep_first;
     none.sinks = sinks;
+    none.slopes = slopes;
+    none.gate = (const __nv_bfloat16*)gate;
+    none.gate_stride = gate_stride;
     none.cap = dl_score_cap(softcap, scale);
     none.pool_heads = pool_heads;
     return ad_dispatch(q, q_stride, out, out_stride, const_cast<void*>(k_pool), const_cast<void*>(v_pool), n_pages, seq_len,
@@ -1062,12 +1085,12 @@ extern "C" int dl_attention_decode_fresh_bf16(const void* q, int q_stride, const
 // [nkv*hd] (float32, each NULL for none) are added before the rotation, with one rounding behind it as in
 // dl_rope_cache_write; gate (bfloat16, one logit per (sequence, query head), rows gate_stride apart, or NULL) multiplies
 // a head's output by sigmoid(logit) where it is written.  k_new and v_new may be NULL: a layer that reads another
-// layer's cache only biases and rotates its queries, and writes nothing to the pages.  sinks, softcap and pool_heads as in
+// layer's cache only biases and rotates its queries, and writes nothing to the pages.  sinks, softcap, slopes and pool_heads as in
 // dl_attention_decode_bf16.
 extern "C" int dl_attention_decode_gated_bf16(const void* q, int q_stride, const void* k_new, int k_stride, const void* v_new,
                                               int v_stride, const float* cos_t, const float* sin_t, int table_rows, int rotate,
                                               const float* q_bias, const float* k_bias, const float* v_bias, const void* gate,
-                                              int gate_stride, const float* sinks, float softcap, int pool_heads, void* out, int out_stride, void* k_pool, void* v_pool, int n_pages,
+                                              int gate_stride, const float* sinks, float softcap, const float* slopes, int pool_heads, void* out, int out_stride, void* k_pool, void* v_pool, int n_pages,
                                               const int32_t* seq_len, const int32_t* block_table, int bt_stride, int n_seqs,
                                               int nh, int nkv, int hd, float scale, int window, int blocks, float* part_o,
                                               float* part_ml, int part_slots, int* pair_counters, int n_counters, int* status,
@@ -1088,6 +1111,7 @@ extern "C" int dl_attention_decode_gated_bf16(const void* q, int q_stride, const
     fresh.gate = (const __nv_bfloat16*)gate;
     fresh.gate_stride = gate_stride;
     fresh.sinks = sinks;
+    fresh.slopes = slopes;
     fresh.cap = dl_score_cap(softcap, scale);
     fresh.pool_heads = pool_heads;
     return ad_dispatch(q, q_stride, out, out_stride, k_pool, v_pool, n_pages, seq_len, block_table, bt_stride, n_seqs, nh, nkv,

@@ -88,7 +88,8 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
                          const int32_t* __restrict__ seq_start, const int32_t* __restrict__ seq_new,
                          const int32_t* __restrict__ cu_new, const int32_t* __restrict__ block_table,
                          int bt_stride, int nh, int nkv, float scale, int window, int keep_first,
-                         const float* __restrict__ sinks, const DlScoreCap cap, int* __restrict__ status) {
+                         const float* __restrict__ sinks, const DlScoreCap cap, const float* __restrict__ slopes,
+                         const __nv_bfloat16* __restrict__ gate, int gate_stride, int* __restrict__ status) {
     constexpr int DC = HD / 32;
     constexpr int DT = HD / 8;
     constexpr int PAGE_ELEMS = DL_PAGE * HD;
@@ -167,7 +168,10 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
         const int first_hi = (window > 0) ? pos_hi - window + 1 : 0;
         const int warp_first = (window > 0 && warp_pos_min - window + 1 > 0) ? warp_pos_min - window + 1 : 0;
         const bool capped = cap.post > 0.f;
-        const float scale2 = capped ? 1.f : scale * 1.4426950408889634f;    // scores in units of log2 (capped ones come in them)
+        const bool sloped = slopes != nullptr;
+        const float to_log2 = capped ? 1.f : scale * 1.4426950408889634f;   // scores in units of log2 (capped ones come in them)
+        const float scale2 = sloped ? 1.f : to_log2;                        // ... and so do those that took a distance penalty
+        const float slope2 = sloped ? slopes[h] * 1.4426950408889634f : 0.f;
 
         uint4 qf_lo[DC], qf_hi[DC];
 #pragma unroll
@@ -233,6 +237,19 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
                         for (int j = 0; j < 4; ++j)
 #pragma unroll
                             for (int e = 0; e < 4; e += 2) dl_cap_scores(sc[hh][j][e], sc[hh][j][e + 1], cap);
+                }
+                if (sloped) {                                 // slope * (key - query), the same places as the masks below
+                    const float b_lo = (float)(base + 8 * t - (start + row0 + g)), b_hi = b_lo - 8.f;
+#pragma unroll
+                    for (int hh = 0; hh < 2; ++hh)
+#pragma unroll
+                        for (int j = 0; j < 4; ++j)
+#pragma unroll
+                            for (int e = 0; e < 2; ++e) {
+                                const float off = (float)(32 * hh + 2 * j + e);
+                                sc[hh][j][e] = fmaf(sc[hh][j][e], to_log2, slope2 * (b_lo + off));
+                                sc[hh][j][2 + e] = fmaf(sc[hh][j][2 + e], to_log2, slope2 * (b_hi + off));
+                            }
                 }
                 if (ragged) {
                     // lane holds keys base + 32hh + 8t + 2j + {0,1} of rows g (lo) and g+8 (hi).  Masked
@@ -340,7 +357,11 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, __nv
                 l_lo += ap_ex2(sink2 - m_lo);
                 l_hi += ap_ex2(sink2 - m_hi);
             }
-            const float inv_lo = 1.0f / l_lo, inv_hi = 1.0f / l_hi;
+            float inv_lo = 1.0f / l_lo, inv_hi = 1.0f / l_hi;
+            if (gate != nullptr) {                           // a gate per (token, head)
+                if (ok_lo) inv_lo *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)(tok0 + g) * gate_stride + h])));
+                if (ok_hi) inv_hi *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)(tok0 + g + 8) * gate_stride + h])));
+            }
             __nv_bfloat16* o_lo = out + (size_t)(tok0 + g) * out_stride + (size_t)h * HD;
             __nv_bfloat16* o_hi = out + (size_t)(tok0 + g + 8) * out_stride + (size_t)h * HD;
 #pragma unroll
@@ -358,7 +379,8 @@ static int ap_launch(dim3 grid, cudaStream_t s, const void* q, int q_stride, voi
                      const void* k_pool, const void* v_pool, int n_pages, const int32_t* tile_seq,
                      const int32_t* tile_row0, const int32_t* seq_start, const int32_t* seq_new,
                      const int32_t* cu_new, const int32_t* block_table, int bt_stride, int nh, int nkv, float scale,
-                     int window, int keep_first, const float* sinks, float softcap, int* status) {
+                     int window, int keep_first, const float* sinks, float softcap, const float* slopes, const void* gate,
+                     int gate_stride, int* status) {
     const size_t smem = (size_t)AP_STAGES * 2 * DL_PAGE * HD * 2;
     static bool configured = false;
     if (!configured) {
@@ -369,7 +391,7 @@ static int ap_launch(dim3 grid, cudaStream_t s, const void* q, int q_stride, voi
     attention_prefill_kernel<HD><<<grid, AP_THREADS, smem, s>>>(
         (const __nv_bfloat16*)q, q_stride, (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)k_pool,
         (const __nv_bfloat16*)v_pool, n_pages, tile_seq, tile_row0, seq_start, seq_new, cu_new, block_table, bt_stride,
-        nh, nkv, scale, window, keep_first, sinks, dl_score_cap(softcap, scale), status);
+        nh, nkv, scale, window, keep_first, sinks, dl_score_cap(softcap, scale), slopes, (const __nv_bfloat16*)gate, gate_stride, status);
     DL_CHECK_LAUNCH("attention_prefill");
     return DL_OK;
 }
@@ -378,14 +400,16 @@ static int ap_launch(dim3 grid, cudaStream_t s, const void* q, int q_stride, voi
 // 128-row tile its sequence and its first row among that sequence's new tokens.  seq_start,
 // seq_new: cached length before the step and new tokens, per sequence; cu_new: packed offsets.
 // keep_first: with a window, that many first keys of a sequence stay visible.  sinks: float32 [nh] or NULL, exp(sinks[h])
-// joins head h's softmax denominator.  softcap: 0 for none, else scaled scores s become softcap * tanh(s / softcap).  status: int32, set non-zero if a wait expired.
+// joins head h's softmax denominator.  softcap: 0 for none, else scaled scores s become softcap * tanh(s / softcap).  slopes:
+// float32 [nh] or NULL, slopes[h] * (key position - query position) is added to head h's scores after that.  gate: bf16, one logit per
+// (token, head) in rows gate_stride apart, or NULL: a head's output is multiplied by its sigmoid.  status: int32, set non-zero if a wait expired.
 extern "C" int dl_attention_prefill_bf16(const void* q, int q_stride, void* out, int out_stride,
                                          const void* k_pool, const void* v_pool, int n_pages,
                                          const int32_t* tile_seq, const int32_t* tile_row0, int n_tiles,
                                          const int32_t* seq_start, const int32_t* seq_new, const int32_t* cu_new,
                                          const int32_t* block_table, int bt_stride, int nh, int nkv, int hd,
-                                         float scale, int window, int keep_first, const float* sinks, float softcap, int* status,
-                                         void* stream) {
+                                         float scale, int window, int keep_first, const float* sinks, float softcap,
+                                         const float* slopes, const void* gate, int gate_stride, int* status, void* stream) {
     DL_REQUIRE(n_tiles >= 0 && nh > 0 && nkv > 0 && nh % nkv == 0, "attention_prefill: bad sizes");
     DL_REQUIRE(scale > 0.f, "attention_prefill: the score scale must be positive");
     DL_REQUIRE(keep_first >= 0 && window >= 0, "attention_prefill: the window and the kept first tokens cannot be negative");
@@ -394,6 +418,7 @@ extern "C" int dl_attention_prefill_bf16(const void* q, int q_stride, void* out,
                    ((uintptr_t)k_pool % 16) == 0 && ((uintptr_t)v_pool % 16) == 0,
                "attention_prefill: q and the pools must be 16-byte aligned");
     DL_REQUIRE(nh <= 65535, "attention_prefill: too many heads");
+    DL_REQUIRE(gate == nullptr || gate_stride >= nh, "attention_prefill: a row of gate logits holds one per query head");
     if (n_tiles == 0) return DL_OK;
     DL_REQUIRE(n_tiles <= 65535, "attention_prefill: too many tiles (%d)", n_tiles);
     dim3 grid(nh, n_tiles);
@@ -401,7 +426,7 @@ extern "C" int dl_attention_prefill_bf16(const void* q, int q_stride, void* out,
 #define AP_CASE(HDV)                                                                                                  \
     if (hd == HDV)                                                                                                    \
         return ap_launch<HDV>(grid, s, q, q_stride, out, out_stride, k_pool, v_pool, n_pages, tile_seq, tile_row0,     \
-                              seq_start, seq_new, cu_new, block_table, bt_stride, nh, nkv, scale, window, keep_first, sinks, softcap, status);
+                              seq_start, seq_new, cu_new, block_table, bt_stride, nh, nkv, scale, window, keep_first, sinks, softcap, slopes, gate, gate_stride, status);
     AP_CASE(32) AP_CASE(64) AP_CASE(96) AP_CASE(128)
 #undef AP_CASE
     return dl_fail(DL_ERR_UNSUPPORTED, "attention_prefill: head_dim %d (takes 32, 64, 96, 128)", hd);

@@ -86,8 +86,10 @@ struct PtTile {
     int j_lo, j_hi;          // the pages of the block's walk it takes part in (j_lo > j_hi: none)
 };
 
-// CAP: scaled scores s become c tanh(s / c) before the softmax.
-template <int HD, bool CAP>
+// What happens to scaled scores before the softmax: nothing; s becomes c tanh(s / c); slope_h * (key - query) is added.
+enum { PT_PLAIN = 0, PT_CAP = 1, PT_SLOPE = 2 };
+
+template <int HD, int SHAPE>
 __global__ void __launch_bounds__(PT_THREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                             const __grid_constant__ CUtensorMap tmap_v, __nv_bfloat16* __restrict__ out, int out_stride,
@@ -95,7 +97,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
                             const int32_t* __restrict__ seq_start, const int32_t* __restrict__ seq_new,
                             const int32_t* __restrict__ cu_new, const int32_t* __restrict__ block_table, int bt_stride,
                             int nkv, int group, float scale, int window, int keep_first, const float* __restrict__ sinks, const DlScoreCap cap,
-                            int* __restrict__ status) {
+                            const float* __restrict__ slopes, const __nv_bfloat16* __restrict__ gate, int gate_stride, int* __restrict__ status) {
+    constexpr bool CAP = SHAPE == PT_CAP;
     constexpr int ATOMS = HD / 64;                           // 64-dim (128-byte) slices of a head
     constexpr int STAGES = PT_STAGES(HD);
     constexpr uint32_t Q_BYTES = PT_ROWS * HD * 2;
@@ -307,7 +310,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
         const bool stamps = (warp == 4 && lane == 0);
         const uint32_t lane_base = (uint32_t)(quarter * 32) << 16;
         const uint32_t my_s = tmem_s + lane_base + (uint32_t)(2 * t * DL_PAGE), my_o = tmem_o + lane_base + (uint32_t)(t * HD);
-        const float scale2 = CAP ? 1.f : scale * 1.4426950408889634f;    // scores in units of log2 (capped ones come in them)
+        const float scale2 = SHAPE != PT_PLAIN ? 1.f : scale * 1.4426950408889634f;    // scores in units of log2 (the others come in them)
+        const float to_log2 = scale * 1.4426950408889634f, slope2 = SHAPE == PT_SLOPE ? slopes[head] * 1.4426950408889634f : 0.f;
         float m_ref = -INFINITY, l = 0.f;                    // reference maximum (log2 units), sum of weights
         bool ok = true;
         const int n_mine = T.j_hi - T.j_lo + 1;
@@ -341,6 +345,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
                 for (int i = 0; i < 64; i += 2) dl_cap_scores(sc[i], sc[i + 1], cap);
             }
             const int key0 = page_of(j) * DL_PAGE;
+            if (SHAPE == PT_SLOPE) {
+                const float from = slope2 * (float)(key0 - pos);
+#pragma unroll
+                for (int i = 0; i < 64; ++i) sc[i] = fmaf(sc[i], to_log2, fmaf(slope2, (float)i, from));
+            }
             // pages wholly visible to every row of the tile need no mask
             const bool ragged = T.rows < PT_ROWS || key0 + DL_PAGE - 1 > T.pos0 || key0 < T.first_key ||
                                 (window > 0 && key0 <= T.pos_last - window);
@@ -433,7 +442,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
             tc_fence_after();
             // the sink: one more term in the sum of weights, with no value; m_ref is in units of log2
             if (sinks != nullptr && m_ref > -INFINITY) l += pt_ex2(fmaf(sinks[head], 1.4426950408889634f, -m_ref));
-            const float inv = l > 0.f ? 1.f / l : 0.f;
+            float inv = l > 0.f ? 1.f / l : 0.f;
+            if (gate != nullptr && live)                     // a gate per (token, head)
+                inv *= 1.f / (1.f + expf(-__bfloat162float(gate[(size_t)(cu_new[b] + row0 + t * PT_ROWS + r) * gate_stride + head])));
             __nv_bfloat16* dst = out + (size_t)(cu_new[b] + row0 + t * PT_ROWS + r) * out_stride + (size_t)head * HD;
 #pragma unroll 1
             for (int c0 = 0; c0 < HD; c0 += 32) {
@@ -491,17 +502,17 @@ static int pt_tensor_map(CUtensorMap* out, const void* base, long long rows, lon
     return DL_OK;
 }
 
-template <int HD, bool CAP>
+template <int HD, int SHAPE>
 static int pt_launch(dim3 grid, cudaStream_t s, const void* q, int q_stride, int n_tokens, void* out, int out_stride,
                      const void* k_pool, const void* v_pool, int n_pages, const int32_t* tile_seq, const int32_t* tile_row0,
                      const int32_t* seq_start, const int32_t* seq_new, const int32_t* cu_new, const int32_t* block_table,
                      int bt_stride, int nh, int nkv, float scale, int window, int keep_first, const float* sinks, float softcap,
-                     int* status) {
+                     const float* slopes, const void* gate, int gate_stride, int* status) {
     const size_t smem = (size_t)PT_TILES * PT_ROWS * HD * 2 + (size_t)PT_STAGES(HD) * 2 * DL_PAGE * HD * 2 +
                         (size_t)PT_TILES * 2 * PT_ROWS * DL_PAGE * 2 + 1024;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<HD, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<HD, SHAPE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return dl_fail(DL_ERR_LAUNCH, "attention_prefill_tc: shared memory %zu: %s", smem, cudaGetErrorString(e));
         configured = true;
     }
@@ -512,10 +523,11 @@ static int pt_launch(dim3 grid, cudaStream_t s, const void* q, int q_stride, int
     if (rc != DL_OK) return rc;
     rc = pt_tensor_map(&tmap_v, v_pool, (long long)n_pages * nkv * HD, DL_PAGE, (long long)DL_PAGE * 2, HD);
     if (rc != DL_OK) return rc;
-    attention_prefill_tc_kernel<HD, CAP><<<grid, PT_THREADS, smem, s>>>(tmap_q, tmap_k, tmap_v, (__nv_bfloat16*)out, out_stride, n_pages,
+    attention_prefill_tc_kernel<HD, SHAPE><<<grid, PT_THREADS, smem, s>>>(tmap_q, tmap_k, tmap_v, (__nv_bfloat16*)out, out_stride, n_pages,
                                                                   tile_seq, tile_row0, seq_start, seq_new, cu_new, block_table,
                                                                   bt_stride, nkv, nh / nkv, scale, window, keep_first, sinks,
-                                                                  dl_score_cap(softcap, scale), status);
+                                                                  dl_score_cap(softcap, scale), slopes, (const __nv_bfloat16*)gate,
+                                                                  gate_stride, status);
     DL_CHECK_LAUNCH("attention_prefill_tc");
     return DL_OK;
 }
@@ -526,13 +538,16 @@ static int pt_launch(dim3 grid, cudaStream_t s, const void* q, int q_stride, int
 // seq_new: cached length before the step and new tokens, per sequence; cu_new: packed offsets.
 // head_dim 64 or 128.  keep_first: with a window, that many first tokens of a sequence stay visible; sinks: float32 [nh]
 // or null, exp(sinks[h]) joins head h's sum of weights; softcap: 0 for none, else scaled scores s become
-// softcap * tanh(s / softcap).  status: int32, set non-zero if a wait expired.
+// softcap * tanh(s / softcap); slopes: float32 [nh] or null, slopes[h] * (key position - query position) is added to head h's scaled
+// scores (not together with a softcap); gate: bf16, one logit per (token, head) in rows gate_stride apart, or null: a head's output is
+// multiplied by its sigmoid.  status: int32, set non-zero if a wait expired.
 extern "C" int dl_attention_prefill_tc_bf16(const void* q, int q_stride, int n_tokens, void* out, int out_stride,
                                             const void* k_pool, const void* v_pool, int n_pages, const int32_t* tile_seq,
                                             const int32_t* tile_row0, int n_tiles, const int32_t* seq_start,
                                             const int32_t* seq_new, const int32_t* cu_new, const int32_t* block_table,
                                             int bt_stride, int nh, int nkv, int hd, float scale, int window, int keep_first,
-                                            const float* sinks, float softcap, int* status, void* stream) {
+                                            const float* sinks, float softcap, const float* slopes, const void* gate,
+                                            int gate_stride, int* status, void* stream) {
     DL_REQUIRE(n_tiles >= 0 && n_tokens >= 0 && nh > 0 && nkv > 0 && nh % nkv == 0, "attention_prefill_tc: bad sizes");
     DL_REQUIRE(scale > 0.f && window >= 0, "attention_prefill_tc: the score scale must be positive, the window not negative");
     DL_REQUIRE(keep_first >= 0 && (keep_first == 0 || window > 0), "attention_prefill_tc: kept first tokens go with a window");
@@ -543,16 +558,19 @@ extern "C" int dl_attention_prefill_tc_bf16(const void* q, int q_stride, int n_t
     DL_REQUIRE(q_stride >= nh * hd && out_stride >= nh * hd, "attention_prefill_tc: row strides shorter than the rows");
     DL_REQUIRE((long long)n_pages * nkv * (hd > DL_PAGE ? hd : DL_PAGE) < (1ll << 31),
                "attention_prefill_tc: too many heads or pages");
+    DL_REQUIRE(softcap <= 0.f || slopes == nullptr, "attention_prefill_tc: a cap or slopes, not both");
+    DL_REQUIRE(gate == nullptr || gate_stride >= nh, "attention_prefill_tc: a row of gate logits holds one per query head");
     if (n_tiles == 0) return DL_OK;
+    const int shape = softcap > 0.f ? PT_CAP : (slopes != nullptr ? PT_SLOPE : PT_PLAIN);
     DL_REQUIRE(n_tiles <= 65535, "attention_prefill_tc: too many tiles (%d)", n_tiles);
     dim3 grid(nh, n_tiles);
     cudaStream_t s = (cudaStream_t)stream;
-#define PT_CASE(HDV, CAPV)                                                                                              \
-    if (hd == HDV && (softcap > 0.f) == CAPV)                                                                          \
-        return pt_launch<HDV, CAPV>(grid, s, q, q_stride, n_tokens, out, out_stride, k_pool, v_pool, n_pages, tile_seq, \
+#define PT_CASE(HDV, SHAPEV)                                                                                              \
+    if (hd == HDV && shape == SHAPEV)                                                                          \
+        return pt_launch<HDV, SHAPEV>(grid, s, q, q_stride, n_tokens, out, out_stride, k_pool, v_pool, n_pages, tile_seq, \
                                     tile_row0, seq_start, seq_new, cu_new, block_table, bt_stride, nh, nkv, scale, window, \
-                                    keep_first, sinks, softcap, status);
-    PT_CASE(64, false) PT_CASE(128, false) PT_CASE(64, true) PT_CASE(128, true)
+                                    keep_first, sinks, softcap, slopes, gate, gate_stride, status);
+    PT_CASE(64, PT_PLAIN) PT_CASE(128, PT_PLAIN) PT_CASE(64, PT_CAP) PT_CASE(128, PT_CAP) PT_CASE(64, PT_SLOPE) PT_CASE(128, PT_SLOPE)
 #undef PT_CASE
     return dl_fail(DL_ERR_UNSUPPORTED, "attention_prefill_tc: head_dim %d (takes 64 and 128)", hd);
 }

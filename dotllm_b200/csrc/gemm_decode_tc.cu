@@ -74,6 +74,7 @@ struct GdFuse {
     const float* sumsq_in;      // set: output row m is multiplied by rsqrt(sum_p sumsq_in[p * 128 + m] * inv_n + eps)
     int n_parts;
     float inv_n, eps;
+    const float* gate_bias;     // gated products: set: [2N], added to the gate and the up rows' products before the gating
 };
 
 struct GdWork {
@@ -107,14 +108,14 @@ __device__ __forceinline__ void gd_epilogue_sync() { asm volatile("bar.sync 1, %
 // form, unrolled).
 //
 // 8 tokens c .. c+7 of output column n, held by this thread: scale, gate, add into the stream, store.
-// `u` is read only when GATED.  `ss_row`: this warp's row of the per-token sums of squares in shared
+// `u` is read only when GATED, `bias_g` / `bias_u` (this column's biases of gate and up) likewise.  `ss_row`: this warp's row of the per-token sums of squares in shared
 // memory (add-into-stream only); `h_in`: the stream's present values of these tokens (gd_stream8).
 // Loads, arithmetic and stores are kept in separate stages so that
 // the 8 tokens' chains overlap (a store between two tokens' loads would order them).
 template <typename TOut, bool GATED>
 __device__ __forceinline__ void gd_finish8(const float (&v)[8], const float (&u)[8], int c, int n, bool n_ok, TOut* __restrict__ out,
                                            int out_stride, int M, const float* __restrict__ row_scale, const GdFuse& fuse,
-                                           float gain_n, float* __restrict__ ss_row, int lane, const float (&h_in)[8]) {
+                                           float gain_n, float* __restrict__ ss_row, int lane, const float (&h_in)[8], float bias_g, float bias_u) {
     float val[8];
 #pragma unroll
     for (int i = 0; i < 8; ++i) val[i] = row_scale != nullptr ? row_scale[min(c + i, GD_MAX_ROWS - 1)] : 1.0f;
@@ -152,7 +153,8 @@ __device__ __forceinline__ void gd_finish8(const float (&v)[8], const float (&u)
         for (int i = 0; i < 8; ++i) {
             float g = row_scale != nullptr ? v[i] * val[i] : v[i];
             if (GATED) {
-                const float up = row_scale != nullptr ? u[i] * val[i] : u[i];
+                const float up = (row_scale != nullptr ? u[i] * val[i] : u[i]) + bias_u;
+                g += bias_g;
                 // bfloat16 keeps 8 bits: the fast exponential and reciprocal (errors of a few float32 ulps) change
                 // no output bit that the exact ones would not; a float32 result gets the exact functions
                 if (std::is_same<TOut, float>::value) g = g * (1.0f / (1.0f + expf(-g))) * up;
@@ -455,6 +457,8 @@ gemm_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_c
                     const int n = tile * GD_BM + lane128;
                     const bool n_ok = n < N;
                     const float gain_n = (adds && n_ok) ? __ldg(work.fuse.gain + n) : 0.f;
+                    const bool biased = GATED && n_ok && work.fuse.gate_bias != nullptr;
+                    const float bias_g = biased ? __ldg(work.fuse.gate_bias + n) : 0.f, bias_u = biased ? __ldg(work.fuse.gate_bias + work.N + n) : 0.f;
                     const int col = c0;                      // first accumulator column of the chunk (gate's when gated)
                     // The stream's values of this group's slices are asked for now: they arrive while the
                     // merge data does (only this tile's finisher ever writes them).
@@ -518,7 +522,7 @@ gemm_decode_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_c
                             }
                         }
                         gd_finish8<TOut, GATED>(v, u, c, n, n_ok, out, work.out_stride, M, row_scale, work.fuse, gain_n,
-                                                ss_part[quarter], lane, h_pre[j]);
+                                                ss_part[quarter], lane, h_pre[j], bias_g, bias_u);
                     }
                     if (bulk) {
                         // Every thread's reads of the buffer have completed (their values went into the stores
@@ -631,12 +635,13 @@ static int gd_launch(const GdPlan& p, cudaStream_t s, const void* x, int x_strid
 // writes w, so the kernel may start reading w before the kernel launched before it has finished.
 // gain / scaled / sumsq_out and sumsq_in / n_parts / inv_n / eps: the fusions described at the top
 // (all null: a plain product); sums are laid out [part of 128 columns][128] floats.
+// gate_bias: float32 [2N] (the gate rows', then the up rows') or NULL, added before the gating.
 // partials / counters: scratch of the sizes dl_gemm_decode_tc_scratch gives; status: int32, set
 // non-zero if a wait expired.
 extern "C" int dl_gemm_decode_tc_bf16(const void* x, int x_stride, const void* w, void* out, int out_dtype, int out_stride, int M,
                                       int N, int K, int flags, const float* gain, void* scaled, int scaled_stride,
                                       float* sumsq_out, const float* sumsq_in, int n_parts, float inv_n, float eps,
-                                      float* partials, long long partial_floats, int* counters, int n_counters, int* status,
+                                      const float* gate_bias, float* partials, long long partial_floats, int* counters, int n_counters, int* status,
                                       void* stream) {
     const int gated = flags & 1, early = (flags >> 1) & 1;
     DL_REQUIRE((flags & ~3) == 0, "gemm_decode_tc: unknown flags %d", flags);
@@ -648,7 +653,9 @@ extern "C" int dl_gemm_decode_tc_bf16(const void* x, int x_stride, const void* w
     DL_REQUIRE(out_dtype == DL_F32 || out_dtype == DL_BF16, "gemm_decode_tc: out dtype %d", out_dtype);
     DL_REQUIRE(status != nullptr && partials != nullptr && counters != nullptr, "gemm_decode_tc: needs scratch and a status word");
     DL_REQUIRE(((uintptr_t)partials % 16) == 0, "gemm_decode_tc: the partial sums must be 16-byte aligned");
+    DL_REQUIRE(gate_bias == nullptr || gated, "gemm_decode_tc: biases go with the gated product");
     GdFuse fuse{};
+    fuse.gate_bias = gate_bias;
     if (gain != nullptr) {
         DL_REQUIRE(out_dtype == DL_F32 && !gated, "gemm_decode_tc: adding into the stream needs a plain float32 product");
         DL_REQUIRE(scaled != nullptr && sumsq_out != nullptr && scaled_stride >= N, "gemm_decode_tc: the scaled copy and the sums need a place");

@@ -108,6 +108,7 @@ struct GsFuse {
     float inv_n, eps;
     int gate_kind;              // gated products: 0 = SwiGLU, else a gating of gating.cuh with ...
     float gate_limit, gate_alpha;   // ... its constants
+    const float* gate_bias;     // gated products: set: [2N], added to the gate and the up rows' products before the gating
 };
 
 // acc[j] = {(row g, tok 2t), (row g, tok 2t+1), (row g+8, tok 2t), (row g+8, tok 2t+1)} of 8-token group j
@@ -128,6 +129,10 @@ __device__ __forceinline__ void gs_epilogue(const float (&acc_in)[NT][4], TOut* 
         if (FUSE_SWIGLU) {
             const int col = tile * 8 + g;
             if (col < N) {
+                if (fuse.gate_bias != nullptr) {
+                    const float bg = __ldg(fuse.gate_bias + col), bu = __ldg(fuse.gate_bias + N + col);
+                    acc[0] += bg, acc[1] += bg, acc[2] += bu, acc[3] += bu;
+                }
                 const float g0 = acc[0], g1 = acc[1];
                 if (fuse.gate_kind != GATE_SILU) {
                     if (tok0 < M)
@@ -638,15 +643,16 @@ extern "C" int dl_gemm_skinny_bf16(const void* x, int x_stride, const void* w, v
 
 // The gated product with another gating than SwiGLU (gating.cuh) in its epilogue; arguments as dl_gemm_skinny_bf16
 // with the gated flag set.  With a `gate_kind` that is an activation of ONE product (relu^2) the gated flag is clear,
-// w is [N, K] and out = act(x W^T).
+// w is [N, K] and out = act(x W^T).  bias: float32 [2N] (the gate rows', then the up rows') or NULL, added before the gating.
 extern "C" int dl_gemm_skinny_gated_bf16(const void* x, int x_stride, const void* w, void* out, int out_dtype,
                                          int out_stride, int M, int N, int K, int flags, int gate_kind, float limit, float alpha,
-                                         float* partials, int partial_floats, int* counters, int n_counters, int* status,
+                                         const float* bias, float* partials, int partial_floats, int* counters, int n_counters, int* status,
                                          void* stream) {
     DL_REQUIRE(gate_kind >= 0 && gate_kind < GATE_KINDS && ((flags & 1) == 1) == dl_gate_is_gated(gate_kind),
                "gemm_skinny_gated: a known gating, and the gated flag exactly where it reads two products");
+    DL_REQUIRE(bias == nullptr || (flags & 1) == 1, "gemm_skinny_gated: biases go with two products");
     GsFuse fuse{};
-    fuse.gate_kind = gate_kind, fuse.gate_limit = limit, fuse.gate_alpha = alpha;
+    fuse.gate_kind = gate_kind, fuse.gate_limit = limit, fuse.gate_alpha = alpha, fuse.gate_bias = bias;
     return gs_run(x, x_stride, w, out, out_dtype, out_stride, M, N, K, flags, partials, partial_floats, counters, n_counters,
                   status, stream, fuse);
 }

@@ -95,6 +95,7 @@ struct GtGroups {
     int up_offset;
     int gate_kind;
     float limit, alpha;
+    const float* bias;               // GT_GATED: [2N] or NULL, added to the gate and the up columns before the gating
 };
 
 // What the Q/K/V epilogue needs: the columns' split, the rotary tables, where every token (row of x)
@@ -349,6 +350,22 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_constant
                     if (GATED) {
                         float u[32];
                         tc_tmem_load32(taddr + (uint32_t)(GT_BN / 2 + c0), u);
+                        if (MODE == GT_GATED && grp.bias != nullptr) {
+                            const int cb = col_base + c0;
+                            if (cb + 32 <= N && (N & 3) == 0) {           // the same 32 columns in every lane: one broadcast read
+#pragma unroll
+                                for (int i = 0; i < 32; i += 4) {
+                                    const float4 bg = __ldg(reinterpret_cast<const float4*>(grp.bias + cb + i));
+                                    const float4 bu = __ldg(reinterpret_cast<const float4*>(grp.bias + N + cb + i));
+                                    v[i] += bg.x, v[i + 1] += bg.y, v[i + 2] += bg.z, v[i + 3] += bg.w;
+                                    u[i] += bu.x, u[i + 1] += bu.y, u[i + 2] += bu.z, u[i + 3] += bu.w;
+                                }
+                            } else {
+#pragma unroll
+                                for (int i = 0; i < 32; ++i)
+                                    if (cb + i < N) v[i] += __ldg(grp.bias + cb + i), u[i] += __ldg(grp.bias + N + cb + i);
+                            }
+                        }
                         if (GROUPED || grp.gate_kind != GATE_SILU) {
 #pragma unroll
                             for (int i = 0; i < 32; ++i) v[i] = dl_gate_value(grp.gate_kind, v[i], u[i], grp.limit, grp.alpha);
@@ -470,14 +487,16 @@ extern "C" int dl_gemm_tc_bf16(const void* x, int x_stride, const void* w, void*
 }
 
 // The gated product with another gating than SwiGLU in its epilogue (gating.cuh: the tanh form of gelu, or the clamped
-// sigmoid gating with its limit and alpha).  Arguments as dl_gemm_tc_bf16 with the gated flag; bfloat16 out.
+// sigmoid gating with its limit and alpha) or with biases (float32 [2N], the gate rows' and then the up rows', or NULL) added
+// before the gating.  Arguments as dl_gemm_tc_bf16 with the gated flag; bfloat16 out.
 extern "C" int dl_gemm_tc_gated_bf16(const void* x, int x_stride, const void* w, void* out, int out_stride, int M, int N, int K,
-                                     int gate_kind, float limit, float alpha, int blocks, int* status, void* stream) {
+                                     int gate_kind, float limit, float alpha, const float* bias, int blocks, int* status, void* stream) {
     DL_REQUIRE(M >= 1 && N >= 1 && K >= 8 && K % 8 == 0, "gemm_tc_gated: M=%d N=%d K=%d (K must be a positive multiple of 8)", M, N, K);
     DL_REQUIRE(x_stride >= K && x_stride % 8 == 0 && out_stride >= N, "gemm_tc_gated: row strides");
     DL_REQUIRE(((uintptr_t)x % 16) == 0 && ((uintptr_t)w % 16) == 0, "gemm_tc_gated: x and W must be 16-byte aligned");
     DL_REQUIRE(gate_kind >= 0 && gate_kind < GATE_KINDS && status != nullptr, "gemm_tc_gated: unknown gating %d", gate_kind);
-    const GtGroups grp{nullptr, 0, 0, gate_kind, limit, alpha};
+    DL_REQUIRE(bias == nullptr || (dl_gate_is_gated(gate_kind) && ((uintptr_t)bias % 16) == 0), "gemm_tc_gated: 16-byte aligned biases of two products");
+    const GtGroups grp{nullptr, 0, 0, gate_kind, limit, alpha, bias};
     if (!dl_gate_is_gated(gate_kind))            // an activation of one product: w is [N, K], the epilogue applies it
         return gt_launch<__nv_bfloat16, GT_PLAIN>((cudaStream_t)stream, x, x_stride, w, out, out_stride, M, N, K, blocks, status, GtQkv{}, grp);
     return gt_launch<__nv_bfloat16, GT_GATED>((cudaStream_t)stream, x, x_stride, w, out, out_stride, M, N, K, blocks, status, GtQkv{}, grp);
@@ -502,11 +521,11 @@ extern "C" int dl_gemm_tc_grouped_bf16(const void* x, int x_stride, const void* 
     cudaStream_t s = (cudaStream_t)stream;
     if (gated) {
         DL_REQUIRE(out_dtype == DL_BF16 && gate_kind >= 0 && gate_kind < GATE_KINDS && dl_gate_is_gated(gate_kind), "gemm_tc_grouped: the gated product writes bfloat16");
-        const GtGroups grp{tile_expert, 2 * N, N, gate_kind, limit, alpha};
+        const GtGroups grp{tile_expert, 2 * N, N, gate_kind, limit, alpha, nullptr};
         return gt_launch<__nv_bfloat16, GT_GROUPED_GATED>(s, x, x_stride, w, out, out_stride, M, N, K, blocks, status, GtQkv{}, grp,
                                                           n_experts);
     }
-    const GtGroups grp{tile_expert, N, 0, dl_gate_is_gated(gate_kind) ? 0 : gate_kind, 0.f, 0.f};
+    const GtGroups grp{tile_expert, N, 0, dl_gate_is_gated(gate_kind) ? 0 : gate_kind, 0.f, 0.f, nullptr};
     if (out_dtype == DL_F32)
         return gt_launch<float, GT_GROUPED>(s, x, x_stride, w, out, out_stride, M, N, K, blocks, status, GtQkv{}, grp, n_experts);
     return gt_launch<__nv_bfloat16, GT_GROUPED>(s, x, x_stride, w, out, out_stride, M, N, K, blocks, status, GtQkv{}, grp, n_experts);

@@ -146,38 +146,114 @@ extern "C" int dl_add_rmsnorm(float* residual, const void* delta, int delta_dtyp
 // A branch output that is normalised before it joins the stream (a layer with a norm behind each
 // sublayer as well as before it), fused with the norm that follows:
 //
-//   residual += delta / sqrt(mean(delta^2) + delta_eps) * delta_gain  (+ extra)
+//   u         = delta + delta_bias
+//   residual += u / sqrt(mean(u^2) + delta_eps) * delta_gain  (+ extra)
 //   out       = residual / sqrt(mean(residual^2) + eps) * gain          (when out is given)
 //
-// One block per row, float32 statistics, a fixed order of additions per row.  `extra` (float32, same
+// One block per row, float32 statistics, a fixed order of additions per row.  `delta_bias` (float32 [width] or NULL) is the
+// bias of the product that made the branch.  `extra` (float32, same
 // shape as the stream, or NULL) is added as it is: the embedding output that a repeated group of
-// layers takes in again before each pass.  Rows of up to 4 * NORM_THREADS values keep the sum in
-// registers between the passes; wider rows go through the stream in memory.
+// layers takes in again before each pass.  Aligned rows of up to 8192 values take the register path: everything the row needs is
+// asked for before the first reduction (the weights ahead of the kernel before this one, where there are registers for
+// them) and read once.  Other rows take the looped path; those of up to BRANCH_MAX * NORM_THREADS values keep the sum in
+// registers between the passes, wider ones go through the stream in memory.
 #define BRANCH_MAX 4
+
+template <typename TDelta, typename TOut, int NV>
+__global__ void __launch_bounds__(NORM_THREADS)
+branch_norm_add_vec_kernel(float* __restrict__ residual, const TDelta* __restrict__ delta, int delta_stride,
+                           const float* __restrict__ delta_bias, const float* __restrict__ delta_gain, float delta_eps,
+                           const float* __restrict__ extra, const float* __restrict__ gain, TOut* __restrict__ out, int width, float eps) {
+    __shared__ float scratch[33];
+    constexpr bool AHEAD = NV <= 4;                          // weights in registers before anything else
+    dl_launch_dependents();
+    const int n_vec = width / 4;
+    const size_t base = (size_t)blockIdx.x * width;
+    const TDelta* drow = delta + (size_t)blockIdx.x * delta_stride;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 dg[AHEAD ? NV : 1], gn[AHEAD ? NV : 1];
+    if (AHEAD) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int c = threadIdx.x + i * NORM_THREADS;
+            dg[AHEAD ? i : 0] = c < n_vec ? Vec4<float>::load(delta_gain + 4 * c) : zero;
+            gn[AHEAD ? i : 0] = c < n_vec && out != nullptr ? Vec4<float>::load(gain + 4 * c) : zero;
+        }
+    }
+    dl_grid_dependency_wait();
+    float4 d[NV], r[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = threadIdx.x + i * NORM_THREADS;
+        d[i] = c < n_vec ? Vec4<TDelta>::load(drow + 4 * c) : zero;
+        r[i] = c < n_vec ? Vec4<float>::load(residual + base + 4 * c) : zero;
+    }
+    if (delta_bias != nullptr) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int c = threadIdx.x + i * NORM_THREADS;
+            const float4 b = c < n_vec ? Vec4<float>::load(delta_bias + 4 * c) : zero;
+            d[i].x += b.x; d[i].y += b.y; d[i].z += b.z; d[i].w += b.w;
+        }
+    }
+    float ssd = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) ssd += d[i].x * d[i].x + d[i].y * d[i].y + d[i].z * d[i].z + d[i].w * d[i].w;
+    ssd = dl_block_sum(ssd, scratch);
+    const float ds = 1.0f / sqrtf(ssd / (float)width + delta_eps);
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = threadIdx.x + i * NORM_THREADS;
+        if (c < n_vec) {
+            const float4 w = AHEAD ? dg[AHEAD ? i : 0] : Vec4<float>::load(delta_gain + 4 * c);
+            r[i].x += d[i].x * ds * w.x; r[i].y += d[i].y * ds * w.y; r[i].z += d[i].z * ds * w.z; r[i].w += d[i].w * ds * w.w;
+            if (extra != nullptr) {
+                const float4 x = Vec4<float>::load(extra + base + 4 * c);
+                r[i].x += x.x; r[i].y += x.y; r[i].z += x.z; r[i].w += x.w;
+            }
+            Vec4<float>::store(residual + base + 4 * c, r[i]);
+            ss += r[i].x * r[i].x + r[i].y * r[i].y + r[i].z * r[i].z + r[i].w * r[i].w;
+        }
+    }
+    if (out == nullptr) return;
+    ss = dl_block_sum(ss, scratch);
+    const float scale = 1.0f / sqrtf(ss / (float)width + eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = threadIdx.x + i * NORM_THREADS;
+        if (c < n_vec) {
+            const float4 w = AHEAD ? gn[AHEAD ? i : 0] : Vec4<float>::load(gain + 4 * c);
+            Vec4<TOut>::store(out + base + 4 * c, make_float4(r[i].x * scale * w.x, r[i].y * scale * w.y, r[i].z * scale * w.z,
+                                                              r[i].w * scale * w.w));
+        }
+    }
+}
 
 template <typename TDelta, typename TOut>
 __global__ void __launch_bounds__(NORM_THREADS)
 branch_norm_add_kernel(float* __restrict__ residual, const TDelta* __restrict__ delta, int delta_stride,
-                       const float* __restrict__ delta_gain, float delta_eps, const float* __restrict__ extra,
-                       const float* __restrict__ gain, TOut* __restrict__ out, int width, float eps) {
+                       const float* __restrict__ delta_bias, const float* __restrict__ delta_gain, float delta_eps,
+                       const float* __restrict__ extra, const float* __restrict__ gain, TOut* __restrict__ out, int width, float eps) {
     __shared__ float scratch[33];
     dl_launch_dependents();
     dl_grid_dependency_wait();
     const size_t base = (size_t)blockIdx.x * width;
     const TDelta* drow = delta + (size_t)blockIdx.x * delta_stride;
     const bool in_regs = width <= BRANCH_MAX * NORM_THREADS;
+    auto branch = [&](int c) { return dl_to_f32<TDelta>(drow[c]) + (delta_bias != nullptr ? delta_bias[c] : 0.f); };
     float d[BRANCH_MAX];
     float ssd = 0.f;
     if (in_regs) {
 #pragma unroll
         for (int i = 0; i < BRANCH_MAX; ++i) {
             const int c = threadIdx.x + i * NORM_THREADS;
-            d[i] = c < width ? dl_to_f32<TDelta>(drow[c]) : 0.f;
+            d[i] = c < width ? branch(c) : 0.f;
             ssd += d[i] * d[i];
         }
     } else {
         for (int c = threadIdx.x; c < width; c += NORM_THREADS) {
-            const float v = dl_to_f32<TDelta>(drow[c]);
+            const float v = branch(c);
             ssd += v * v;
         }
     }
@@ -198,7 +274,7 @@ branch_norm_add_kernel(float* __restrict__ residual, const TDelta* __restrict__ 
         }
     } else {
         for (int c = threadIdx.x; c < width; c += NORM_THREADS) {
-            float v = residual[base + c] + dl_to_f32<TDelta>(drow[c]) * dscale * delta_gain[c];
+            float v = residual[base + c] + branch(c) * dscale * delta_gain[c];
             if (extra != nullptr) v += extra[base + c];
             residual[base + c] = v;
             ss += v * v;
@@ -220,19 +296,31 @@ branch_norm_add_kernel(float* __restrict__ residual, const TDelta* __restrict__ 
 }
 
 template <typename TDelta, typename TOut>
-static int launch_branch(float* residual, const void* delta, int delta_stride, const float* delta_gain, float delta_eps,
-                         const float* extra, const float* gain, void* out, int rows, int width, float eps, cudaStream_t s) {
-    cudaError_t e = dl_launch_dependent(branch_norm_add_kernel<TDelta, TOut>, dim3(rows), dim3(NORM_THREADS), 0, s, residual,
-                                        (const TDelta*)delta, delta_stride, delta_gain, delta_eps, extra, gain, (TOut*)out,
-                                        width, eps);
+static int launch_branch(float* residual, const void* delta, int delta_stride, const float* delta_bias, const float* delta_gain,
+                         float delta_eps, const float* extra, const float* gain, void* out, int rows, int width, float eps, cudaStream_t s) {
+    const uintptr_t places = (uintptr_t)residual | (uintptr_t)delta | (uintptr_t)delta_bias | (uintptr_t)delta_gain | (uintptr_t)extra |
+                             (uintptr_t)gain | (uintptr_t)out;
+    const bool vec = places % 16 == 0 && width % 4 == 0 && delta_stride % 4 == 0 && width <= 4 * NORM_THREADS * NORM_MAX_VEC;
+    const TDelta* d = (const TDelta*)delta;
+    TOut* o = (TOut*)out;
+    cudaError_t e;
+    const dim3 grid(rows), block(NORM_THREADS);
+#define BN_GO(KERNEL) e = dl_launch_dependent(KERNEL, grid, block, 0, s, residual, d, delta_stride, delta_bias, delta_gain, delta_eps, extra, gain, o, width, eps)
+    const int per_thread = (width + 4 * NORM_THREADS - 1) / (4 * NORM_THREADS);
+    if (!vec) BN_GO((branch_norm_add_kernel<TDelta, TOut>));
+    else if (per_thread <= 1) BN_GO((branch_norm_add_vec_kernel<TDelta, TOut, 1>));
+    else if (per_thread <= 2) BN_GO((branch_norm_add_vec_kernel<TDelta, TOut, 2>));
+    else if (per_thread <= 4) BN_GO((branch_norm_add_vec_kernel<TDelta, TOut, 4>));
+    else BN_GO((branch_norm_add_vec_kernel<TDelta, TOut, 8>));
+#undef BN_GO
     if (e != cudaSuccess) return dl_fail(DL_ERR_LAUNCH, "branch_norm_add: %s", cudaGetErrorString(e));
     return DL_OK;
 }
 
 // residual float32 [rows, width] contiguous, updated in place; delta [rows, width] of delta_dtype, rows
-// delta_stride elements apart; delta_gain, gain float32 [width]; extra float32 [rows, width] or NULL;
+// delta_stride elements apart; delta_bias float32 [width] or NULL; delta_gain, gain float32 [width]; extra float32 [rows, width] or NULL;
 // out [rows, width] of out_dtype or NULL (then gain may be NULL too: the stream is only added to).
-extern "C" int dl_branch_norm_add(float* residual, const void* delta, int delta_dtype, int delta_stride,
+extern "C" int dl_branch_norm_add(float* residual, const void* delta, int delta_dtype, int delta_stride, const float* delta_bias,
                                   const float* delta_gain, float delta_eps, const float* extra, const float* gain,
                                   void* out, int out_dtype, int rows, int width, float eps, void* stream) {
     DL_REQUIRE(rows >= 0 && width > 0 && delta_stride >= width, "branch_norm_add: bad sizes rows=%d width=%d", rows, width);
@@ -242,10 +330,27 @@ extern "C" int dl_branch_norm_add(float* residual, const void* delta, int delta_
     const bool df = (delta_dtype == DL_F32), of = (out_dtype == DL_F32);
     DL_REQUIRE(df || delta_dtype == DL_BF16, "branch_norm_add: delta dtype %d", delta_dtype);
     DL_REQUIRE(of || out_dtype == DL_BF16, "branch_norm_add: out dtype %d", out_dtype);
-    if (df && of) return launch_branch<float, float>(residual, delta, delta_stride, delta_gain, delta_eps, extra, gain, out, rows, width, eps, s);
-    if (df && !of) return launch_branch<float, __nv_bfloat16>(residual, delta, delta_stride, delta_gain, delta_eps, extra, gain, out, rows, width, eps, s);
-    if (!df && of) return launch_branch<__nv_bfloat16, float>(residual, delta, delta_stride, delta_gain, delta_eps, extra, gain, out, rows, width, eps, s);
-    return launch_branch<__nv_bfloat16, __nv_bfloat16>(residual, delta, delta_stride, delta_gain, delta_eps, extra, gain, out, rows, width, eps, s);
+    if (df && of) return launch_branch<float, float>(residual, delta, delta_stride, delta_bias, delta_gain, delta_eps, extra, gain, out, rows, width, eps, s);
+    if (df && !of) return launch_branch<float, __nv_bfloat16>(residual, delta, delta_stride, delta_bias, delta_gain, delta_eps, extra, gain, out, rows, width, eps, s);
+    if (!df && of) return launch_branch<__nv_bfloat16, float>(residual, delta, delta_stride, delta_bias, delta_gain, delta_eps, extra, gain, out, rows, width, eps, s);
+    return launch_branch<__nv_bfloat16, __nv_bfloat16>(residual, delta, delta_stride, delta_bias, delta_gain, delta_eps, extra, gain, out, rows, width, eps, s);
+}
+
+// x[r, :] += bias[:], float32, in place: a branch whose bias no norm behind it takes in.
+__global__ void __launch_bounds__(256) add_bias_kernel(float* __restrict__ x, const float* __restrict__ bias, size_t n, int width) {
+    dl_launch_dependents();
+    dl_grid_dependency_wait();
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) x[i] += bias[i % width];
+}
+
+extern "C" int dl_add_bias(float* x, const float* bias, int rows, int width, void* stream) {
+    DL_REQUIRE(rows >= 0 && width > 0 && x != nullptr && bias != nullptr, "add_bias: bad arguments");
+    if (rows == 0) return DL_OK;
+    const size_t n = (size_t)rows * width;
+    const int blocks = (int)((n + 255) / 256 < 148 * 8 ? (n + 255) / 256 : 148 * 8);
+    cudaError_t e = dl_launch_dependent(add_bias_kernel, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, x, bias, n, width);
+    if (e != cudaSuccess) return dl_fail(DL_ERR_LAUNCH, "add_bias: %s", cudaGetErrorString(e));
+    return DL_OK;
 }
 
 // Stream += other, float32, elementwise (a stream that takes another in when no norm follows at once).

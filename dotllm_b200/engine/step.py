@@ -66,6 +66,7 @@ class StepContext:
     seq_new: torch.Tensor         # int32 [B]
     cu_new: torch.Tensor          # int32 [B+1]
     packed: Optional[torch.Tensor] = None     # the one int32 device buffer all of the above are views of
+    carry: dict = field(default_factory=dict) # what a layer hands to later layers of the same step (values that others mix in, say)
 
 
 PROMPT_PAD_LIMIT = 1024         # prompts (or chunks) of more tokens than this run at their own length in a captured step

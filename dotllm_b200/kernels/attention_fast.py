@@ -13,16 +13,16 @@ from . import library as _library
 
 _P, _I, _F = _library._P, _library._I, _library._F
 _library.register_signatures({
-    "dl_attention_decode_bf16": [_P, _I, _P, _I, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _P, _F, _I, _I,
+    "dl_attention_decode_bf16": [_P, _I, _P, _I, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _P, _F, _P, _P, _I, _I, _I,
                                  _P, _P, _I, _P, _I, _P, _P],
     "dl_attention_decode_fresh_bf16": [_P, _I, _P, _I, _P, _I, _P, _P, _I, _I, _P, _I, _P, _P, _I, _P, _P, _I, _I, _I, _I,
                                        _I, _F, _I, _I, _P, _P, _I, _P, _I, _P, _P],
-    "dl_attention_decode_gated_bf16": [_P, _I, _P, _I, _P, _I, _P, _P, _I, _I, _P, _P, _P, _P, _I, _P, _F, _I, _P, _I, _P, _P, _I, _P, _P, _I, _I,
+    "dl_attention_decode_gated_bf16": [_P, _I, _P, _I, _P, _I, _P, _P, _I, _I, _P, _P, _P, _P, _I, _P, _F, _P, _I, _P, _I, _P, _P, _I, _P, _P, _I, _I,
                                        _I, _I, _I, _F, _I, _I, _P, _P, _I, _P, _I, _P, _P],
     "dl_attention_prefill_bf16": [_P, _I, _P, _I, _P, _P, _I, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I,
-                                  _F, _I, _I, _P, _F, _P, _P],
+                                  _F, _I, _I, _P, _F, _P, _P, _I, _P, _P],
     "dl_attention_prefill_tc_bf16": [_P, _I, _I, _P, _I, _P, _P, _I, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I,
-                                     _F, _I, _I, _P, _F, _P, _P],
+                                     _F, _I, _I, _P, _F, _P, _P, _I, _P, _P],
 })
 
 PREFILL_ROWS = 128       # query rows per block of the mma.sync prefill kernel (AP_ROWS)
@@ -52,8 +52,15 @@ def decode_tiles(n_heads, n_kv_heads, split=True):
     return n_kv_heads * next(p for p in range(1, group + 1) if group % p == 0 and group // p <= 16)
 
 
+def _gate_args(gate):
+    """(pointer, row stride) of a gate [T, n_heads], or of none."""
+    if gate is None:
+        return None, 0
+    return gate.data_ptr(), gate.stride(0) if gate.shape[0] > 1 else max(gate.stride(0), gate.shape[1])
+
+
 def _decode(q, q_stride, out, k_pool, v_pool, n_pages, block_table, n_heads, n_kv_heads, head_dim,
-            scale, window, plan, keep_first=0, sinks=None, softcap=0.0):
+            scale, window, plan, keep_first=0, sinks=None, softcap=0.0, slopes=None, gate=None):
     B = plan.n_seqs
     tiles = decode_tiles(n_heads, n_kv_heads)
     group = n_heads // tiles
@@ -62,7 +69,8 @@ def _decode(q, q_stride, out, k_pool, v_pool, n_pages, block_table, n_heads, n_k
     _library.call("dl_attention_decode_bf16", q.data_ptr(), q_stride, out.data_ptr(), out.stride(0),
                   k_pool.data_ptr(), v_pool.data_ptr(), n_pages, plan.seq_total.data_ptr(),
                   block_table.data_ptr(), block_table.shape[1], B, n_heads, tiles, head_dim,
-                  scale, window, int(keep_first), None if sinks is None else sinks.data_ptr(), float(softcap), n_kv_heads, DECODE_BLOCKS,
+                  scale, window, int(keep_first), None if sinks is None else sinks.data_ptr(), float(softcap),
+                  None if slopes is None else slopes.data_ptr(), *_gate_args(gate), n_kv_heads, DECODE_BLOCKS,
                   part_o.data_ptr(), part_ml.data_ptr(), slots, counters.data_ptr(), counters.numel(),
                   _library.status_word(q.device).data_ptr(), _library.current_stream())
     return True
@@ -94,13 +102,13 @@ FRESH_ROTATE_HEAD_DIMS = (64, 128)   # head sizes whose rotation the decode kern
 
 
 def decode_fresh(q, k, v, cos, sin, rotary_dim, block_table, k_pool, v_pool, n_heads, n_kv_heads, head_dim,
-                 scale, window, plan, biases=None, gate=None, sinks=None, softcap=0.0, split=False):
+                 scale, window, plan, biases=None, gate=None, sinks=None, softcap=0.0, split=False, slopes=None):
     """A decode step with the new token handled inside the attention kernel (rotation of q and k,
     cache write, attention): returns the output, or None when the sizes are not the kernel's.
     ``biases`` (q, k, v: float32 vectors or None) are added before the rotation and ``gate`` ([B, n_heads] logits of
     q's dtype, a column view is fine) multiplies each head's output by its sigmoid, both inside the kernel; with them
     k and v may be None (a layer that reads another's cache: only the queries are biased and rotated).  ``sinks``,
-    ``softcap`` and ``split`` as in ``run``."""
+    ``softcap``, ``slopes`` and ``split`` as in ``run``."""
     tiles = decode_tiles(n_heads, n_kv_heads, split)
     if tiles == 0:
         return None
@@ -110,7 +118,7 @@ def decode_fresh(q, k, v, cos, sin, rotary_dim, block_table, k_pool, v_pool, n_h
                                                                       and head_dim in FRESH_ROTATE_HEAD_DIMS))):
         return None
     rows = lambda t: t.stride(0) if t.shape[0] > 1 else max(t.stride(0), t.shape[1])
-    extras = biases is not None or gate is not None or sinks is not None or softcap > 0 or tiles != n_kv_heads
+    extras = biases is not None or gate is not None or sinks is not None or softcap > 0 or slopes is not None or tiles != n_kv_heads
     if k is None and not extras:
         return None
     qs = rows(q)
@@ -136,7 +144,7 @@ def decode_fresh(q, k, v, cos, sin, rotary_dim, block_table, k_pool, v_pool, n_h
         _library.call("dl_attention_decode_gated_bf16", q.data_ptr(), qs, ptr(k), ks, ptr(v), vs,
                       cos.data_ptr() if rotary_dim else None, sin.data_ptr() if rotary_dim else None,
                       cos.shape[0] if rotary_dim else 0, 1 if rotary_dim else 0, ptr(qb), ptr(kb) if k is not None else None,
-                      ptr(vb) if k is not None else None, ptr(gate), rows(gate) if gate is not None else 0, ptr(sinks), float(softcap), n_kv_heads,
+                      ptr(vb) if k is not None else None, ptr(gate), rows(gate) if gate is not None else 0, ptr(sinks), float(softcap), ptr(slopes), n_kv_heads,
                       out.data_ptr(), out.stride(0), k_pool.data_ptr(), v_pool.data_ptr(), k_pool.shape[0],
                       plan.seq_total.data_ptr(), block_table.data_ptr(), block_table.shape[1], B, n_heads, tiles, head_dim,
                       scale, window, DECODE_BLOCKS, part_o.data_ptr(), part_ml.data_ptr(), slots, counters.data_ptr(),
@@ -153,9 +161,9 @@ def decode_fresh(q, k, v, cos, sin, rotary_dim, block_table, k_pool, v_pool, n_h
 
 
 def _prefill(q, q_stride, out, k_pool, v_pool, n_pages, block_table, n_heads, n_kv_heads, head_dim,
-             scale, window, plan, keep_first=0, sinks=None, softcap=0.0):
+             scale, window, plan, keep_first=0, sinks=None, softcap=0.0, slopes=None, gate=None):
     tc = PREFILL_TC and head_dim in PREFILL_TC_HEAD_DIMS and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0 \
-        and (PREFILL_TC_SPECIAL or (not keep_first and sinks is None))
+        and (PREFILL_TC_SPECIAL or (not keep_first and sinks is None)) and (slopes is None or softcap <= 0)
     rows = PREFILL_TC_ROWS if tc else PREFILL_ROWS
     if ("prefill_tiles", rows) not in plan.scratch:
         # tiles that see the most keys first: the kernels start blocks in this order, and the short
@@ -174,24 +182,25 @@ def _prefill(q, q_stride, out, k_pool, v_pool, n_pages, block_table, n_heads, n_
                       n_tiles, plan.seq_start.data_ptr(), plan.seq_new.data_ptr(), plan.cu_new.data_ptr(),
                       block_table.data_ptr(), block_table.shape[1], n_heads, n_kv_heads, head_dim, scale, window,
                       int(keep_first), None if sinks is None else sinks.data_ptr(), float(softcap),
-                      _library.status_word(q.device).data_ptr(), _library.current_stream())
+                      None if slopes is None else slopes.data_ptr(), *_gate_args(gate), _library.status_word(q.device).data_ptr(), _library.current_stream())
         return True
     _library.call("dl_attention_prefill_bf16", q.data_ptr(), q_stride, out.data_ptr(), out.stride(0),
                   k_pool.data_ptr(), v_pool.data_ptr(), n_pages, tile_seq.data_ptr(), tile_row0.data_ptr(),
                   n_tiles, plan.seq_start.data_ptr(), plan.seq_new.data_ptr(), plan.cu_new.data_ptr(),
                   block_table.data_ptr(), block_table.shape[1], n_heads, n_kv_heads, head_dim, scale, window,
                   int(keep_first), None if sinks is None else sinks.data_ptr(), float(softcap),
-                  _library.status_word(q.device).data_ptr(), _library.current_stream())
+                  None if slopes is None else slopes.data_ptr(), *_gate_args(gate), _library.status_word(q.device).data_ptr(), _library.current_stream())
     return True
 
 
 def run(q, q_stride, out, k_pool, v_pool, n_pages, token_seq, token_pos, block_table,
-        n_heads, n_kv_heads, head_dim, scale, window, plan, keep_first=0, sinks=None, softcap=0.0, split=False):
+        n_heads, n_kv_heads, head_dim, scale, window, plan, keep_first=0, sinks=None, softcap=0.0, split=False, slopes=None, gate=None):
     """Run a tensor-core kernel into ``out`` and return True, or return False to let the
     generic kernel take the call.  Kept first tokens and sinks are taken by the decode kernel (the kept pages join the
     step's list of pages; the sink's term enters where a head is normalised) and by both prefill kernels (the tcgen05 one
     walks the kept pages ahead of the window's, the mma.sync one lists them per tile).  ``softcap`` c > 0: scaled scores s
-    become c tanh(s / c), in all three.  ``split``: decode steps of more than 16 query heads a KV head run as several tiles of
+    become c tanh(s / c), in all three; then ``slopes`` add slope_h * (key - query), likewise (a prompt with both takes the mma.sync
+    kernel); ``gate`` [T, n_heads] of q's dtype: a head's output times its sigmoid, where it is written.  ``split``: decode steps of more than 16 query heads a KV head run as several tiles of
     query heads over the same pages (otherwise they are the generic kernel's)."""
     if q.dtype != torch.bfloat16 or q_stride % 8 or q.data_ptr() % 16 or head_dim not in DECODE_HEAD_DIMS:
         return False
@@ -203,8 +212,8 @@ def run(q, q_stride, out, k_pool, v_pool, n_pages, token_seq, token_pos, block_t
         if tiles == 0 or not decode_fits(n_heads // tiles, head_dim):
             return False
         return _decode(q, q_stride, out, k_pool, v_pool, n_pages, block_table, n_heads, n_kv_heads,
-                       head_dim, scale, window, plan, keep_first, sinks, softcap)
+                       head_dim, scale, window, plan, keep_first, sinks, softcap, slopes, gate)
     if plan.news and q.shape[0] == sum(plan.news):
         return _prefill(q, q_stride, out, k_pool, v_pool, n_pages, block_table, n_heads, n_kv_heads,
-                        head_dim, scale, window, plan, keep_first, sinks, softcap)
+                        head_dim, scale, window, plan, keep_first, sinks, softcap, slopes, gate)
     return False

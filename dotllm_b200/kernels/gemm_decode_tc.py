@@ -15,7 +15,7 @@ from . import library as _library
 
 _P, _I, _F, _L = _library._P, _library._I, _library._F, ctypes.c_longlong
 _library.register_signatures({
-    "dl_gemm_decode_tc_bf16": [_P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P, _I, _P, _P, _I, _F, _F,
+    "dl_gemm_decode_tc_bf16": [_P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P, _I, _P, _P, _I, _F, _F, _P,
                                _P, _L, _P, _I, _P, _P],
     "dl_gemm_decode_tc_scratch": [_I, _I, _I, _I, _I, _P, _P],
 })
@@ -54,8 +54,8 @@ def takes(x, w, gated=False):
             and w.is_contiguous() and w.data_ptr() % 16 == 0 and (n_out + 127) // 128 <= _MAX_TILES)
 
 
-def run(x, w, out_dtype, fuse_swiglu=False, resident=False, row_sums=None, into=None):
-    """Same contract as ``gemm_skinny.run``; sums of squares are laid out [tile of 128 columns][128]."""
+def run(x, w, out_dtype, fuse_swiglu=False, resident=False, row_sums=None, into=None, bias=None):
+    """Same contract as ``gemm_skinny.run``; ``bias`` (the gated product: float32 [2N]) is added before the gating; sums of squares are laid out [tile of 128 columns][128]."""
     M, K = x.shape
     n_out = w.shape[0] // 2 if fuse_swiglu else w.shape[0]
     counters, partials = _device_state(x.device)
@@ -76,6 +76,6 @@ def run(x, w, out_dtype, fuse_swiglu=False, resident=False, row_sums=None, into=
                   gain.data_ptr() if gain is not None else None, scaled.data_ptr() if scaled is not None else None, n_out,
                   sums_out.data_ptr() if sums_out is not None else None,
                   sums_in.data_ptr() if sums_in is not None else None, parts, 1.0 / width, float(eps),
-                  partials.data_ptr(), partials.numel(), counters.data_ptr(), counters.numel(),
+                  None if bias is None else bias.data_ptr(), partials.data_ptr(), partials.numel(), counters.data_ptr(), counters.numel(),
                   _library.status_word(x.device).data_ptr(), _library.current_stream())
     return result

@@ -18,9 +18,12 @@ PAGE = 64                      # tokens per cache page (DL_PAGE in csrc/common.c
 _P, _I, _F = _library._P, _library._I, _library._F
 _library.register_signatures({
     "dl_embed_positions": [_P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _P],
-    "dl_branch_norm_add": [_P, _P, _I, _I, _P, _F, _P, _P, _P, _I, _I, _I, _F, _P],
+    "dl_embed_pairs": [_P, _P, _I, _P, _P, _P, _P, _P, _P, _I, _I, _P, _I, _I, _I, _I, ctypes.c_longlong, ctypes.c_longlong, _F, _P],
+    "dl_add_bias": [_P, _P, _I, _I, _P],
+    "dl_qkv_rows": [_P, _I, _I, _P, _P, _P, _P, _P, _F, _I, _I, _I, _I, _I, _I, _P, _I, _I, _P, _P, _I, _I, _P],
+    "dl_branch_norm_add": [_P, _P, _I, _I, _P, _P, _F, _P, _P, _P, _I, _I, _I, _F, _P],
     "dl_add_rows": [_P, _P, _I, _I, _P],
-    "dl_gated_activation": [_P, _P, _I, _P, _I, _I, _I, _I, _F, _F, _P],
+    "dl_gated_activation": [_P, _P, _I, _P, _I, _I, _I, _I, _F, _F, _P, _P],
     "dl_gla_scan": [_P, _P, _P, _I, _P, _I, _P, _I, _P, _P, _P, _I, _P, _I, _I, _I, _I, _I, _I, _F, _F, _P],
     "dl_head_norm_gate": [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _F, _I, _P],
     "dl_route_topk": [_P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _I, _F, _P],
@@ -129,6 +132,28 @@ def embed_positions(table, pos_table, ids, positions):
     return out
 
 
+def embed_pairs(table, pairs, step, last, mul_prev, mul_cur, scale=1.0):
+    """out[r] = table[id] * scale + pairs[row] in float32 for the step's packed tokens: row = (before * mul_prev + id * mul_cur) mod
+    buckets with the token before it in its sequence, the last row (number ``buckets`` = pairs' rows - 1) for a sequence's first.
+    table [n, width], pairs [buckets + 1, width] contiguous of one dtype; ``last`` int32 [slots, >= 1]: per slot the last token of
+    what its sequence holds, read and moved on."""
+    _need_cuda(table, pairs, step.tokens, step.token_seq, step.token_pos, step.cu_new, step.slots, last)
+    if table.dim() != 2 or pairs.dim() != 2 or table.shape[1] != pairs.shape[1] or table.dtype != pairs.dtype \
+            or not table.is_contiguous() or not pairs.is_contiguous() or pairs.shape[0] < 2:
+        raise KernelError("embed_pairs: need two contiguous tables of one dtype and one width")
+    if last.dtype != torch.int32 or last.dim() != 2 or last.stride(1) != 1:
+        raise KernelError("embed_pairs: the last tokens must be int32 [slots, n]")
+    for t, what in ((step.tokens, "tokens"), (step.token_seq, "token_seq"), (step.token_pos, "token_pos"), (step.cu_new, "cu_new"),
+                    (step.slots, "slots")):
+        _int32(t, "embed_pairs " + what)
+    rows = step.tokens.numel()
+    out = torch.empty((rows, table.shape[1]), dtype=torch.float32, device=table.device)
+    _library.call("dl_embed_pairs", _ptr(table), _ptr(pairs), _code(table.dtype), _ptr(step.tokens), _ptr(step.token_seq), _ptr(step.token_pos),
+                  _ptr(step.cu_new), _ptr(step.slots), _ptr(last), last.stride(0), last.shape[0], _ptr(out), rows, table.shape[1], table.shape[0],
+                  pairs.shape[0] - 1, int(mul_prev), int(mul_cur), float(scale), _stream())
+    return out
+
+
 # ------------------------------------------------- products not yet launched
 class PendingProduct:
     """x W^T (float32 result of bfloat16 operands) that ``linear(..., lazy=True)`` has not launched
@@ -157,6 +182,33 @@ class PendingProduct:
         return True
 
 
+class Biased:
+    """A branch output whose bias (float32 [H]) has not been added: ``data`` [T, H] is a tensor or a product not yet launched.  A
+    ``NormedBranch`` of it adds the bias in the kernel that normalises the branch; anyone else calls ``tensor()`` (or
+    ``resolve``)."""
+
+    def __init__(self, data, bias):
+        self.data, self.bias = data, bias
+        self.shape = tuple(data.shape)
+        if bias.dtype != torch.float32 or bias.shape != (self.shape[1],) or not bias.is_contiguous():
+            raise KernelError(f"a branch's bias must be contiguous float32 [{self.shape[1]}]")
+
+    def tensor(self):
+        data = resolve(self.data)
+        if data.dtype != torch.float32 or not data.is_contiguous():
+            raise KernelError("a branch's bias is added to contiguous float32 rows")
+        return add_bias(data, self.bias)
+
+
+def add_bias(x, bias):
+    """x += bias per row, in place; x contiguous float32 [T, H], bias float32 [H].  Returns x."""
+    _need_cuda(x, bias)
+    if x.dtype != torch.float32 or x.dim() != 2 or not x.is_contiguous() or bias.dtype != torch.float32 or bias.shape != (x.shape[1],):
+        raise KernelError("add_bias: contiguous float32 rows and one float32 value per column")
+    _library.call("dl_add_bias", _ptr(x), _ptr(bias), x.shape[0], x.shape[1], _stream())
+    return x
+
+
 class ScaledRows:
     """A normalised stream still lacking its factor per row: ``data`` = stream * gain (bfloat16) and the
     sums of squares per part of 16 (the mma.sync product's) or 128 columns (the tcgen05 product's), left by the product that added into the stream.  ``linear``
@@ -178,7 +230,7 @@ class ScaledRows:
 
 class NormedBranch:
     """A branch output that joins the stream only after a norm of its own: ``data`` [T, H] (float32 or
-    bfloat16, or a product not yet launched) is divided by its rows' root mean square (``eps`` inside
+    bfloat16, or a product not yet launched; a ``Biased`` one brings its bias along) is divided by its rows' root mean square (``eps`` inside
     the root) and multiplied by ``gain`` before the addition.  ``extra`` (float32 [T, H] or None) is
     added to the stream as it is at the same time.  ``add_rmsnorm`` takes it as the delta and does
     norm, addition and the next norm in one kernel."""
@@ -200,8 +252,8 @@ class NormedBranch:
 
 
 def resolve(value):
-    """The tensor behind a PendingProduct, ScaledRows or NormedBranch; tensors and None pass through."""
-    return value.tensor() if isinstance(value, (PendingProduct, ScaledRows, NormedBranch)) else value
+    """The tensor behind a PendingProduct, Biased, ScaledRows or NormedBranch; tensors and None pass through."""
+    return value.tensor() if isinstance(value, (PendingProduct, Biased, ScaledRows, NormedBranch)) else value
 
 
 def narrow_rows(value, ids):
@@ -214,6 +266,8 @@ def narrow_rows(value, ids):
         return PendingProduct(gather_rows(x, ids, out_dtype=x.dtype), value.w, value.resident)
     if isinstance(value, (StreamWrite, PostNormed)):
         return value.narrowed(ids)
+    if isinstance(value, Biased):
+        return Biased(narrow_rows(value.data, ids), value.bias)
     if isinstance(value, NormedBranch):
         return NormedBranch(narrow_rows(value.data, ids), value.gain, value.eps,
                             None if value.extra is None else gather_rows(value.extra, ids))
@@ -236,6 +290,7 @@ def add_rmsnorm(residual, delta, gain, eps, out_dtype, lazy=False):
         if fused is not None:
             return fused
         delta = None if delta.add_into(residual) else delta.tensor()
+    delta = resolve(delta)
     _need_cuda(residual, delta, gain)
     if residual.dtype != torch.float32 or residual.dim() != 2 or not residual.is_contiguous():
         raise KernelError("rmsnorm: the residual stream must be contiguous float32 [T, H]")
@@ -254,8 +309,9 @@ def add_rmsnorm(residual, delta, gain, eps, out_dtype, lazy=False):
 def add_normed_branch(residual, branch, gain=None, eps=0.0, out_dtype=None):
     """residual += rmsnorm(branch.data) * branch.gain (+ branch.extra), in place; with ``gain`` also returns
     rmsnorm(residual) * gain in ``out_dtype`` (one kernel), else None."""
-    data = resolve(branch.data)
-    _need_cuda(residual, data, branch.gain, branch.extra, gain)
+    data, bias = (branch.data.data, branch.data.bias) if isinstance(branch.data, Biased) else (branch.data, None)
+    data = resolve(data)
+    _need_cuda(residual, data, bias, branch.gain, branch.extra, gain)
     if residual.dtype != torch.float32 or residual.dim() != 2 or not residual.is_contiguous():
         raise KernelError("normed branch: the residual stream must be contiguous float32 [T, H]")
     rows, width = residual.shape
@@ -269,7 +325,7 @@ def add_normed_branch(residual, branch, gain=None, eps=0.0, out_dtype=None):
     if extra is not None and (extra.dtype != torch.float32 or tuple(extra.shape) != (rows, width) or not extra.is_contiguous()):
         raise KernelError("normed branch: the extra addend must be contiguous float32 with the stream's shape")
     out = torch.empty((rows, width), dtype=out_dtype, device=residual.device) if gain is not None else None
-    _library.call("dl_branch_norm_add", _ptr(residual), _ptr(data), _code(data.dtype), stride, _ptr(branch.gain),
+    _library.call("dl_branch_norm_add", _ptr(residual), _ptr(data), _code(data.dtype), stride, _ptr(bias), _ptr(branch.gain),
                   branch.eps, _ptr(extra), _ptr(gain), _ptr(out), _code(out_dtype) if out is not None else 0, rows, width,
                   float(eps), _stream())
     return out
@@ -370,6 +426,38 @@ def group_rmsnorm(x, gain, width_a, width_b, eps):
     _library.call("dl_group_rmsnorm", _ptr(x), _rows_view(x, "group_rmsnorm x"), _ptr(out), out.stride(0), _code(x.dtype), _ptr(gain),
                   x.shape[0], int(width_a), int(width_b), float(eps), _stream())
     return out
+
+
+def qkv_rows(x, n_heads, n_kv_heads, dim, vdim, lay_k, lay_v, biases=None, gains=None, eps=0.0, first=None, mix=None):
+    """The rows of a stacked query/key/value product made ready for attention and cache, in one kernel: x [T, H*dim + G*(dim + vdim)]
+    (a column view is fine) plus ``biases`` (q, k, v: float32 vectors, each may be None); the queries and the keys each divided by
+    their root mean square over all heads and multiplied by ``gains`` (q, k: float32 per channel; None: no norm); values v with
+    ``first`` (another layer's values of the same tokens, [T, G*lay] with lay = first.shape[1] / G) and ``mix`` (float32, one
+    number w): (1 - w) v + w first.  Returns (q [T, H*lay_k], k [T, G*lay_k], v [T, G*lay_v]), views of one tensor of x's dtype,
+    zeros behind each head's values."""
+    H, G, d, vd = int(n_heads), int(n_kv_heads), int(dim), int(vdim)
+    qb, kb, vb = biases if biases is not None else (None, None, None)
+    qg, kg = gains if gains is not None else (None, None)
+    _need_cuda(x, qb, kb, vb, qg, kg, first, mix)
+    T = x.shape[0]
+    if x.dim() != 2 or x.shape[1] != H * d + G * (d + vd):
+        raise KernelError(f"qkv_rows: rows of {H * d + G * (d + vd)} values, got {tuple(x.shape)}")
+    for t, n, what in ((qb, H * d, "q bias"), (kb, G * d, "k bias"), (vb, G * vd, "v bias"), (qg, H * d, "q gain"), (kg, G * d, "k gain")):
+        if t is not None and (t.dtype != torch.float32 or t.shape != (n,) or not t.is_contiguous()):
+            raise KernelError(f"qkv_rows: the {what} must be contiguous float32 [{n}]")
+    first_ld = first_lay = 0
+    if (first is None) != (mix is None):
+        raise KernelError("qkv_rows: mixed values need the other values and their weight")
+    if first is not None:
+        first_ld, first_lay = _rows_view(first, "qkv_rows first"), first.shape[1] // G
+        if first.shape[0] != T or first.dtype != x.dtype or first.shape[1] % G or first_lay < vd or mix.dtype != torch.float32 or mix.numel() != 1:
+            raise KernelError("qkv_rows: the other values are [T, G*lay] of x's dtype, their weight one float32 number")
+    width = (H + G) * lay_k + G * lay_v
+    ld = -(-width // 8) * 8
+    out = torch.empty((T, ld), dtype=x.dtype, device=x.device)
+    _library.call("dl_qkv_rows", _ptr(x), _code(x.dtype), _rows_view(x, "qkv_rows x"), _ptr(qb), _ptr(kb), _ptr(vb), _ptr(qg), _ptr(kg), float(eps),
+                  H, G, d, vd, int(lay_k), int(lay_v), _ptr(first), first_ld, first_lay, _ptr(mix), _ptr(out), ld, T, _stream())
+    return out[:, :H * lay_k], out[:, H * lay_k:(H + G) * lay_k], out[:, (H + G) * lay_k:width]
 
 
 def pair_norm_sum(a, b, gain_a, gain_b, eps, weight_a=0.5, weight_b=0.5):
@@ -568,7 +656,7 @@ def head_gate(o, gate, n_heads, width):
 class ScoreHook:
     """A change of the attention scores before the softmax: ``softcap`` > 0 turns a score s into
     softcap * tanh(s / softcap); ``slopes`` (float32 [n_heads] on the device) then adds
-    slope * (key position - query position).  The tensor-core kernels take the cap; slopes send a mixer to the generic kernel."""
+    slope * (key position - query position).  The tensor-core kernels take both."""
 
     def __init__(self, softcap=0.0, slopes=None):
         self.softcap = float(softcap)
@@ -588,9 +676,9 @@ def attention(q, k_pool, v_pool, token_seq, token_pos, block_table, n_heads, n_k
     q [T, nh*hd] (row-contiguous view); returns [T, nh*vd] of q's dtype (vd = ``value_dim``, default hd).
     ``window`` 0 means every earlier key; w > 0 means the last w keys.  ``plan`` carries the per-step layout
     (sequence lengths, chunking) that the tensor-core kernels need; without one, for sizes
-    they do not take (values of another width than the keys among them), or with a ``score_hook`` that has slopes, the
+    they do not take (values of another width than the keys among them), the
     generic kernel runs.  ``gate`` [T, nh] of q's dtype (a column view is fine): head h's output is multiplied by
-    sigmoid(gate[t, h]) - in the generic kernel's last step, or by ``head_gate`` behind a tensor-core kernel.
+    sigmoid(gate[t, h]) where it is written.
     ``keep_first`` n > 0 (with a window): a sequence's first n keys stay visible when the window has passed them.
     ``sinks`` float32 [nh]: head h's softmax has one more term exp(sinks[h]) in its denominator, with no key and no value.
     ``split``: let a bfloat16 decode step of more than 16 query heads a KV head run as several tiles of query heads over the same
@@ -623,11 +711,11 @@ def attention(q, k_pool, v_pool, token_seq, token_pos, block_table, n_heads, n_k
         if slopes is not None and (slopes.dtype != torch.float32 or slopes.shape != (n_heads,) or not slopes.is_contiguous()
                                    or not slopes.is_cuda):
             raise KernelError(f"attention: a score hook's slopes must be contiguous float32 [{n_heads}] on the device")
-    if plan is not None and q.dtype == torch.bfloat16 and slopes is None and vd == head_dim:
+    if plan is not None and q.dtype == torch.bfloat16 and vd == head_dim:
         if attention_fast.run(q, qs, out, k_pool, v_pool, n_pages, token_seq, token_pos, block_table,
                               n_heads, n_kv_heads, head_dim, float(scale), int(window), plan,
-                              keep_first=int(keep_first), sinks=sinks, softcap=softcap, split=split):
-            return out if gate is None else head_gate(out, gate, n_heads, vd)
+                              keep_first=int(keep_first), sinks=sinks, softcap=softcap, split=split, slopes=slopes, gate=gate):
+            return out
     _library.call("dl_attention_generic", _ptr(q), qs, _ptr(out), out.stride(0), _code(q.dtype),
                   _ptr(k_pool), _ptr(v_pool), n_pages, _ptr(token_seq), _ptr(token_pos),
                   _ptr(block_table), block_table.shape[1], T, n_heads, n_kv_heads, head_dim, vd,
@@ -642,11 +730,12 @@ def rope_cache_attention(q, k, v, cos, sin, rotary_dim, token_seq, token_pos, bl
     decode step (one new token per sequence) with a full-width rotation of head size 64 or 128, or
     with no rotation, runs as one kernel that adds the biases, rotates q, puts the new keys and values into the
     cache, attends and gates the heads; everything else runs the kernels one after the other."""
-    if plan is not None and q.is_cuda and q.dtype == torch.bfloat16 and (not score_hook or score_hook.slopes is None) \
+    if plan is not None and q.is_cuda and q.dtype == torch.bfloat16 \
             and (value_dim or head_dim) == head_dim and (k is not None or biases is not None or gate is not None) and not keep_first:
         out = attention_fast.decode_fresh(q, k, v, cos, sin, rotary_dim, block_table, k_pool, v_pool, n_heads,
                                           n_kv_heads, head_dim, float(scale), int(window), plan, biases=biases, gate=gate, sinks=sinks,
-                                          softcap=score_hook.softcap if score_hook else 0.0, split=split)
+                                          softcap=score_hook.softcap if score_hook else 0.0, split=split,
+                                          slopes=score_hook.slopes if score_hook else None)
         if out is not None:
             return out
     rope_cache_write(q, k, v, cos, sin, rotary_dim, token_seq, token_pos, block_table, k_pool, v_pool,
@@ -697,11 +786,18 @@ GATINGS = {"silu": 0, "gelu_tanh": 1, "clamped_sigmoid": 2, "relu2": 3, "gelu": 
 UNGATED = frozenset({"relu2", "gelu"})      # activations of ONE product, act(u): no gate rows in the matrix ("gelu": the exact, erf form)
 
 
-def gated_activation(gate_up, kind, limit=0.0, alpha=1.0):
+def _gate_bias(bias, two_i, what):
+    if bias is not None and (bias.dtype != torch.float32 or bias.shape != (two_i,) or not bias.is_contiguous()):
+        raise KernelError(f"{what}: the biases must be contiguous float32 [{two_i}]")
+    return bias
+
+
+def gated_activation(gate_up, kind, limit=0.0, alpha=1.0, bias=None):
     """act(gate, up) for gate_up = [gate | up] of shape [T, 2I]; returns [T, I].  ``kind``: "silu"
     (g sigmoid(g) u), "gelu_tanh" (tanh form of gelu(g), times u) or "clamped_sigmoid"
-    (g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit))."""
-    _need_cuda(gate_up)
+    (g' sigmoid(alpha g') (u' + 1) with g' = min(g, limit), u' = clamp(u, -limit, limit)).  ``bias`` (float32 [2I] or None) is
+    added to both halves first."""
+    _need_cuda(gate_up, bias)
     if kind not in GATINGS or kind in UNGATED:
         raise KernelError(f"gated_activation: unknown gating {kind!r}; known: {sorted(set(GATINGS) - UNGATED)}")
     if gate_up.dim() != 2 or gate_up.shape[1] % 2 or not gate_up.is_contiguous():
@@ -710,7 +806,8 @@ def gated_activation(gate_up, kind, limit=0.0, alpha=1.0):
     width = two_i // 2
     out = torch.empty((rows, width), dtype=gate_up.dtype, device=gate_up.device)
     _library.call("dl_gated_activation", gate_up.data_ptr(), gate_up.data_ptr() + width * gate_up.element_size(), two_i,
-                  _ptr(out), _code(gate_up.dtype), rows, width, GATINGS[kind], float(limit), float(alpha), _stream())
+                  _ptr(out), _code(gate_up.dtype), rows, width, GATINGS[kind], float(limit), float(alpha),
+                  _ptr(_gate_bias(bias, two_i, "gated_activation")), _stream())
     return out
 
 
@@ -1280,23 +1377,31 @@ def softcap(values, cap):
     return values
 
 
-def gated_linear(x, w_gate_up, resident=False, kind="silu", limit=0.0, alpha=1.0):
+def gated_linear(x, w_gate_up, resident=False, kind="silu", limit=0.0, alpha=1.0, bias=None):
     """silu(x Wg^T) * (x Wu^T) for W = [Wg; Wu] of shape [2I, K]; returns [T, I] in x's dtype.
     In bfloat16 one kernel does the product and the gating in float32: the weight-streaming
     kernel for a few rows, the tcgen05 kernel for many.  In float32 the product is followed by
     the gating kernel.  ``kind``: another gating of ``GATINGS`` instead of silu; the weight-streaming
     product (up to 10 rows) and the tcgen05 product (17 rows and more) have it in their epilogues too; the rows
-    between, and float32, run the product and then ``gated_activation``."""
-    if kind != "silu":
+    between, and float32, run the product and then ``gated_activation``.  ``bias`` (float32 [2I]): added to the two products
+    before the gating, in the same epilogues (silu: also in the tcgen05 kernel for 11 to 128 rows)."""
+    if bias is not None:
+        _gate_bias(bias, w_gate_up.shape[0], "gated_linear")
+    if kind == "silu" and bias is not None and not isinstance(x, ScaledRows) and x.dtype == torch.bfloat16 and x.dim() == 2 \
+            and w_gate_up.dim() == 2 and x.shape[1] == w_gate_up.shape[1] and gemm_skinny.SKINNY_ROWS < x.shape[0] \
+            and gemm_skinny.takes(x, w_gate_up, True):
+        _need_cuda(x, w_gate_up, bias)
+        return gemm_skinny.gemm_decode_tc.run(x, w_gate_up, x.dtype, True, resident, bias=bias)
+    if kind != "silu" or bias is not None:
         x = resolve(x) if isinstance(x, ScaledRows) else x
         _need_cuda(x, w_gate_up)
         if x.dtype == torch.bfloat16 and w_gate_up.dim() == 2 and x.dim() == 2 and x.shape[1] == w_gate_up.shape[1] \
                 and w_gate_up.is_contiguous() and w_gate_up.shape[0] % 2 == 0 and x.shape[0] > 0:
             if gemm_skinny.takes_gating(x, w_gate_up):
-                return gemm_skinny.run_gating(x, w_gate_up, GATINGS[kind], limit, alpha, resident=resident)
+                return gemm_skinny.run_gating(x, w_gate_up, GATINGS[kind], limit, alpha, resident=resident, bias=bias)
             if gemm_tc.takes(x, w_gate_up, fuse_swiglu=True):
-                return gemm_tc.run_gated(x, w_gate_up, GATINGS[kind], limit, alpha)
-        return gated_activation(linear(x, w_gate_up, resident=resident), kind, limit, alpha)
+                return gemm_tc.run_gated(x, w_gate_up, GATINGS[kind], limit, alpha, bias=bias)
+        return gated_activation(linear(x, w_gate_up, resident=resident), kind, limit, alpha, bias=bias)
     if isinstance(x, ScaledRows):
         if w_gate_up.dim() == 2 and x.shape[1] == w_gate_up.shape[1] and gemm_skinny.takes(x.data, w_gate_up, True):
             _need_cuda(x.data, w_gate_up)

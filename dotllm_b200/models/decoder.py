@@ -92,16 +92,23 @@ class DecoderModel:
 
     # --------------------------------------------------------------- cache
     def cache_needs(self):
-        return [self.blocks[e.layer].cache_need() for e in self.spec.schedule]
+        """What every execution of the schedule keeps, in its order, and behind them what the embedding keeps (if it does)."""
+        needs = [self.blocks[e.layer].cache_need() for e in self.spec.schedule]
+        need = self.embedding.cache_need()
+        return needs if need is None else needs + [need]
 
     def new_cache(self, max_tokens, max_sequences=None):
-        return ModelCache(self.cache_needs(), [e.cache_of for e in self.spec.schedule], self.runtime,
-                          max_tokens, max_sequences)
+        needs = self.cache_needs()
+        cache_of = [e.cache_of for e in self.spec.schedule]
+        return ModelCache(needs, cache_of + [None] * (len(needs) - len(cache_of)), self.runtime, max_tokens, max_sequences)
 
     # ------------------------------------------------------------- forward
     def forward(self, step, cache):
         """Logits float32 [wanted rows, vocab] of one step (see engine.step)."""
-        residual = self.embedding.forward(step)
+        if self.embedding.cache_need() is None:
+            residual = self.embedding.forward(step)
+        else:
+            residual = self.embedding.forward(step, cache.view(len(self.spec.schedule), step.block_tables, step.slots))
         pending = None
         # the embedding output, for executions that take it in again (the stream itself is updated in place)
         embedded = residual.clone() if any(e.takes_embedding for e in self.spec.schedule) else None

@@ -19,7 +19,15 @@ with a gain per channel (``qk_norm`` with ``over`` "projection"); a window that 
 (``keep_first``); a learned number per head in the softmax's denominator, a sink without key or value (``sink``), or a sink
 of score zero without a tensor (``sink`` "zero": one is added to the denominator); a rotation that pairs channel 2i
 with 2i + 1 (``pairing`` "interleaved"); and a gate per output channel (``gate`` "channel_sigmoid": the concatenated heads
-times sigmoid of a projection of the mixer's input as wide as they are, behind the attention).
+times sigmoid of a projection of the mixer's input as wide as they are, behind the attention); a bias on the output projection
+(``bias`` "all"; the norm that takes the branch in adds it); a penalty per distance (``score`` with ``slopes``: slope_h times the
+distance is taken off a head's scores); and values mixed with another layer's values of the same tokens (``value_mix``).
+
+The rows kernel.  Biases in front of a norm over the whole projections, and mixed values, go through one kernel between the product
+and the attention (``ops.qkv_rows``): it adds the biases, normalises, mixes, and lays every head out at the kernels' width, so the
+stacked matrix keeps its own rows and a mixer of this kind runs on the tensor cores whatever its heads' widths (up to 128).  A
+layer that others mix in leaves its values in the step (``StepContext.carry``): they are values of the step's own tokens, so
+nothing of them outlives it; what is cached are the mixed ones.
 
 Interleaved pairs on kernels that pair channel i with i + r/2.  Scores do not change when the channels of q and k are
 permuted alike, so for a rotation of the first r channels in interleaved pairs the rows of the q and k projections (and
@@ -65,20 +73,22 @@ class AttentionMixer(Mixer):
     """params: ``n_heads``, ``n_kv_heads``, ``head_dim``, ``window`` (None = all keys),
     ``position`` ({"kind", "params"} of a position encoding), optional ``scale``, optional ``score``
     ({"softcap": c, "slopes": [one per head]}: scores are capped and biased by distance before the
-    softmax; slopes send the mixer to the generic attention kernel); optional ``value_dim`` (per head, default
+    softmax); optional ``value_dim`` (per head, default
     ``head_dim``), ``bias`` (True: q, k and v have biases), ``gate`` (None, "head_sigmoid" or "channel_sigmoid"), ``own_kv`` (False: no key
     and value projections, the layer reads another's cache) and ``tensors``: the local names of ``q``, ``k``, ``v``,
-    ``o``, ``gate`` and the bias suffix ``bias`` (appended to a projection's name); optional ``values`` ("own", or "keys":
+    ``o``, ``gate`` and the biases (``q_bias`` and so on); optional ``values`` ("own", or "keys":
     v is k as projected, there is no value projection and ``value_dim`` is ``head_dim``), ``qk_norm`` ({"eps"}: tensors
     ``q_norm``, ``k_norm`` [head_dim]), ``keep_first`` (with a window: that many first tokens of a sequence stay visible) and
     ``sink`` (True: tensor ``sink`` [n_heads], exp(sink_h) joins head h's softmax denominator; "zero": no tensor, every
     head's denominator gets exp(0) = 1 more); ``qk_norm`` may carry ``over`` "projection" (one RMS over all the query
     channels of a token and one over all its key channels, tensors ``q_norm`` [n_heads * head_dim], ``k_norm``
-    [n_kv_heads * head_dim]); ``pairing`` ("half", or "interleaved": the rotation pairs channel 2i with 2i + 1)."""
+    [n_kv_heads * head_dim]); ``pairing`` ("half", or "interleaved": the rotation pairs channel 2i with 2i + 1); ``bias`` "all": the output projection has one
+    too; ``value_mix`` {"first": True}: later layers mix this one's values in, {"first": False}: v becomes (1 - w) v + w v_first with
+    w the tensor ``mix``, one number (``key`` names the values in the step, where several groups of layers mix)."""
 
     NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
              "gate": "g_proj.weight", "q_bias": "q_proj.bias", "k_bias": "k_proj.bias", "v_bias": "v_proj.bias",
-             "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "sink": "sinks"}
+             "o_bias": "o_proj.bias", "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "sink": "sinks", "mix": "v_mix"}
     GATES = (None, "head_sigmoid", "channel_sigmoid")
     stacks = True
     ROW_STEP = 16                # the stacked matrix's rows are a multiple of this: its product's rows stay 16-byte aligned
@@ -105,6 +115,11 @@ class AttentionMixer(Mixer):
                                                                                  device=runtime.device))
         self.value_dim = int(params.get("value_dim") or self.head_dim)
         self.bias = bool(params.get("bias", False))
+        self.out_bias = params.get("bias") == "all"
+        mix = params.get("value_mix")
+        self.mixes = mix is not None and not mix.get("first")
+        self.mixed_in = mix is not None and bool(mix.get("first"))
+        self.mix_key = ("values", str((mix or {}).get("key", "")))
         self.gate = params.get("gate")
         self.channel_gate = self.gate == "channel_sigmoid"
         if self.gate not in self.GATES:
@@ -134,29 +149,36 @@ class AttentionMixer(Mixer):
         self.kv_dim = self.n_kv_heads * self.head_dim
         self.v_width = self.n_kv_heads * self.value_dim
         self.o_dim = self.n_heads * self.value_dim
+        # biases ahead of a norm over the projections, and mixed values, are the rows kernel's (see the module's text)
+        self.rows_kernel = mix is not None or (self.bias and self.qk_norm_over == "projection")
+        if self.rows_kernel and (not self.own_kv or self.values != "own" or self.qk_norm_over == "head" or self.pairing != "half"):
+            raise ConfigError("attention: biases ahead of a norm and mixed values go with keys and values of the layer's own, norms over whole "
+                              "projections or none, and half pairs")
         # the reference's block as it is (one matrix of q, k and v rows, nothing added): its fused paths apply
         self.plain = not self.bias and self.gate is None and self.value_dim == self.head_dim and self.own_kv \
             and self.values == "own" and self.qk_norm_eps is None and not self.sink and not self.keep_first \
-            and params.get("pairing", "half") == "half"
+            and params.get("pairing", "half") == "half" and mix is None
         self.w_qkv = None
         self.w_o = None
-        self.biases = None
+        self.biases = self.o_bias = self.mix = None
+        self.stacks = not self.out_bias                    # a product shared with another mixer has no place for one side's bias
         fused = self.position.fused_rotary()         # (cos, sin, r)
         rd = int(fused[2]) if fused is not None else 0
         # a norm per head writes its result wherever the kernels want it: queries and keys that no rotation follows may be
         # projected at their stored width and laid out by the norm
         self.norm_lays = self.qk_norm_over == "head" and fused is not None and rd == 0 and self.values == "own"
         # heads keep their own width and channel order where a norm runs over them or the keys double as values
-        as_stored = self.values == "keys" or (self.qk_norm_eps is not None and not self.norm_lays) or params.get("pairing") == "interleaved"
+        as_stored = self.values == "keys" or (self.qk_norm_eps is not None and not self.norm_lays and not self.rows_kernel) \
+            or params.get("pairing") == "interleaved"
         # the width every head is laid out at (see the module's text); head_dim / value_dim stay the stored widths
         self.lay_k, self.lay_v = self.head_dim, self.value_dim
         if runtime.dtype == torch.bfloat16 and not self.plain and not as_stored and \
                 (self.value_dim != self.head_dim or self.head_dim not in self.TENSOR_CORE_WIDTHS):
             fits = [w for w in self.TENSOR_CORE_WIDTHS if w >= max(self.head_dim, self.value_dim)]
-            if fits and self.n_heads // self.n_kv_heads <= 16:
+            if fits and (self.n_heads // self.n_kv_heads <= 16 or self.rows_kernel):
                 self.lay_k = self.lay_v = fits[0]
         # a partial rotation spread over the whole head (see the module's text)
-        self.spread = bool(runtime.dtype == torch.bfloat16 and not self.plain and not as_stored and self.lay_k == self.lay_v
+        self.spread = bool(runtime.dtype == torch.bfloat16 and not self.plain and not as_stored and not self.rows_kernel and self.lay_k == self.lay_v
                            and self.lay_k in self.TENSOR_CORE_WIDTHS and 0 < rd < self.lay_k)
         self.rotation = None if fused is None else (self._wide_tables(fused[0], fused[1], rd, self.lay_k) + (self.lay_k,)
                                                     if self.spread else fused)
@@ -222,6 +244,10 @@ class AttentionMixer(Mixer):
             if self.own_kv:
                 specs[n["k_bias"]] = WeightSpec((self.kv_dim,), "precise", ("normal", 0.1))
                 specs[n["v_bias"]] = WeightSpec((self.v_width,), "precise", ("normal", 0.1))
+        if self.out_bias:
+            specs[n["o_bias"]] = WeightSpec((h,), "precise", ("normal", 0.1))
+        if self.mixes:
+            specs[n["mix"]] = WeightSpec((), "precise", ("uniform", 0.2, 0.8))
         if self.gate:
             specs[n["gate"]] = WeightSpec((self.o_dim if self.channel_gate else self.n_heads, h), init=("normal", 0.1))
         if self.qk_norm_eps is not None:
@@ -234,15 +260,19 @@ class AttentionMixer(Mixer):
         specs[n["o"]] = WeightSpec((h, self.o_dim))
         return specs
 
+    def optional_names(self):
+        return {self.names["mix"]} if self.mixed_in else set()      # the first mixing layer mixes nothing in
+
     def bind(self, tensors):
         n = self.names
         H, G, hd, vd, lk, lv = self.n_heads, self.n_kv_heads, self.head_dim, self.value_dim, self.lay_k, self.lay_v
-        pk = hd if self.norm_lays else lk                  # the width q and k leave the product at
+        pk = hd if self.norm_lays or self.rows_kernel else lk      # the width q and k leave the product at, and v
+        pv = vd if self.rows_kernel else lv
         rows = [self._reorder(self._widen(tensors[n["q"]], H, hd, pk), H)]
         if self.own_kv:
             rows.append(self._reorder(self._widen(tensors[n["k"]], G, hd, pk), G))
             if self.values == "own":
-                rows.append(self._widen(tensors[n["v"]], G, vd, lv))
+                rows.append(self._widen(tensors[n["v"]], G, vd, pv))
         if self.gate:
             rows.append(tensors[n["gate"]])
         self.w_qkv = torch.cat(rows, dim=0).contiguous() if self.plain else pad_rows(rows, self.ROW_STEP)
@@ -263,9 +293,11 @@ class AttentionMixer(Mixer):
         elif self.sink:
             self.sinks = tensors[n["sink"]].contiguous()
         if self.bias:
-            self.biases = (self._reorder(self._widen(tensors[n["q_bias"]], H, hd, lk), H).contiguous(),
-                           self._reorder(self._widen(tensors[n["k_bias"]], G, hd, lk), G).contiguous() if self.own_kv else None,
-                           self._widen(tensors[n["v_bias"]], G, vd, lv).contiguous() if self.own_kv else None)
+            self.biases = (self._reorder(self._widen(tensors[n["q_bias"]], H, hd, pk), H).contiguous(),
+                           self._reorder(self._widen(tensors[n["k_bias"]], G, hd, pk), G).contiguous() if self.own_kv else None,
+                           self._widen(tensors[n["v_bias"]], G, vd, pv).contiguous() if self.own_kv else None)
+        self.o_bias = tensors[n["o_bias"]].contiguous() if self.out_bias else None
+        self.mix = tensors[n["mix"]].reshape(1).contiguous() if self.mixes else None
 
     def weight_bytes(self):
         return (self.w_qkv.numel() + self.w_o.numel()) * self.w_qkv.element_size()
@@ -307,13 +339,32 @@ class AttentionMixer(Mixer):
             a = self.heads(y, step, cache_view)
         else:
             a, _ = self._attend(y, step, cache_view)
-        return ops.linear(a, self.w_o, out_dtype=BRANCH_DTYPE, resident=True, lazy=True)
+        return self._project(a)
+
+    def _project(self, a):
+        y = ops.linear(a, self.w_o, out_dtype=BRANCH_DTYPE, resident=True, lazy=True)
+        return y if self.o_bias is None else ops.Biased(y, self.o_bias)
+
+    def _ready_rows(self, y, step):
+        """Queries, keys and values from the stacked product through the rows kernel: biased, normed, mixed, laid out."""
+        width = self.q_dim + self.kv_dim + self.v_width
+        first = None
+        if self.mixes:
+            first = step.carry.get(self.mix_key)
+            if first is None:
+                raise ConfigError("attention: a layer that mixes values needs a layer before it whose values are mixed in")
+        gains = (self.q_gain, self.k_gain) if self.qk_norm_eps is not None else None
+        q, k, v = ops.qkv_rows(y[:, :width], self.n_heads, self.n_kv_heads, self.head_dim, self.value_dim, self.lay_k, self.lay_v,
+                               biases=self.biases, gains=gains, eps=self.qk_norm_eps or 0.0, first=first, mix=self.mix)
+        if self.mixed_in:
+            step.carry[self.mix_key] = v
+        return q, k, v
 
     def _attend(self, y, step, cache_view):
         """From the stacked product to the heads' outputs [T, n_heads * lay_v] and the logits of a gate per channel (or None)."""
         lk, lv = self.lay_k, self.lay_v
-        pk = self.head_dim if self.norm_lays else lk
-        qd, kvd, vw = self.n_heads * pk, self.n_kv_heads * pk, self.n_kv_heads * lv
+        pk = self.head_dim if self.norm_lays or self.rows_kernel else lk
+        qd, kvd, vw = self.n_heads * pk, self.n_kv_heads * pk, self.v_width if self.rows_kernel else self.n_kv_heads * lv
         q, at = y[:, :qd], qd
         k = v = None
         if self.own_kv and self.values == "keys":
@@ -323,7 +374,11 @@ class AttentionMixer(Mixer):
             k, v, at = y[:, at:at + kvd], y[:, at + kvd:at + kvd + vw], at + kvd + vw
         g = y[:, at:at + self.n_heads] if self.gate == "head_sigmoid" else None
         channel_g = y[:, at:at + self.o_dim] if self.channel_gate else None
-        if self.qk_norm_eps is not None and self.qk_norm_over == "projection":
+        biases = self.biases
+        if self.rows_kernel:
+            q, k, v = self._ready_rows(y, step)
+            biases = None
+        elif self.qk_norm_eps is not None and self.qk_norm_over == "projection":
             if self.own_kv:
                 normed = ops.group_rmsnorm(y[:, :qd + kvd], self.qk_gain, qd, kvd, self.qk_norm_eps)
                 q, k = normed[:, :qd], normed[:, qd:]
@@ -337,7 +392,7 @@ class AttentionMixer(Mixer):
                 q = ops.head_rmsnorm(q, self.q_gain, self.n_heads, pk, self.qk_norm_eps, lay=lk)
         fused = self.rotation
         if fused is None:
-            if self.biases is not None:
+            if biases is not None:
                 raise ConfigError("attention: biases need a position encoding that rides the cache-write kernel")
             self.position.apply(q, k, step.token_pos)
             cos = sin = None
@@ -349,7 +404,8 @@ class AttentionMixer(Mixer):
                                      self.n_heads, self.n_kv_heads, lk, self.scale,
                                      int(self.window or 0), plan=step.attention_plan,
                                      score_hook=self.score_hook if self.score_hook else None,
-                                     value_dim=lv, biases=self.biases, gate=g, keep_first=self.keep_first, sinks=self.sinks)
+                                     value_dim=lv, biases=biases, gate=g, keep_first=self.keep_first, sinks=self.sinks,
+                                     split=self.rows_kernel)
         return a, channel_g
 
     def forward(self, x, step, cache_view):

@@ -119,6 +119,10 @@ class Part:
         """Bytes of weights that one step reads (for the roofline account)."""
         return 0
 
+    def cache_need(self):
+        """What the part keeps per sequence: None, one CacheNeed, or (mixers made of several) a tuple of them."""
+        return None
+
 
 class Norm(Part):
     """``fuses_products``: ``add_forward`` also takes ``lazy=True`` and a delta that is a product not yet

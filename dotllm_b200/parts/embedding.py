@@ -10,7 +10,8 @@ from __future__ import annotations
 import torch
 
 from ..kernels import ops
-from .base import Part, WeightSpec, register_embedding, register_head
+from ..errors import ConfigError
+from .base import CacheNeed, Part, WeightSpec, register_embedding, register_head
 
 
 class TokenEmbedding(Part):
@@ -68,6 +69,43 @@ class TokenPositionEmbedding(Part):
         return ops.embed_positions(self.table, self.positions, step.tokens, step.token_pos)
 
 
+class TokenPairEmbedding(Part):
+    """Token embedding times a constant plus a row for the pair of a token and the one before it:
+    h[t] = E[token t] * scale + B[(token (t-1) * mul_prev + token t * mul_cur) mod buckets], and B[buckets], the last row, for a
+    sequence's first token.  The token before is part of a sequence's state: the cache keeps a sequence's last token in its slot.
+
+    params: ``vocab_size``, ``buckets``, ``mul_prev``, ``mul_cur``; optional ``scale``, ``tensor`` and ``pair_tensor`` (local names,
+    default "weight" and "pairs.weight") and ``init_std`` (of both tables in the random-weights mode)."""
+
+    def __init__(self, params, hidden_size, runtime):
+        super().__init__(params, hidden_size, runtime)
+        self.vocab_size = int(params["vocab_size"])
+        self.buckets = int(params["buckets"])
+        self.mul_prev, self.mul_cur = int(params["mul_prev"]), int(params["mul_cur"])
+        self.scale = float(params.get("scale", 1.0))
+        # (token * multiplier and the sum of two such stay within 64 bits)
+        if self.buckets < 1 or max(abs(self.mul_prev), abs(self.mul_cur)) >= 1 << 31:
+            raise ConfigError("pair embedding: at least one bucket, and multipliers below 2^31")
+        self.token_name = str(params.get("tensor", "weight"))
+        self.pair_name = str(params.get("pair_tensor", "pairs.weight"))
+        self.table = self.pairs = None
+
+    def weight_specs(self):
+        init = ("normal", float(self.params.get("init_std", 0.02)))
+        return {self.token_name: WeightSpec((self.vocab_size, self.hidden_size), init=init),
+                self.pair_name: WeightSpec((self.buckets + 1, self.hidden_size), init=init)}
+
+    def bind(self, tensors):
+        self.table = tensors[self.token_name].contiguous()
+        self.pairs = tensors[self.pair_name].contiguous()
+
+    def cache_need(self):
+        return CacheNeed("state", state_shape=(1,), state_dtype=torch.int32)
+
+    def forward(self, step, cache_view):
+        return ops.embed_pairs(self.table, self.pairs, step, cache_view.state, self.mul_prev, self.mul_cur, self.scale)
+
+
 class LinearHead(Part):
     """params: ``vocab_size``; optional ``softcap`` (c > 0: logits become c tanh(logits / c)), ``scale`` (the logits are
     multiplied by it, in float32, before any cap) and ``tensor`` (the
@@ -105,4 +143,5 @@ class LinearHead(Part):
 
 register_embedding("token_embedding", TokenEmbedding)
 register_embedding("token_position_embedding", TokenPositionEmbedding)
+register_embedding("token_pair_embedding", TokenPairEmbedding)
 register_head("linear_head", LinearHead)

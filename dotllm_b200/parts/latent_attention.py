@@ -13,13 +13,16 @@ attention kernels (prefill on tcgen05, decode over pages, windows, page recyclin
 The two per-head changes of basis are batched products around the attention.
 
 A part of the keys may carry positions (``rot_dim`` R, ``position``): the queries then hold R more channels per head, one more
-projection of x gives R channels that all heads share as keys, and both are rotated (channel 2i with 2i + 1):
+projection of x gives R channels that all heads share as keys, and both are rotated (channel 2i with 2i + 1, or, with ``pairing``
+"half", channel i with i + half the rotated ones: then those rows of the two projections are interleaved once, when the weights are
+bound, and the same kernels serve; scores do not change when queries and keys are permuted alike):
 
     score = (q_h . k_h + rot(q'_h) . rot(k')) * scale
 
 The cached row is [c | rot(k')] (width r + R), the query against it [Wuk_h^T q_h | rot(q'_h)].  Options that go with it, each a
-parameter: a learned sink per head in the softmax's denominator (``sink``) and a gate per output channel (``gate``
-"channel_sigmoid").  In this form every projection of x - query latent, key/value latent with the shared key part, gate - is a row of
+parameter: a learned sink per head in the softmax's denominator (``sink``), a gate per output channel (``gate``
+"channel_sigmoid") and a gate per head ("head_sigmoid": o_h times sigmoid of one logit; being one factor per head it is applied to
+the attention's output in the latent's basis, where the attention kernel writes it).  In this form every projection of x - query latent, key/value latent with the shared key part, gate - is a row of
 one stacked matrix.  In a bfloat16 run whose r + R fits a width of the tensor-core attention kernels the row is laid out at that
 width, zeros behind it, and serves as key and value alike: the value's channels beyond r are read by nobody.
 """
@@ -40,13 +43,13 @@ class LatentAttentionMixer(Mixer):
     """params: ``n_heads``, ``key_dim``, ``value_dim`` (per head), ``q_rank`` (None: queries without a latent), ``kv_rank`` (the latents),
     ``eps`` (of the latents' norms), optional ``scale`` (default key_dim^-1/2), ``window`` (None: every
     earlier key; w: a query sees itself and the w - 1 tokens before it), ``tensors`` (local names); optional ``rot_dim`` with
-    ``position`` ({"kind": "rotary", "params"}), ``sink`` (True: tensor ``sink`` [n_heads]) and ``gate`` (None or "channel_sigmoid":
-    tensor ``gate`` [n_heads * value_dim, H])."""
+    ``position`` ({"kind": "rotary", "params"}), ``sink`` (True: tensor ``sink`` [n_heads]), ``gate`` (None, "channel_sigmoid":
+    tensor ``gate`` [n_heads * value_dim, H], or "head_sigmoid": [n_heads, H]) and ``pairing`` ("interleaved" or "half")."""
 
     NAMES = {"q_down": "q_a_proj.weight", "q_norm": "q_a_norm.weight", "q_up": "q_b_proj.weight",
              "kv_down": "kv_a_proj.weight", "kv_norm": "kv_a_norm.weight", "k_up": "k_b_proj.weight",
              "v_up": "v_b_proj.weight", "out": "o_proj.weight", "q": "q_proj.weight", "gate": "g_proj.weight", "sink": "sinks"}
-    GATES = (None, "channel_sigmoid")
+    GATES = (None, "channel_sigmoid", "head_sigmoid")
 
     def __init__(self, params, hidden_size, runtime):
         super().__init__(params, hidden_size, runtime)
@@ -68,6 +71,10 @@ class LatentAttentionMixer(Mixer):
         self.rot_dim = int(params.get("rot_dim") or 0)
         self.sink = bool(params.get("sink", False))
         self.gate = params.get("gate")
+        self.gate_width = {None: 0, "channel_sigmoid": self.n_heads * self.value_dim, "head_sigmoid": self.n_heads}.get(self.gate, 0)
+        self.pairing = str(params.get("pairing", "interleaved"))
+        if self.pairing not in ("half", "interleaved"):
+            raise ConfigError(f"latent attention: rotation pairs are 'half' or 'interleaved', not {self.pairing!r}")
         if self.gate not in self.GATES or self.rot_dim < 0:
             raise ConfigError(f"latent attention: unknown gate {self.gate!r} or a negative rotated width")
         position = params.get("position")
@@ -101,7 +108,7 @@ class LatentAttentionMixer(Mixer):
         if self.sink:
             queries[n["sink"]] = WeightSpec((H,), "precise", ("normal", 1.0))
         if self.gate:
-            queries[n["gate"]] = WeightSpec((H * self.value_dim, h), init=("normal", 0.1))
+            queries[n["gate"]] = WeightSpec((self.gate_width, h), init=("normal", 0.1))
         return {**queries,
                 n["kv_down"]: WeightSpec((self.row, h)),
                 n["kv_norm"]: WeightSpec((self.kv_rank,), "precise", ("one_plus_uniform", 0.1)),
@@ -109,15 +116,24 @@ class LatentAttentionMixer(Mixer):
                 n["v_up"]: WeightSpec((H * self.value_dim, self.kv_rank), init=("normal", 0.1)),
                 n["out"]: WeightSpec((h, H * self.value_dim))}
 
+    def _interleaved(self, rows, head, heads):
+        """``rows`` [heads * head, n] whose heads end in the rotated part: its pairs (i, i + r/2) brought side by side."""
+        dims = 2 * self.tables[0].shape[1] if self.tables is not None else 0
+        if self.pairing == "interleaved" or not dims:
+            return rows
+        at = head - self.rot_dim
+        order = list(range(at)) + [at + i + half for i in range(dims // 2) for half in (0, dims // 2)] + list(range(at + dims, head))
+        return rows.view(heads, head, -1)[:, torch.tensor(order, device=rows.device)].reshape(rows.shape)
+
     def bind(self, tensors):
         n, H = self.names, self.n_heads
         if self.q_rank is None:
-            self.w_uq = tensors[n["q"]].contiguous()
+            self.w_uq = self._interleaved(tensors[n["q"]], self.key_dim + self.rot_dim, H).contiguous()
         else:
             self.w_dq = tensors[n["q_down"]].contiguous()
             self.q_gain = tensors[n["q_norm"]].contiguous()
-            self.w_uq = tensors[n["q_up"]].contiguous()
-        self.w_dkv = tensors[n["kv_down"]].contiguous()
+            self.w_uq = self._interleaved(tensors[n["q_up"]], self.key_dim + self.rot_dim, H).contiguous()
+        self.w_dkv = self._interleaved(tensors[n["kv_down"]], self.row, 1).contiguous()
         self.kv_gain = tensors[n["kv_norm"]].contiguous()
         # [H, r, d]: the transposed key expansion of every head, applied to its query
         self.w_uk_t = tensors[n["k_up"]].view(H, self.key_dim, self.kv_rank).transpose(1, 2).contiguous()
@@ -141,7 +157,7 @@ class LatentAttentionMixer(Mixer):
 
     def _forward_stacked(self, x, step, cache_view):
         """One product of x, both latents' norms with the rotated key part in one kernel, the queries changed to the latent's basis,
-        attention over the cached rows, back to the values' basis, the gate, the output product."""
+        attention over the cached rows (a gate per head in it), back to the values' basis, a gate per channel, the output product."""
         x = ops.resolve(x)
         H, r, rq = self.n_heads, self.kv_rank, self.q_rank or 0
         proj = ops.linear(x, self.w_in, resident=True)
@@ -150,11 +166,13 @@ class LatentAttentionMixer(Mixer):
         q = ops.linear(cq if cq is not None else x, self.w_uq, resident=True)
         q = ops.latent_queries(q, self.w_uk_t, self.rot_dim, self.tables, step.token_pos, self.key_width)
         keys, values = (rows, rows[:, :self.value_width]) if cache_view.writes else (None, None)
+        g = proj[:, self.gate_at:self.gate_at + self.gate_width] if self.gate else None
+        per_head = self.gate == "head_sigmoid"
         a = ops.rope_cache_attention(q, keys, values, None, None, 0, step.token_seq, step.token_pos, cache_view.block_table,
                                      cache_view.k, cache_view.v, H, 1, self.key_width, self.scale, int(self.window or 0),
-                                     plan=step.attention_plan, value_dim=self.value_width, sinks=self.sinks, split=True)
-        g = proj[:, self.gate_at:self.gate_at + H * self.value_dim] if self.gate else None
-        o = ops.latent_values(a, self.w_uv, self.value_width, gate=g)                             # [T, H*dv]
+                                     plan=step.attention_plan, value_dim=self.value_width, gate=g if per_head else None,
+                                     sinks=self.sinks, split=True)
+        o = ops.latent_values(a, self.w_uv, self.value_width, gate=None if per_head else g)       # [T, H*dv]
         return ops.linear(o, self.w_o, out_dtype=BRANCH_DTYPE, resident=True, lazy=True)
 
     def forward(self, x, step, cache_view):
