@@ -55,9 +55,46 @@ def embed_positions(table, pos_table, ids, positions):
     return table[ids.long()].to(torch.float32) + pos_table[positions.long()].to(torch.float32)
 
 
-def gated_activation(gate_up, kind, limit=0.0, alpha=1.0):
+def embed_pairs(table, pairs, step, last, mul_prev, mul_cur, scale=1.0):
+    buckets = pairs.shape[0] - 1
+    out = table[step.tokens.long()].to(torch.float32) * scale
+    for b in range(step.slots.numel()):
+        lo, hi, slot = int(step.cu_new[b]), int(step.cu_new[b + 1]), int(step.slots[b])
+        before = int(last[slot, 0])
+        for t in range(lo, hi):
+            row = buckets if int(step.token_pos[t]) == 0 else (before * mul_prev + int(step.tokens[t]) * mul_cur) % buckets
+            out[t] += pairs[row].to(torch.float32)
+            before = int(step.tokens[t])
+        last[slot, 0] = before
+    return out
+
+
+def add_bias(x, bias):
+    x += bias
+    return x
+
+
+def qkv_rows(x, n_heads, n_kv_heads, dim, vdim, lay_k, lay_v, biases=None, gains=None, eps=0.0, first=None, mix=None):
+    T, H, G = x.shape[0], n_heads, n_kv_heads
+    parts = [p.to(torch.float32) for p in x.split([H * dim, G * dim, G * vdim], dim=1)]
+    if biases is not None:
+        parts = [p if b is None else p + b for p, b in zip(parts, biases)]
+    if gains is not None:
+        parts = [_rms(parts[0], eps) * gains[0], _rms(parts[1], eps) * gains[1], parts[2]]
+    if first is not None:
+        other = first.to(torch.float32).reshape(T, G, -1)[..., :vdim].reshape(T, G * vdim)
+        parts[2] = (1.0 - mix) * parts[2] + mix * other
+    pad = lambda p, heads, width, lay: torch.nn.functional.pad(p.reshape(T, heads, width), (0, lay - width)).reshape(T, heads * lay).to(x.dtype)
+    return pad(parts[0], H, dim, lay_k), pad(parts[1], G, dim, lay_k), pad(parts[2], G, vdim, lay_v)
+
+
+def gated_activation(gate_up, kind, limit=0.0, alpha=1.0, bias=None):
     i = gate_up.shape[1] // 2
     g, u = gate_up[:, :i].to(torch.float32), gate_up[:, i:].to(torch.float32)
+    if bias is not None:
+        g, u = g + bias[:i], u + bias[i:]
+    if kind == "silu":
+        return plain_llama.swiglu(g, u).to(gate_up.dtype)
     if kind == "silu":
         y = g * torch.sigmoid(g) * u
     elif kind == "gelu_tanh":
@@ -509,9 +546,9 @@ def linear(x, w, out_dtype=None, resident=False, lazy=False):
     return y.to(out_dtype or x.dtype)
 
 
-def gated_linear(x, w_gate_up, resident=False, kind="silu", limit=0.0, alpha=1.0):
-    if kind != "silu":
-        return gated_activation(linear(x, w_gate_up, torch.float32), kind, limit, alpha).to(x.dtype)
+def gated_linear(x, w_gate_up, resident=False, kind="silu", limit=0.0, alpha=1.0, bias=None):
+    if kind != "silu" or bias is not None:
+        return gated_activation(linear(x, w_gate_up, torch.float32), kind, limit, alpha, bias).to(x.dtype)
     return swiglu(linear(x, w_gate_up, torch.float32)).to(x.dtype)
 
 
