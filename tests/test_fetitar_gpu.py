@@ -257,3 +257,347 @@ def test_slopes_gates_and_windows_in_the_tensor_core_kernels(nh, nkv, hd):
             close(got, kernel_refs.attention(q.cpu(), kr, vr, seq.cpu(), pos.cpu(), table, *args, window=65, score_hook=rhook, gate=gate.cpu()), torch.bfloat16)
             assert torch.equal(torch.nan_to_num(kd.cpu().float()), torch.nan_to_num(kr.float())) and \
                 torch.equal(torch.nan_to_num(vd.cpu().float()), torch.nan_to_num(vr.float()))
+
+
+# ------------------------------------------------------------------ the model
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("which", ["A", "B", "C", "D", "E"])
+def test_whole_portions_and_decoding(tmp, which, dtype):
+    model, cfg, w, _ = load_pair(tmp, which, dtype)
+    tokens = tf.random_tokens(150, cfg["vocab"], 7)
+    ref = tf.plain_logits(cfg, w, tokens)
+    whole = run_cuts(model, tokens, [150])
+    assert_rows(whole, ref, dtype, "whole prompt")
+    for cuts in ([100, 50], [64, 64, 2, 20], [63, 3, 2, 2, 70], [1, 2, 129, 5], [130], [2]):
+        got = run_cuts(model, tokens, cuts)
+        assert_rows(got, ref, dtype, f"cuts {cuts}")
+        if dtype == torch.float32:
+            assert rel_err(got, whole) < 1e-5, cuts
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("which", ["A", "B", "D"])
+def test_unequal_batches_slots_and_pages_used_again(tmp, which, dtype):
+    from dotllm_b200.engine import StepEntry
+    model, cfg, w, _ = load_pair(tmp, which, dtype)
+    lens = [1, 70, 23, 131]
+    prompts = [tf.random_tokens(n + 12, cfg["vocab"], 20 + n) for n in lens]
+    refs = [tf.plain_logits(cfg, w, p) for p in prompts]
+    cache = model.new_cache(64 * 8)
+    for again in range(2):                                           # the second time every slot and page has been used before
+        cache.fill_free_pages(float("nan"))
+        seqs = [cache.open_sequence() for _ in prompts]
+        order = list(range(len(prompts))) if again == 0 else [2, 0, 3, 1]
+        out = model.step(cache, [StepEntry(seqs[i], prompts[i][:lens[i]], [0, lens[i] - 1]) for i in order])
+        want = torch.cat([refs[i][[0, lens[i] - 1]] for i in order])
+        assert_rows(out, want, dtype, "a batch of unequal prompts")
+        live = list(order)
+        for t in range(12):
+            if t == 5:
+                gone = live.pop(1)                                   # a request ends early; its slot and pages go back ...
+                cache.close_sequence(seqs[gone])
+                cache.fill_free_pages(float("nan"))
+            out = model.step(cache, [StepEntry(seqs[i], [prompts[i][lens[i] + t]]) for i in live])
+            assert_rows(out, torch.stack([refs[i][lens[i] + t] for i in live]), dtype, f"decoding together, step {t}")
+        for i in live:
+            cache.close_sequence(seqs[i])
+        cache.check()
+    assert not cache.live
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_many_sequences_decode_together_as_each_alone(tmp, dtype):
+    """Batches of 12, 40 and 140 rows: the products for some and for many rows, with the biases in their epilogues."""
+    from dotllm_b200.engine import StepEntry
+    model, cfg, w, _ = load_pair(tmp, "B", dtype)
+    base = [tf.random_tokens(n, cfg["vocab"], 200 + n) for n in (3, 17, 66, 40)]
+    refs = [tf.plain_logits(cfg, w, p) for p in base]
+    for n in (12, 40, 140):
+        cache = model.new_cache(64 * (n * 2 + 4))
+        seqs = [cache.open_sequence() for _ in range(n)]
+        which = [i % 4 for i in range(n)]
+        model.step(cache, [StepEntry(s, base[k][:-1], []) for s, k in zip(seqs, which)])
+        out = model.step(cache, [StepEntry(s, base[k][-1:]) for s, k in zip(seqs, which)])
+        assert_rows(out, torch.stack([refs[k][-1] for k in which]), dtype, f"{n} sequences")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_steps_that_mix_portions_and_single_tokens(tmp, dtype):
+    """One step with a prompt, a portion of another, and sequences that go on by one token."""
+    from dotllm_b200.engine import StepEntry
+    model, cfg, w, _ = load_pair(tmp, "A", dtype)
+    prompts = [tf.random_tokens(n, cfg["vocab"], 90 + n) for n in (90, 140, 30, 66)]
+    refs = [tf.plain_logits(cfg, w, p) for p in prompts]
+    cache = model.new_cache(64 * 10)
+    cache.fill_free_pages(float("nan"))
+    seqs = [cache.open_sequence() for _ in prompts]
+    at = [0] * 4
+    for sizes in ([0, 70, 5, 0], [40, 1, 2, 64], [2, 64, 1, 1], [1, 1, 1, 1], [47, 4, 21, 0]):
+        entries = [(i, n) for i, n in enumerate(sizes) if n]
+        out = model.step(cache, [StepEntry(seqs[i], prompts[i][at[i]:at[i] + n], [0, n - 1]) for i, n in entries])
+        assert_rows(out, torch.cat([refs[i][[at[i], at[i] + n - 1]] for i, n in entries]), dtype, f"{sizes}")
+        for i, n in entries:
+            at[i] += n
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_layers_at_a_real_models_widths(tmp, dtype):
+    """Width 1,024, heads of 128 channels, latent rows of 96 + 32 and 64 + 64: the sizes of the tensor-core kernels."""
+    model, cfg, w, _ = load_pair(tmp, "wide", dtype)
+    tokens = tf.random_tokens(230, cfg["vocab"], 11)
+    ref = tf.plain_logits(cfg, w, tokens)
+    assert_rows(run_cuts(model, tokens, [200]), ref, dtype, "a prompt of 200 tokens and 30 decoded")
+    assert_rows(run_cuts(model, tokens[:200], [130, 70]), ref[:200], dtype, "two portions")
+
+
+@pytest.mark.parametrize("seed", range(8))
+def test_configurations_drawn_at_random(tmp_path, seed):
+    """Configurations that nobody chose (`tiny_fetitar.random_config`): a prompt and twenty decoded tokens, then a batch of
+    three unequal prompts (one of a single token) decoded together, eager and through captured steps, in both dtypes."""
+    from dotllm_b200 import Model
+    from dotllm_b200.engine import StepEntry
+    rng = random.Random(300 + seed)
+    cfg_dict = tf.random_config(rng)
+    n = rng.randrange(100, 200)
+    lens = [1, rng.randrange(2, 80), rng.randrange(80, 150)]
+    for dtype in DTYPES:
+        folder = tf.make_folder(tmp_path, f"random{seed}", dtype=dtype, cfg=cfg_dict)
+        cfg, w = tf.read_folder(folder)
+        model = Model.load(folder, dtype=dtype)
+        tokens = tf.random_tokens(n, cfg["vocab"], seed)
+        prompts = [tf.random_tokens(L + 8, cfg["vocab"], seed * 7 + L) for L in lens]
+        ref, refs = tf.plain_logits(cfg, w, tokens), [tf.plain_logits(cfg, w, p) for p in prompts]
+        got = [run_cuts(model, tokens, [n - 20])]
+        want = [ref]
+        cache = model.new_cache(64 * 12)
+        cache.fill_free_pages(float("nan"))
+        seqs = [cache.open_sequence() for _ in prompts]
+        got.append(model.step(cache, [StepEntry(q, p[:L], [L - 1]) for q, p, L in zip(seqs, prompts, lens)]).clone())
+        want.append(torch.stack([r[L - 1] for r, L in zip(refs, lens)]))
+        for t in range(8):
+            got.append(model.step(cache, [StepEntry(q, [p[L + t]]) for q, p, L in zip(seqs, prompts, lens)], graphs=t >= 4).clone())
+            want.append(torch.stack([r[L + t] for r, L in zip(refs, lens)]))
+        assert_rows(torch.cat(got), torch.cat(want), dtype, f"{seed}: {cfg_dict}")
+
+
+def _sharp_sloped(t):
+    t["l0.mix.o"] *= 6.0
+
+
+def _sharp_latent(t):
+    t["l0.mix.uq"] *= 2.0
+    t["l0.mix.o"] *= 12.0
+
+
+def _agrees(tmp, which, change, tokens, ref):
+    model = load_pair(tmp, which, torch.float32, change=change, tag="sharp")[0]
+    n = len(tokens)
+    for cuts in ([n], [63, 1, 1, 200], [128, 64, 2], [n - 50], [20]):
+        assert rel_err(run_cuts(model, tokens, cuts), ref) < 1e-4, cuts
+    bf, cfg, w, _ = load_pair(tmp, which, torch.bfloat16, change=change, tag="sharp")
+    ref16 = tf.plain_logits(cfg, w, tokens)
+    for cuts in ([n - 20], [100]):
+        err = row_errors(run_cuts(bf, tokens, cuts), ref16)
+        assert float(err.median()) < 3e-2 and int((err > 0.3).sum()) <= 8, (cuts, float(err.median()), int((err > 0.3).sum()))
+
+
+def test_slopes_biases_norms_and_window_edges_decide_whole_rows(tmp):
+    """One attention layer whose scores are sharpened until single keys decide.  A window one token off either way, no slopes, the next
+    head's slopes, slopes that start at one, a missing bias and norms per head must each change rows of the plain result;
+    the engine agrees with the design over prompts, portions and decoding."""
+    import plain_fetitar as pf
+    tokens = tf.random_tokens(400, 120, 5)
+    _, cfg, w, _ = load_pair(tmp, "sharp_sloped", torch.float32, change=_sharp_sloped, tag="sharp")
+    ref = tf.plain_logits(cfg, w, tokens)
+    rms = ref.pow(2).mean(-1).sqrt()
+    differs = lambda other: int(((other - ref).pow(2).mean(-1).sqrt() / rms > 1e-2).sum())
+
+    def with_window(n):
+        other = copy.deepcopy(cfg)
+        other["layers"][0]["mixer"]["mask"]["size"] = n
+        return tf.plain_logits(other, w, tokens)
+    assert min(differs(with_window(69)), differs(with_window(71))) >= 10 and differs(with_window(400)) >= 100
+    saved = pf.distance_slopes, pf.rms
+    try:
+        for slopes in (lambda H: None, lambda H: saved[0](H)[1:] + saved[0](H)[:1], lambda H: [2.0 ** (-8.0 * h / H) for h in range(H)]):
+            pf.distance_slopes = slopes
+            assert differs(tf.plain_logits(cfg, w, tokens)) >= 100
+        pf.distance_slopes = saved[0]
+        pf.rms = lambda x, eps: saved[1](x.reshape(len(x), -1, 16), eps).reshape(x.shape) if x.shape[-1] == 32 else saved[1](x, eps)
+        assert differs(tf.plain_logits(cfg, w, tokens)) >= 100           # a norm per key head instead of one over all
+    finally:
+        pf.distance_slopes, pf.rms = saved
+    for name in ("q.b", "k.b", "v.b", "o.b"):
+        assert differs(tf.plain_logits(cfg, {**w, f"l0.mix.{name}": 0 * w[f"l0.mix.{name}"]}, tokens)) >= 100, name
+    _agrees(tmp, "sharp_sloped", _sharp_sloped, tokens, ref)
+
+
+def test_far_keys_the_rotation_and_the_gate_decide_whole_rows(tmp):
+    """One latent-attention layer sharpened the same way: a window one token off, plain frequencies, cosines without their factor,
+    channels paired the other way and no gate must each change rows of the plain result; the engine agrees with the design."""
+    import plain_fetitar as pf
+    tokens = tf.random_tokens(400, 120, 5)
+    _, cfg, w, _ = load_pair(tmp, "sharp_latent", torch.float32, change=_sharp_latent, tag="sharp")
+    ref = tf.plain_logits(cfg, w, tokens)
+    rms = ref.pow(2).mean(-1).sqrt()
+    differs = lambda other: int(((other - ref).pow(2).mean(-1).sqrt() / rms > 1e-2).sum())
+
+    def changed(**mixer):
+        other = copy.deepcopy(cfg)
+        other["layers"][0]["mixer"].update(mixer)
+        return tf.plain_logits(other, w, tokens)
+    assert min(differs(changed(mask={"size": n})) for n in (149, 151)) >= 8 and differs(changed(mask={"size": 100})) >= 100
+    assert differs(changed(rot={"dims": 8, "base": 100.0})) >= 100
+    saved = pf.yarn_frequencies, pf.rotate_halves
+    try:
+        pf.yarn_frequencies = lambda *a: (saved[0](*a)[0], 1.0)
+        assert differs(tf.plain_logits(cfg, w, tokens)) >= 100
+        pf.yarn_frequencies = saved[0]
+
+        def neighbours(x, positions, dims, base, scaling=None):
+            order = list(range(0, dims, 2)) + list(range(1, dims, 2))
+            y = x.copy()
+            y[..., :dims] = saved[1](x[..., :dims][..., order], positions, dims, base, scaling)[..., np.argsort(order)]
+            return y
+        pf.rotate_halves = neighbours
+        assert differs(tf.plain_logits(cfg, w, tokens)) >= 100
+    finally:
+        pf.yarn_frequencies, pf.rotate_halves = saved
+    assert differs(tf.plain_logits(cfg, {**w, "l0.mix.g": 0 * w["l0.mix.g"]}, tokens)) >= 100
+    _agrees(tmp, "sharp_latent", _sharp_latent, tokens, ref)
+
+
+def _first_counts(t):
+    t["l5.mix.vmix"].fill_(0.9)
+    for name in ("l0.mix.v", "l0.mix.v.b"):
+        t[name] *= 4.0
+    t["l5.mix.o"] *= 4.0
+
+
+def test_mixed_values_and_pair_rows_show(tmp):
+    """Values not mixed, or mixed the wrong way round, a pair table that is read without the token before, and a first token with
+    another row than the last are far from the design; the engine is close to it."""
+    import plain_fetitar as pf
+    model, cfg, w, _ = load_pair(tmp, "A", torch.float32, change=_first_counts, tag="mixed")
+    tokens = tf.random_tokens(120, cfg["vocab"], 17)
+    ref = tf.plain_logits(cfg, w, tokens)
+    rms = ref.pow(2).mean(-1).sqrt()
+    off = lambda: (tf.plain_logits(cfg, w, tokens) - ref).pow(2).mean(-1).sqrt() / rms
+    saved = pf.mixed_values, pf.bigram_rows
+    try:
+        for mixed in (lambda v, first, weight: v, lambda v, first, weight: weight * v + (1.0 - weight) * first):
+            pf.mixed_values = mixed
+            assert int((off() > 1e-2).sum()) >= 100
+        pf.mixed_values = saved[0]
+        pf.bigram_rows = lambda tokens, buckets, a, b: [(int(t) * b) % buckets for t in tokens]
+        assert int((off() > 1e-2).sum()) >= 100
+        pf.bigram_rows = lambda tokens, buckets, a, b: [(int(tokens[0]) * b) % buckets] + saved[1](tokens, buckets, a, b)[1:]
+        assert float(off()[0]) > 1e-2
+    finally:
+        pf.mixed_values, pf.bigram_rows = saved
+    for cuts in ([120], [1, 2, 3, 64], [50]):
+        assert_rows(run_cuts(model, tokens, cuts), ref, torch.float32, f"cuts {cuts}")
+    bf, cfg16, w16, _ = load_pair(tmp, "A", torch.bfloat16, change=_first_counts, tag="mixed")
+    assert_rows(run_cuts(bf, tokens, [90]), tf.plain_logits(cfg16, w16, tokens), torch.bfloat16, "bfloat16")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_long_decoding_over_page_borders(tmp, dtype):
+    model, cfg, w, _ = load_pair(tmp, "A", dtype)
+    tokens = tf.random_tokens(330, cfg["vocab"], 5)
+    ref = tf.plain_logits(cfg, w, tokens)
+    assert_rows(run_cuts(model, tokens, [30]), ref, dtype, "300 tokens decoded one by one, over five page borders")
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("which", ["A", "B"])
+def test_greedy_generation_through_the_entry_point(tmp, which, dtype):
+    from dotllm_b200 import InferenceOptions
+    model, cfg, w, _ = load_pair(tmp, which, dtype)
+    prompts = [tf.random_tokens(n, cfg["vocab"], 60 + n) for n in (1, 9, 40, 70)]
+    n_new = 24
+    options = InferenceOptions(temperature=0.0, max_tokens=n_new, stop_token_ids=[])
+    outs = model.generate(prompts, options)
+    again = model.generate(prompts, options)                         # through captured steps now
+    for p, o in list(zip(prompts, outs)) + list(zip(prompts, again)):
+        assert o.finish_reason.value == "length" and o.generated_token_count == n_new
+        ref = tf.plain_logits(cfg, w, p + o.generated_token_ids)
+        spread = float(ref.std())
+        for i, tok in enumerate(o.generated_token_ids):              # teacher-forced: the plain arg-max, or within rounding of it
+            row = ref[len(p) - 1 + i]
+            assert int(row.argmax()) == tok or float(row.max() - row[tok]) <= (1e-4 if dtype == torch.float32 else 0.1) * spread, \
+                (i, tok, int(row.argmax()))
+    alone = model.generate(prompts[2], options)
+    if dtype == torch.float32:
+        assert [o.generated_token_ids for o in again] == [o.generated_token_ids for o in outs]
+        assert alone.generated_token_ids == outs[2].generated_token_ids
+
+
+def test_steps_replayed_from_graphs(tmp):
+    """Prompts and decode steps captured as graphs (exact batch size and the shared widths with idle rows) give the eager steps'
+    logits; the trial run before a capture leaves the last tokens as they were."""
+    from dotllm_b200.engine import StepEntry
+    for dtype in DTYPES:
+        model, cfg, w, _ = load_pair(tmp, "A", dtype)
+        prompts = [tf.random_tokens(n + 10, cfg["vocab"], 80 + n) for n in (5, 66, 30)]
+        refs = [tf.plain_logits(cfg, w, p) for p in prompts]
+        for graphs in (True, "lazy"):
+            cache = model.new_cache(64 * 12)
+            for again in range(3):                                   # the third prompt step of this shape runs from its graph
+                seqs = [cache.open_sequence() for _ in prompts]
+                out = model.step(cache, [StepEntry(s, p[:-10], [len(p) - 11]) for s, p in zip(seqs, prompts)], graphs=graphs)
+                assert_rows(out, torch.stack([r[len(r) - 11] for r in refs]), dtype, f"graphs={graphs} prompt {again}")
+                for t in range(10):
+                    out = model.step(cache, [StepEntry(s, [p[len(p) - 10 + t]]) for s, p in zip(seqs, prompts)], graphs=graphs)
+                    assert_rows(out, torch.stack([r[len(r) - 10 + t] for r in refs]), dtype, f"graphs={graphs} step {t}")
+                for s in seqs:
+                    cache.close_sequence(s)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_replay_program_on_a_fetitar_folder(tmp_path, dtype):
+    tdtype = {"float32": torch.float32, "bfloat16": torch.bfloat16}[dtype]
+    folder = tf.make_folder(tmp_path, "A", seed=2, dtype=tdtype)
+    cfg, w = tf.read_folder(folder)
+    a, b = tf.random_tokens(90, cfg["vocab"], 1), tf.random_tokens(30, cfg["vocab"], 2)
+    ra, rb = tf.plain_logits(cfg, w, a), tf.plain_logits(cfg, w, b)
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": a[:80], "want": [0, 79]}, {"id": "b", "tokens": b[:20], "want": []}], "end": []}]
+    for t in range(10):
+        steps.append({"step": t + 1, "entries": [{"id": "a", "tokens": [a[80 + t]], "want": [0]},
+                                                 {"id": "b", "tokens": [b[20 + t]], "want": [0] if t % 2 else []}],
+                      "end": ["a", "b"] if t == 9 else []})
+    out_dir = tmp_path / "out"
+    proc = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", str(folder), "--dtype", dtype, "--out", str(out_dir),
+                           "--max-tokens", "256"], input="\n".join(json.dumps(s) for s in steps) + "\n", capture_output=True,
+                          text=True, timeout=600)
+    assert proc.returncode == 0, proc.stderr[-2000:]
+    assert proc.stdout.split() == [x for s in steps for x in ("done", str(s["step"]))]
+    read = lambda n: torch.from_numpy(np.fromfile(out_dir / f"{n}.f32", dtype="<f4").reshape(-1, cfg["vocab"]).copy())
+    assert_rows(read(0), ra[[0, 79]], tdtype, "prompt step")
+    for t in range(10):
+        want = [ra[80 + t]] + ([rb[20 + t]] if t % 2 else [])
+        assert_rows(read(t + 1), torch.stack(want), tdtype, f"decode step {t}")
+
+
+def test_command_line_makes_and_runs_a_fetitar_folder(tmp_path):
+    """`random` writes a folder from a configuration file, `run` generates from it: greedy tokens are the plain
+    implementation's, a seeded sampled request gives the same tokens twice."""
+    cfg_path = tmp_path / "cfg.json"
+    cfg_path.write_text(json.dumps(tf.CONFIGS["C"]))
+    folder = tmp_path / "model"
+    made = subprocess.run([sys.executable, "-m", "dotllm_b200", "random", str(cfg_path), str(folder), "--seed", "3", "--dtype", "float32"],
+                          cwd=ROOT, capture_output=True, text=True, timeout=600)
+    assert made.returncode == 0, made.stderr[-2000:]
+    cfg, w = tf.read_folder(folder)
+    prompt = tf.random_tokens(11, cfg["vocab"], 9)
+    run = lambda *extra: subprocess.run([sys.executable, "-m", "dotllm_b200", "run", str(folder), "-p", ",".join(map(str, prompt)),
+                                         "-n", "6", "--dtype", "float32", "--json", *extra], cwd=ROOT, capture_output=True, text=True,
+                                        timeout=600)
+    proc = run("-t", "0", "--stop-ids", "")
+    assert proc.returncode == 0, proc.stderr[-2000:]
+    tokens = json.loads(proc.stdout)["results"][0]["generated_token_ids"]
+    ref = tf.plain_logits(cfg, w, prompt + tokens)
+    assert tokens == [int(ref[len(prompt) - 1 + i].argmax()) for i in range(6)]
+    a, b = run("-t", "0.9", "--top-k", "30", "-s", "5"), run("-t", "0.9", "--top-k", "30", "-s", "5")
+    assert a.returncode == 0 and json.loads(a.stdout)["results"][0]["generated_token_ids"] == \
+        json.loads(b.stdout)["results"][0]["generated_token_ids"]
