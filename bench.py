@@ -10,6 +10,7 @@
     python bench.py --workload zemezen [--shape 1b]   # the Zemezen design beside a Kubedra of equal width and depth, and its kernels
     python bench.py --workload sopalorn [--shape 1b]  # the Sopalorn design beside a Zemezen of equal width and depth, and its kernels
     python bench.py --workload semanex [--shape 1b]   # the Semanex design beside a Sopalorn and a Zemezen of equal width and depth, and its kernels
+    python bench.py --workload fetitar [--shape 1b]   # the Fetitar design beside a Kubedra and a Llama of equal width and depth, and its kernels
     python bench.py --impl plain-cpu                  # the plain implementation under tests/, timed on the CPU
 
 A "step" is one decode step: one new token for each of ``batch`` sequences that already hold
@@ -131,7 +132,7 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference", "plain-cpu"])
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"])
     ap.add_argument("--repeats", type=int, default=5, help="repetitions of every timed region (best and CV are reported)")
-    ap.add_argument("--workload", default="steady", choices=["steady", "unequal", "staggered", "short-prompts", "kubedra", "komulorn", "zemezen", "sopalorn", "semanex"],
+    ap.add_argument("--workload", default="steady", choices=["steady", "unequal", "staggered", "short-prompts", "kubedra", "komulorn", "zemezen", "sopalorn", "semanex", "fetitar"],
                     help="unequal: 64 prompts of 16..2048 tokens in one prefill step, then 256 decode steps; "
                          "staggered: Model.generate on 64 prompts whose requests end five steps apart; "
                          "short-prompts: the time to the first token of single prompts of 20 to 1,024 tokens; "
@@ -140,7 +141,8 @@ def main():
                          "komulorn: the same for the Komulorn design beside a Llama of equal width, heads and depth; "
                          "zemezen: the same for the Zemezen design beside a Kubedra of equal width and depth; "
                          "sopalorn: the same for the Sopalorn design beside a Zemezen of equal width and depth; "
-                         "semanex: the same for the Semanex design beside a Sopalorn and a Zemezen")
+                         "semanex: the same for the Semanex design beside a Sopalorn and a Zemezen; "
+                         "fetitar: the same for the Fetitar design beside a Kubedra and a Llama")
     ap.add_argument("--no-generate", action="store_true", help="skip the Model.generate cells")
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--context", type=int, default=8192)
@@ -180,6 +182,8 @@ def main():
         return sopalorn_workload(args)
     if args.workload == "semanex":
         return semanex_workload(args)
+    if args.workload == "fetitar":
+        return fetitar_workload(args)
     pk = peaks()
     shape_name, shape = SHAPES[args.shape]
     cfg_dict = dict(shape, num_hidden_layers=args.layers or shape["num_hidden_layers"])
@@ -1269,6 +1273,169 @@ def semanex_workload(args):
                       "n_gpus": 1, "steps": args.steps, "warmup": max(3, args.warmup), "higher_is_better": True, "dtype": "bf16",
                       "data": "synthetic", "vs_baseline": None, "clocks": sampler.stop(),
                       "config": {"model": "Semanex, four layers at the sizes named", "batch": 8, "context": ctx, "prefill_tokens": T,
+                                 "l2": "flushed between a kernel's timed launches"},
+                      "peaks": pk, "sizes": out}))
+    return 0
+
+
+FETITAR_SIZES = {
+    # width, heads, latent row and feed-forward of the sizes above; every window holds the context, so that a layer sees as many keys
+    # as the Llama's and the Kubedra's
+    "1b": dict(width=2048, heads=16, kv_heads=4, dim=128, q_rank=768, kv_rank=96, rot=32, window=2048, ff=8192, buckets=65521),
+    "8b": dict(width=4096, heads=32, kv_heads=8, dim=128, q_rank=1536, kv_rank=96, rot=32, window=2048, ff=14336, buckets=65521),
+}
+
+
+def fetitar_workload(args):
+    """Prefill (one prompt of 2,048 tokens) and decode (batch 8 and 64 at context 2,048) tokens per second of a four-layer Fetitar
+    model at a real model's layer sizes (attention, latent attention, latent attention, attention), beside a four-layer Kubedra of
+    latent attention (the closest design here: norms on both sides of every sublayer, latent attention) and a four-layer Llama
+    (attention) of the same width, heads, latent row and feed-forward; then every kernel the design added or changed, alone, against its
+    roofline, beside the like kernel of the closest path.  Random weights, synthetic tokens, bfloat16, CUDA events, an L2 flush
+    between the timed launches of a kernel."""
+    import types
+    import numpy as np
+    import torch
+    from dotllm_b200 import Model
+    from dotllm_b200.config import config_from_dict
+    from dotllm_b200.engine.step import AttentionPlan
+    from dotllm_b200.kernels import ops
+    tools = design_bench_tools(args)
+    pk, hbm, tflops, dev, T, ctx, sampler, timed, model_points = (tools.pk, tools.hbm, tools.tflops, tools.dev, tools.T, tools.ctx,
+                                                                  tools.sampler, tools.timed, tools.model_points)
+    sizes = ["1b", "8b"] if args.shape not in ("1b",) else ["1b"]
+    vocab = 32000
+
+    def kernel_table(z):
+        W, H, hd, nkv, r, rot, rq = z["width"], z["heads"], z["dim"], z["kv_heads"], z["kv_rank"], z["rot"], z["q_rank"]
+        lay, bf = r + rot, torch.bfloat16
+        rows = {}
+        i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+        rnd = lambda *s: torch.randn(*s, device=dev)
+
+        def row(name, fn, bytes_=0, flops=0):
+            us = timed(fn) * 1000.0
+            need = max(bytes_ / hbm, flops / tflops) * 1e6
+            rows[name] = {"us": round(us, 1), "roofline_us": round(need, 2), "frac": round(need / us, 4)}
+        for label, n, n_seqs in (("prefill", T, 1), ("decode", 64, 64)):
+            each = n // n_seqs
+            starts, news = ([0], [n]) if label == "prefill" else ([ctx - 1] * n_seqs, [1] * n_seqs)
+            totals = [s0 + s1 for s0, s1 in zip(starts, news)]
+            seq = torch.arange(n, dtype=torch.int32, device=dev) // each
+            pos = i32([s0 + i for s0, s1 in zip(starts, news) for i in range(s1)])
+            cu = i32([0] + list(np.cumsum(news)))
+            slots = torch.arange(n_seqs, dtype=torch.int32, device=dev)
+            tokens = torch.randint(0, vocab, (n,), dtype=torch.int32, device=dev)
+            # the embedding with its pair rows, beside the plain one
+            table, pairs, last = rnd(vocab, W).to(bf), rnd(z["buckets"] + 1, W).to(bf), torch.zeros(n_seqs + 1, 1, dtype=torch.int32, device=dev)
+            step = types.SimpleNamespace(tokens=tokens, token_seq=seq, token_pos=pos, cu_new=cu, slots=slots)
+            row(f"embed_pairs {label}", lambda: ops.embed_pairs(table, pairs, step, last, 331, 17, 45.0), bytes_=n * W * (2 + 2 + 4))
+            row(f"llama embedding {label}", lambda: ops.gather_rows(table, tokens), bytes_=n * W * (2 + 4))
+            del table, pairs
+            # the norm of a biased branch, the sum and the next norm
+            x, y, ones, bias = rnd(n, W), rnd(n, W), torch.ones(W, device=dev), rnd(W)
+            row(f"biased branch norm + sum + norm {label}",
+                lambda: ops.add_normed_branch(x, ops.NormedBranch(ops.Biased(y, bias), ones, 1e-5), ones, 1e-5, bf), bytes_=n * W * (8 + 4 + 2))
+            row(f"kubedra branch norm + sum + norm {label}", lambda: ops.add_normed_branch(x, ops.NormedBranch(y, ones, 1e-5), ones, 1e-5, bf),
+                bytes_=n * W * (8 + 4 + 2))
+            row(f"llama add_rmsnorm {label}", lambda: ops.add_rmsnorm(x, y, ones, 1e-5, bf), bytes_=n * W * (8 + 4 + 2))
+            # between the projection and the cache
+            width = (H + 2 * nkv) * hd
+            qkv, first, mix = rnd(n, width).to(bf), rnd(n, nkv * hd).to(bf), torch.full((1,), 0.4, device=dev)
+            biases, gains = (rnd(H * hd), rnd(nkv * hd), rnd(nkv * hd)), (rnd(H * hd), rnd(nkv * hd))
+            row(f"qkv_rows {label}", lambda: ops.qkv_rows(qkv, H, nkv, hd, hd, hd, hd, biases=biases, gains=gains, eps=1e-5, first=first, mix=mix),
+                bytes_=n * (2 * width + nkv * hd) * 2)
+            both = torch.cat(gains)
+            row(f"sopalorn norm of queries and keys {label}", lambda: ops.group_rmsnorm(qkv[:, :(H + nkv) * hd], both, H * hd, nkv * hd, 1e-5),
+                bytes_=n * (H + nkv) * hd * 4)
+            # attention over pages
+            per = ctx if label == "decode" else n
+            pages = (per + 63) // 64
+            tables = torch.arange(n_seqs * pages, dtype=torch.int32, device=dev).reshape(n_seqs, pages)
+
+            def attend(name, q, heads, kv, width, window, **kw):
+                k_pool, v_pool = rnd(n_seqs * pages + 1, kv, 64, width).to(bf), rnd(n_seqs * pages + 1, kv, width, 64).to(bf)
+                plan = AttentionPlan(n_seqs, max(news), max(totals), label == "decode", i32(starts), i32(news), cu, i32(totals), list(starts), list(news))
+                seen = [min(p + 1, window or p + 1) for p in pos.tolist()]
+                keys = sum(seen) if label == "decode" else per * n_seqs
+                row(f"{name} {label}", lambda: ops.attention(q, k_pool, v_pool, seq, pos, tables, heads, kv, width, width ** -0.5, window, plan=plan, **kw),
+                    bytes_=keys * kv * width * 2 * 2 + n * heads * width * 4, flops=4 * sum(seen) * heads * width)
+            q = qkv[:, :H * hd]
+            hook = ops.ScoreHook(0.0, torch.tensor([2.0 ** (-8.0 * (h + 1) / H) for h in range(H)], device=dev))
+            attend("attention, slopes", q, H, nkv, hd, z["window"], score_hook=hook, split=True)
+            attend("llama attention", q, H, nkv, hd, 0)
+            attend("attention, slopes, window 512", q, H, nkv, hd, 512, score_hook=hook, split=True)
+            attend("attention, window 512", q, H, nkv, hd, 512)
+            # latent attention: the rows, the queries, the attention over them with a gate per head, the way back
+            lp = rnd(n, rq + r + rot).to(bf)
+            ang = torch.arange(8192, device=dev)[:, None] * 1e-4 ** (torch.arange(rot // 2, device=dev) * 2.0 / rot)[None, :]
+            turn = (torch.cos(ang).contiguous(), torch.sin(ang).contiguous())
+            gq, gk = torch.ones(rq, device=dev), torch.ones(r, device=dev)
+            row(f"latent_rows {label}", lambda: ops.latent_rows(lp, gq, gk, 1e-5, rot, turn, pos, lay), bytes_=n * (rq + r + rot) * 4)
+            lat = rnd(n, rq)
+            row(f"kubedra norm of a query latent {label}", lambda: ops.add_rmsnorm(lat, None, gq, 1e-5, bf), bytes_=n * rq * 6)
+            d_un = hd - rot
+            lq, wk = rnd(n, H * hd).to(bf), (rnd(H, r, d_un) * 0.1).to(bf)
+            row(f"latent_queries {label}", lambda: ops.latent_queries(lq, wk, rot, turn, pos, lay),
+                bytes_=n * H * (hd + lay) * 2 + H * r * d_un * 2, flops=2 * n * H * r * d_un)
+            wk2 = (rnd(H, lay, hd) * 0.1).to(bf)
+            row(f"kubedra queries to the latent {label}", lambda: ops.linear_per_head(lq, wk2), bytes_=n * H * (hd + lay) * 2 + H * lay * hd * 2,
+                flops=2 * n * H * lay * hd)
+            lqw, hg = rnd(n, H * lay).to(bf), rnd(n, H).to(bf)
+            attend("latent attention, gate per head", lqw, H, 1, lay, z["window"], gate=hg, split=True)
+            attend("kubedra latent attention", lqw, H, 1, lay, z["window"])
+            attend("latent attention, gate per head, window 512", lqw, H, 1, lay, 512, gate=hg, split=True)
+            wv, wv2 = (rnd(H, hd, r) * 0.1).to(bf), (rnd(H, hd, lay) * 0.1).to(bf)
+            row(f"back from the latent {label}", lambda: ops.latent_values(lqw, wv, lay), bytes_=n * H * (r + hd) * 2 + H * r * hd * 2,
+                flops=2 * n * H * r * hd)
+            row(f"kubedra back from the latent {label}", lambda: ops.linear_per_head(lqw, wv2), bytes_=n * H * (lay + hd) * 2 + H * lay * hd * 2,
+                flops=2 * n * H * lay * hd)
+            # the gated product with biases in its epilogue
+            xb, wgu, bgu = rnd(n, W).to(bf), (rnd(2 * z["ff"], W) * 0.02).to(bf), rnd(2 * z["ff"])
+            io, fl = 2 * z["ff"] * W * 2 + n * W * 2 + n * z["ff"] * 2, 2 * n * 2 * z["ff"] * W
+            row(f"gated product + biases {label}", lambda: ops.gated_linear(xb, wgu, resident=True, bias=bgu), bytes_=io, flops=fl)
+            row(f"llama gated product {label}", lambda: ops.gated_linear(xb, wgu, resident=True), bytes_=io, flops=fl)
+            if label == "decode":
+                x8 = xb[:8].contiguous()
+                row("gated product + biases decode, 8 rows", lambda: ops.gated_linear(x8, wgu, resident=True, bias=bgu), bytes_=io, flops=fl // 8)
+                row("llama gated product decode, 8 rows", lambda: ops.gated_linear(x8, wgu, resident=True), bytes_=io, flops=fl // 8)
+            del wgu
+        return rows
+
+    out = {}
+    for name in sizes:
+        z = FETITAR_SIZES[name]
+        scale, D = z["dim"] ** -0.5, z["dim"]
+        dense = {"kind": "dense", "ff": z["ff"]}
+        att = {"type": "attention", "mlp": dense, "mixer": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": D, "vdim": D, "scale": scale,
+                                                            "v_mix": True, "mask": {"size": z["window"]}}}
+        lat = {"type": "latent_attention", "mlp": dense,
+               "mixer": {"heads": z["heads"], "dim": D - z["rot"], "rot_dim": z["rot"], "vdim": D, "q_rank": z["q_rank"], "kv_rank": z["kv_rank"],
+                         "scale": scale, "mask": {"size": z["window"]},
+                         "rot": {"dims": z["rot"], "base": 10000.0, "scaling": {"factor": 8.0, "original": 2048, "fast": 32.0, "slow": 1.0}}}}
+        fcfg = {"architecture": "Fetitar", "vocab": vocab, "width": z["width"], "max_positions": 8192, "norm": {"eps": 1e-5},
+                "embedding": {"scale": 1.0, "bigram": {"buckets": z["buckets"], "mul_prev": 331, "mul_cur": 17}}, "layers": [att, lat, lat, att]}
+        klat = {"type": "latent_attention", "mlp": dense, "mixer": {"heads": z["heads"], "dim": D, "vdim": D, "q_rank": z["q_rank"],
+                                                                    "kv_rank": z["kv_rank"] + z["rot"], "scale": scale, "mask": {"size": z["window"]}}}
+        kcfg = {"architecture": "Kubedra", "vocab": vocab, "width": z["width"], "max_positions": 8192, "norm": {"eps": 1e-5}, "layers": [klat] * 4}
+        lcfg = dict(LLAMA_31_8B, num_hidden_layers=4, hidden_size=z["width"], num_attention_heads=z["heads"], num_key_value_heads=z["kv_heads"],
+                    intermediate_size=z["ff"], vocab_size=vocab, head_dim=D)
+        point = {}
+        for label, cfg_dict in (("fetitar", fcfg), ("kubedra", kcfg), ("llama", lcfg)):
+            model = Model.random(config_from_dict(cfg_dict), seed=0, dtype="bfloat16", device="cuda:0", on_device=True)
+            point[label] = model_points(model, vocab)
+            print(f"[bench] {name} {label}: {point[label]}", file=sys.stderr, flush=True)
+            del model
+            torch.cuda.empty_cache()
+        point["kernels"] = kernel_table(z)
+        for k, v in point["kernels"].items():
+            print(f"[bench] {name} {k}: {v}", file=sys.stderr, flush=True)
+        out[name] = point
+    first = out[sizes[0]]
+    print(json.dumps({"metric": "fetitar_decode_tokens_per_second", "value": first["fetitar"]["decode_b8_tok_s"], "unit": "tokens/s",
+                      "n_gpus": 1, "steps": args.steps, "warmup": max(3, args.warmup), "higher_is_better": True, "dtype": "bf16",
+                      "data": "synthetic", "vs_baseline": None, "clocks": sampler.stop(),
+                      "config": {"model": "Fetitar, four layers at the sizes named", "batch": 8, "context": ctx, "prefill_tokens": T,
                                  "l2": "flushed between a kernel's timed launches"},
                       "peaks": pk, "sizes": out}))
     return 0
