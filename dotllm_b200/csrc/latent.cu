@@ -214,6 +214,35 @@ latent_query_tail_kernel(const T* __restrict__ q, int q_ld, int dim, int rot, in
     }
 }
 
+// The same for bfloat16 tails that move 16 bytes at a time: a thread takes four pairs of one head.
+__global__ void __launch_bounds__(256)
+latent_query_tail_vec_kernel(const __nv_bfloat16* __restrict__ q, int q_ld, int dim, int rot, int rot_dims, const float* __restrict__ cos_t,
+                             const float* __restrict__ sin_t, int table_rows, const int32_t* __restrict__ token_pos,
+                             __nv_bfloat16* __restrict__ out, int out_ld, int rank, int lay, int H, int n_tokens) {
+    dl_launch_dependents();
+    dl_grid_dependency_wait();
+    const int units = (lay - rank) / 8, per_row = H * units;
+    const long long idx = (long long)blockIdx.x * 256 + threadIdx.x;
+    if (idx >= (long long)n_tokens * per_row) return;
+    const int t = (int)(idx / per_row), e = (int)(idx - (long long)t * per_row), h = e / units, c = (e - h * units) * 8;
+    uint4 raw = make_uint4(0u, 0u, 0u, 0u);
+    if (c < rot) raw = *reinterpret_cast<const uint4*>(q + (size_t)t * q_ld + (size_t)h * (dim + rot) + dim + c);
+    if (c < rot_dims) {
+        const int pos = min(token_pos[t], table_rows - 1);       // host-validated
+        const size_t at = (size_t)pos * (rot_dims / 2) + (c >> 1);
+        const float4 cs = *reinterpret_cast<const float4*>(cos_t + at), sn = *reinterpret_cast<const float4*>(sin_t + at);
+        const float cc[4] = {cs.x, cs.y, cs.z, cs.w}, ss[4] = {sn.x, sn.y, sn.z, sn.w};
+        __nv_bfloat162* v = reinterpret_cast<__nv_bfloat162*>(&raw);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            float a, b;
+            lt_pair(__low2float(v[i]), __high2float(v[i]), cc[i], ss[i], a, b);
+            v[i] = __floats2bfloat162_rn(a, b);
+        }
+    }
+    *reinterpret_cast<uint4*>(out + (size_t)t * out_ld + (size_t)h * lay + rank + c) = raw;
+}
+
 extern "C" int dl_latent_query_tail(const void* q, int dtype, int q_ld, int dim, int rot, int rot_dims, const float* cos_t,
                                     const float* sin_t, int table_rows, const int32_t* token_pos, void* out, int out_ld, int rank,
                                     int lay, int H, int n_tokens, void* stream) {
@@ -224,6 +253,16 @@ extern "C" int dl_latent_query_tail(const void* q, int dtype, int q_ld, int dim,
     if (n_tokens == 0 || lay == rank) return DL_OK;
     const dim3 grid(n_tokens), block(256);
     cudaError_t e;
+    const uintptr_t places = (uintptr_t)q | (uintptr_t)out | (uintptr_t)cos_t | (uintptr_t)sin_t;
+    if (dtype == DL_BF16 && places % 16 == 0 && q_ld % 8 == 0 && out_ld % 8 == 0 && dim % 8 == 0 && rot % 8 == 0 && rot_dims % 8 == 0 &&
+        rank % 8 == 0 && lay % 8 == 0) {
+        const long long n = (long long)n_tokens * H * ((lay - rank) / 8);
+        e = dl_launch_dependent(latent_query_tail_vec_kernel, dim3((unsigned)((n + 255) / 256)), block, 0, (cudaStream_t)stream,
+                                (const __nv_bfloat16*)q, q_ld, dim, rot, rot_dims, cos_t, sin_t, table_rows, token_pos,
+                                (__nv_bfloat16*)out, out_ld, rank, lay, H, n_tokens);
+        if (e != cudaSuccess) return dl_fail(DL_ERR_LAUNCH, "latent_query_tail: %s", cudaGetErrorString(e));
+        return DL_OK;
+    }
     if (dtype == DL_F32)
         e = dl_launch_dependent(latent_query_tail_kernel<float>, grid, block, 0, (cudaStream_t)stream, (const float*)q, q_ld, dim, rot, rot_dims,
                                 cos_t, sin_t, table_rows, token_pos, (float*)out, out_ld, rank, lay, H);

@@ -336,7 +336,10 @@ extern "C" int dl_rope_cache_write(void* q, int q_stride, const void* k, int k_s
     const size_t tile_smem = (size_t)RT_TOKENS * (vd + 4 / elem) * elem;
     const bool biases_aligned = ((uintptr_t)q_bias % 16) == 0 && ((uintptr_t)k_bias % 16) == 0 && ((uintptr_t)v_bias % 16) == 0;
     if (n_tokens >= RT_TOKENS && tile_smem <= 48 * 1024 && (dtype == DL_F32 || dtype == DL_BF16)) {
-        dim3 tgrid((n_tokens + RT_TOKENS - 1) / RT_TOKENS, write_cache ? nh + nkv : nh);
+        // queries that are neither rotated nor biased stay as they are: no blocks for them
+        const int q_blocks = (rotary_dim > 0 || q_bias != nullptr) ? nh : 0;
+        if (q_blocks == 0 && !write_cache) return DL_OK;
+        dim3 tgrid((n_tokens + RT_TOKENS - 1) / RT_TOKENS, (write_cache ? nkv : 0) + q_blocks);
         const bool aligned = ((uintptr_t)q % 16) == 0 && q_stride % 8 == 0 && ((uintptr_t)cos_t % 16) == 0 &&
                              ((uintptr_t)sin_t % 16) == 0 &&
                              (!write_cache || (((uintptr_t)k % 16) == 0 && ((uintptr_t)v % 16) == 0 && k_stride % 8 == 0 &&
