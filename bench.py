@@ -1412,7 +1412,7 @@ def fetitar_workload(args):
         lat = {"type": "latent_attention", "mlp": dense,
                "mixer": {"heads": z["heads"], "dim": D - z["rot"], "rot_dim": z["rot"], "vdim": D, "q_rank": z["q_rank"], "kv_rank": z["kv_rank"],
                          "scale": scale, "mask": {"size": z["window"]},
-                         "rot": {"dims": z["rot"], "base": 10000.0, "scaling": {"factor": 8.0, "original": 2048, "fast": 32.0, "slow": 1.0}}}}
+                         "rot": {"dims": z["rot"], "base": 10000.0, "scaling": {"factor": 4.0, "original": 4096, "fast": 16.0, "slow": 2.0}}}}
         fcfg = {"architecture": "Fetitar", "vocab": vocab, "width": z["width"], "max_positions": 8192, "norm": {"eps": 1e-5},
                 "embedding": {"scale": 1.0, "bigram": {"buckets": z["buckets"], "mul_prev": 331, "mul_cur": 17}}, "layers": [att, lat, lat, att]}
         klat = {"type": "latent_attention", "mlp": dense, "mixer": {"heads": z["heads"], "dim": D, "vdim": D, "q_rank": z["q_rank"],

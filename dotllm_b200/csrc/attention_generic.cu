@@ -13,7 +13,7 @@
 // the kernel of the float32 path and the fallback of the bfloat16 path for sizes that the
 // tensor-core kernels do not take.
 //
-// It also honours every change of the scores before the softmax (the tensor-core kernels take the cap), the place where
+// It also honours every change of the scores before the softmax (as the tensor-core kernels do), the place where
 // the reference's seam for position encodings that bias scores sits
 // (src/DotLLM.Core/PositionEncoding/IPositionEncoding.cs:10-34): with `softcap` > 0 a score becomes
 // softcap * tanh(score / softcap), and with `slopes` (one float per query head) slope * (key position -

@@ -151,7 +151,7 @@ def test_plain_rotation_against_the_packages_tables():
     z = lambda t: t[..., :4] + 1j * t[..., 4:8]
     assert np.allclose(z(y[1]) / z(x[1]), np.exp(1j * rotary_frequencies(8, 100.0))[None, :])
     assert np.array_equal(pf.rotate_halves(x, np.arange(5), 0, 100.0), x)
-    for dims, base, s in ((8, 100.0, (4.0, 64.0, 8.0, 1.0)), (32, 1e5, (8.0, 3000.0, 32.0, 1.0)), (12, 50.0, (8.0, 100.0, 3.0, 0.5)), (2, 10.0, (2.0, 4.0, 50.0, 40.0))):
+    for dims, base, s in ((8, 100.0, (4.0, 64.0, 8.0, 1.0)), (32, 1e5, (5.0, 3000.0, 24.0, 1.5)), (12, 50.0, (8.0, 100.0, 3.0, 0.5)), (2, 10.0, (2.0, 4.0, 50.0, 40.0))):
         mine = dict(zip(("factor", "original", "fast", "slow"), s))
         theirs = {"rope_type": "yarn", "factor": s[0], "original_max_position_embeddings": s[1], "fast_turns": s[2], "slow_turns": s[3]}
         f, grow = pf.yarn_frequencies(dims, base, mine)

@@ -77,7 +77,7 @@ CONFIGS = {
                 embedding_scale=5.0, bigram=None),
     # a latent row wider than any tensor-core width, heads wider than any, a single layer type in a row, multipliers of both signs
     "E": config(72, 90, 1e-6,
-                [latent(2, 24, 40, 24, 24, 130, 0.1, (40, 300.0, (3.0, 50.0, 2.0, 1.0)), 40, None),
+                [latent(2, 24, 40, 24, 24, 130, 0.1, (40, 300.0, (3.0, 50.0, 2.0, 1.0)), 42, None),
                  latent(2, 16, 8, 16, 16, 24, 0.2, (8, 300.0), 63, dense(48)),
                  sloped(2, 1, 136, 40, 0.09, 80, True, dense(56)),
                  sloped(2, 1, 8, 40, 0.3, 20, True, dense(56))],
@@ -89,7 +89,7 @@ SHARP_SLOPED = config(64, 120, 1e-5, [sloped(8, 2, 16, 16, 3.0, 70, True)], embe
 SHARP_LATENT = config(64, 120, 1e-5, [latent(4, 16, 8, 16, 32, 32, 3.0, (8, 100.0, (8.0, 64.0, 4.0, 1.0)), 150)], embedding_scale=4.0, bigram=None)
 # Layers at the widths of a real model's layers.
 WIDE = config(1024, 1000, 1e-5,
-              [latent(8, 96, 32, 128, 512, 96, 128 ** -0.5, (32, 10000.0, (8.0, 4096.0, 32.0, 1.0)), 100, dense(2048)),
+              [latent(8, 96, 32, 128, 512, 96, 128 ** -0.5, (32, 10000.0, (6.0, 4096.0, 24.0, 1.0)), 100, dense(2048)),
                sloped(8, 2, 128, 128, 128 ** -0.5, 150, True, dense(2048)),
                latent(32, 64, 64, 64, 256, 64, 128 ** -0.5, (64, 10000.0), 77, dense(1024)),
                sloped(16, 2, 64, 128, 64 ** -0.5, 64, True, dense(1024))],
