@@ -55,7 +55,8 @@ def takes(x, w, gated=False):
 
 
 def run(x, w, out_dtype, fuse_swiglu=False, resident=False, row_sums=None, into=None, bias=None):
-    """Same contract as ``gemm_skinny.run``; ``bias`` (the gated product: float32 [2N]) is added before the gating; sums of squares are laid out [tile of 128 columns][128]."""
+    """Arguments and results as ``gemm_skinny.run``'s; ``bias`` (the gated product: float32 [2N]) is added before the gating; sums of
+    squares are laid out [tile of 128 columns][128]."""
     M, K = x.shape
     n_out = w.shape[0] // 2 if fuse_swiglu else w.shape[0]
     counters, partials = _device_state(x.device)
@@ -76,6 +77,7 @@ def run(x, w, out_dtype, fuse_swiglu=False, resident=False, row_sums=None, into=
                   gain.data_ptr() if gain is not None else None, scaled.data_ptr() if scaled is not None else None, n_out,
                   sums_out.data_ptr() if sums_out is not None else None,
                   sums_in.data_ptr() if sums_in is not None else None, parts, 1.0 / width, float(eps),
-                  None if bias is None else bias.data_ptr(), partials.data_ptr(), partials.numel(), counters.data_ptr(), counters.numel(),
+                  None if bias is None else bias.data_ptr(), partials.data_ptr(), partials.numel(), counters.data_ptr(),
+                  counters.numel(),
                   _library.status_word(x.device).data_ptr(), _library.current_stream())
     return result
